@@ -433,6 +433,111 @@ int ds41_act_quant_nvfp4_rows(const void* x, long long ldx, void* q, long long l
                               float global_scale, const int* rows_dev, int batch, long long x_batch_stride,
                               long long q_batch_stride, long long sf_batch_stride, const int* n_active, void* stream);
 
+// ---------------------------------------------------------------------------------------------------
+// Layer stacks with one fp32 residual stream (stack_ops.cu, latent_attn.cu, mlstm.cu, gemm_f32.cu).  `f32` selects 32-bit
+// activations, cache rows and weights; 0 = bf16 (the streams, norms, gates, scores and recurrent states are fp32 in both).
+//
+// A projection as its consumer reads it: columns [col, ...) of `splits` fp32 planes [rows][ld] (split-K partial sums), or
+// of one bf16 matrix.  data == NULL: absent.
+typedef struct ds41_proj {
+  const void* data;
+  long long plane;      // elements between planes
+  int ld, splits, bf16, col;
+} ds41_proj;
+
+// Close a sublayer and open the next one; see stack_ops.cu.  x rows are fp32 with leading dimension ldx.
+typedef struct ds41_resid_args {
+  ds41_proj y;          // sublayer result (absent: only the norm / mix part runs)
+  ds41_proj gate;       // pre-activation of the sigmoid gate on the result (absent: no gate)
+  const float* gate_bias;
+  const float* post_w;  // weight of the norm of the gated result (NULL: added as it is)
+  const int* tokens;    // not NULL: the row starts as embed[token] (bf16) instead of x_in
+  const void* embed;
+  long long embed_ld;
+  const float* x_in;
+  float* x_out;         // the stream after the addition
+  const float* mix;     // not NULL: x_avg = sum_j mix[j] * kept[j], j < n_mix; kept[n_mix - 1] is the row just computed
+  const float* kept;
+  long long kept_stride;
+  float* x_avg;
+  const float* next_w;  // not NULL: h = norm(stream) * next_w
+  void* h;
+  long long ldx;
+  int ldh, n_mix, vocab;
+  int rows, W;
+  int norm_kind;        // 0 layer norm without bias, 1 RMS norm
+  float eps;
+  int f32;
+} ds41_resid_args;
+int ds41_resid_step(const ds41_resid_args* args, void* stream);
+
+// out = a N(z) + b N(z^2) + c N(z^3) + e with coef = {a, b, c, e}, N(v) = v / sqrt(mean(v^2) + eps) over the row
+int ds41_polynorm(const ds41_proj* z, const float* coef, int rows, int ff, float eps, void* out, int ld_out, int f32,
+                  void* stream);
+// out = y * sigmoid(gate)
+int ds41_gate_mul(const ds41_proj* y, const ds41_proj* gate, int rows, int n, void* out, int ld_out, int f32, void* stream);
+// heads of `stride` columns, `width` of them live: o / rms(o) * w * sigmoid(gate)
+int ds41_head_norm_gate(const float* o, int ld_o, const ds41_proj* gate, const float* w, int rows, int heads, int width,
+                        int stride, float eps, void* out, int ld_out, int f32, void* stream);
+int ds41_gather_rows(const void* src, int ld, const int* index, int n_src, int rows, int W, void* dst, int f32,
+                     void* stream);
+
+typedef struct ds41_latent_post_args {
+  ds41_proj dq, kv, kr;           // query latent, key/value latent, shared rotated key part
+  const float* dq_norm;
+  const float* kv_norm;
+  const float* freq;              // [rot_dim / 2] rotation per position
+  void* cq;                       // [rows][ld_cq]
+  void* pool;                     // cache rows (NULL: this layer stores none)
+  const int* page_table;
+  const int* row_pos;
+  const int* row_slot;
+  float magnitude, eps;           // factor on cos and sin
+  int rows, q_rank, ld_cq, kv_rank, kv_pad, rot_dim, row_len, max_pages, page_tokens, f32;
+} ds41_latent_post_args;
+int ds41_latent_post(const ds41_latent_post_args* args, void* stream);
+int ds41_latent_query(const ds41_proj* q, const int* row_pos, const float* freq, float magnitude, int rows, int heads,
+                      int dim_pad, int rot_pad, int rot_dim, void* out, int ld_out, int f32, void* stream);
+// rows [0, n_keys) of the request that owns pass row `slot_row`: lat [n_keys][kv_pad], rot [n_keys][row_len - kv_pad]
+int ds41_latent_gather(const void* pool, const int* page_table, int max_pages, int page_tokens, int row_len, int kv_pad,
+                       int slot_row, const int* row_slot, int n_keys, void* lat, void* rot, int f32, void* stream);
+
+typedef struct ds41_latent_attend_args {
+  const void* q_abs;              // [rows][ld_q_abs]: head h at h * kv_pad (query times W_uk)
+  const void* q_rot;              // [rows][ld_q_rot]: head h at h * q_rot_stride, rotated
+  void* pool;
+  const int* page_table;
+  const int* row_pos;
+  const int* row_slot;
+  float* part_o;                  // [rows][n_splits][heads][kv_pad]
+  float* part_ml;                 // [rows][n_splits][heads]{maximum, sum}
+  long long ld_q_abs, ld_q_rot;
+  float scale;
+  int rows, heads, kv_pad, row_len, q_rot_stride, n_splits, max_pages, page_tokens, f32;
+} ds41_latent_attend_args;
+int ds41_latent_attend(const ds41_latent_attend_args* args, void* stream);
+int ds41_latent_merge(const float* part_o, const float* part_ml, const float* sink, int n_splits, int rows, int heads,
+                      int kv_pad, void* out, int ld_out, int f32, void* stream);
+
+typedef struct ds41_mlstm_args {
+  ds41_proj q, k, v, gate_i, gate_f;     // q, k: heads x dim_pad; v: heads x vdim_pad; gates: heads
+  const float* bias_i;
+  const float* bias_f;
+  const int* row_pos;
+  const int* row_slot;
+  float* state_s;                 // [slots][heads][dim_pad][vdim_pad]
+  float* state_n;                 // [slots][heads][ceil(vdim_pad / 32)][dim_pad]
+  float* state_m;                 // [slots][heads][ceil(vdim_pad / 32)]
+  float* out;                     // [rows][ld_out]
+  float gate_cap, q_scale, den_eps;
+  int rows, heads, dim_pad, vdim_pad, slots, ld_out;
+} ds41_mlstm_args;
+int ds41_mlstm_step(const ds41_mlstm_args* args, void* stream);
+
+int ds41_gemm_f32(const float* A, const float* B, float* out, int M, int N, int K, long long lda, long long ldb,
+                  long long ldo, int batch, long long a_batch_stride, long long b_batch_stride,
+                  long long out_batch_stride, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -16,7 +16,7 @@ from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
 
-@dataclass
+@dataclass(frozen=True)
 class RopeConfig:
     theta: float = 10000.0
     # YaRN parameters; factor == 1 disables scaling.
@@ -24,6 +24,10 @@ class RopeConfig:
     beta_fast: float = 32.0
     beta_slow: float = 1.0
     original_max_position: int = 65536
+
+    @property
+    def scaled(self) -> bool:
+        return self.factor != 1.0
 
 
 @dataclass
@@ -321,7 +325,7 @@ def rope_inv_freq(rope: RopeConfig, dim: int) -> List[float]:
     correction when factor > 1 (native/cuda/kernels/v41_attention_ops.cu:328-341)."""
     half = dim // 2
     base = [rope.theta ** (-2.0 * i / dim) for i in range(half)]
-    if rope.factor <= 1.0:
+    if not rope.scaled:
         return base
 
     def corr_dim(rot: float) -> float:
@@ -329,11 +333,10 @@ def rope_inv_freq(rope: RopeConfig, dim: int) -> List[float]:
 
     low = max(math.floor(corr_dim(rope.beta_fast)), 0)
     high = min(math.ceil(corr_dim(rope.beta_slow)), dim - 1)
-    if high == low:
-        high += 0.001
+    span = max(high - low, 0.001)
     out = []
     for i in range(half):
-        ramp = min(max((i - low) / (high - low), 0.0), 1.0)
+        ramp = min(max((i - low) / span, 0.0), 1.0)
         mask = 1.0 - ramp            # 1 -> keep extrapolated (high-frequency) value
         out.append(base[i] / rope.factor * (1 - mask) + base[i] * mask)
     return out

@@ -30,6 +30,8 @@ from ..ops import attention as A
 from ..ops import gemm as G
 from ..ops import lib
 from ..parallel.fabric import Fabric, SymBuffer
+from .base import RowsEngine
+from .paged import PagedSlots
 
 BF16 = torch.bfloat16
 F32 = torch.float32
@@ -459,7 +461,7 @@ class KVSnapshot:
         return n + sum(t.numel() * t.element_size() for t in self.pending.values())
 
 
-class KVCache:
+class KVCache(PagedSlots):
     """Window rings, paged compressed pools and the page table for `slots` concurrent requests.
 
     A page covers `page_tokens` token positions; a source with compress ratio r stores
@@ -469,7 +471,8 @@ class KVCache:
     def __init__(self, cfg: ModelConfig, n_layers: int, slots: int, max_ctx: int, device, page_tokens: int = 64,
                  n_pages: Optional[int] = None, spec_slack: int = 16, kv_dtype: str = "bf16",
                  index_dtype: Optional[str] = None):
-        self.cfg, self.slots, self.max_ctx, self.page_tokens = cfg, slots, max_ctx, page_tokens
+        self.cfg = cfg
+        self._init_pages(slots, max_ctx, device, page_tokens, n_pages)
         assert kv_dtype in ("bf16", "fp8", "fp4")
         self.kv_dtype = kv_dtype
         # index keys: "fp4" = E2M1 pairs + one UE8M0 scale per 32 values (68 bytes per key of 128 values instead of
@@ -488,8 +491,6 @@ class KVCache:
         D = cfg.head_dim
         ring = cfg.window + spec_slack
         self.ring = ring
-        self.max_pages = (max_ctx + page_tokens - 1) // page_tokens
-        self.n_pages = n_pages if n_pages is not None else self.max_pages * slots
         kv_shape, kv_dt = ((D,), BF16) if self.row_bytes == 0 else ((self.row_bytes,), torch.uint8)
         self.win = torch.zeros(n_layers, slots, ring, *kv_shape, dtype=kv_dt, device=device)
         self.comp: Dict[int, torch.Tensor] = {}
@@ -508,62 +509,6 @@ class KVCache:
                              torch.zeros(self.n_pages * pr, cfg.index_dim, dtype=BF16, device=device))
             if ratio == 2:
                 self.pending[src] = torch.zeros(slots, 4, 2 * D, dtype=F32, device=device)
-        self.page_table_host = torch.full((slots, self.max_pages), -1, dtype=I32)
-        self.page_table = self.page_table_host.to(device)
-        # Pages, reference counts and slot leases live in the host runtime's allocator (csrc/core/kvalloc.cc); this
-        # class only mirrors each slot's page list into the device page table.
-        from ..runtime import core as K
-        self.alloc = K.KvAllocator(self.n_pages, slots, page_tokens)
-
-    # ------------------------------------------------------------------ slots and pages
-    @property
-    def free_pages(self) -> int:
-        return self.alloc.free_pages
-
-    def pages_of(self, slot: int) -> List[int]:
-        return self.alloc.pages(slot)
-
-    def admit(self):
-        """Lease a free slot -> (slot, generation), or None when every slot is taken."""
-        return self.alloc.admit()
-
-    def _gen(self, slot: int) -> int:
-        """Generation of the slot's lease; a slot used without admit() (single-request drivers) is leased here."""
-        g = self.alloc.generation(slot)
-        if g == 0:
-            g = self.alloc.admit_slot(slot)
-            assert g is not None
-        return g
-
-    def _publish(self, slot: int, first: int = 0):
-        pages = self.alloc.pages(slot)
-        n = len(pages)
-        if n > first:
-            self.page_table_host[slot, first:n] = torch.tensor(pages[first:], dtype=I32)
-            self.page_table[slot, first:n].copy_(self.page_table_host[slot, first:n], non_blocking=True)
-
-    def ensure(self, slot: int, n_tokens: int) -> bool:
-        """Make sure `slot` has pages for positions [0, n_tokens).  Returns False when the pool is exhausted."""
-        need = (n_tokens + self.page_tokens - 1) // self.page_tokens
-        if need > self.max_pages:
-            return False
-        gen = self._gen(slot)
-        have = self.alloc.page_count(slot)
-        if need <= have:
-            return True
-        try:
-            self.alloc.ensure(slot, gen, n_tokens)
-        except MemoryError:
-            return False
-        self._publish(slot, have)
-        return True
-
-    def release(self, slot: int):
-        g = self.alloc.generation(slot)
-        if g:
-            self.alloc.retire(slot, g)
-        self.page_table_host[slot].fill_(-1)
-        self.page_table[slot].fill_(-1)
 
     # ------------------------------------------------------------------ prefix snapshots
     def snapshot(self, slot: int, n_tokens: int) -> KVSnapshot:
@@ -630,17 +575,12 @@ class KVCache:
             self.pending[src][slot].copy_(t)
         return True
 
-    def drop_snapshot(self, snap: KVSnapshot):
-        if snap.pages:
-            self.alloc.release_pages(snap.pages)
-        snap.pages = []
-
     def nbytes(self) -> int:
         ts = [self.win] + list(self.comp.values()) + list(self.idx.values()) + list(self.pending.values())
         return sum(t.numel() * t.element_size() for t in ts)
 
 
-class DS41Engine:
+class DS41Engine(RowsEngine):
     def __init__(self, cfg: ModelConfig, weights: EngineWeights, fabric: Optional[Fabric] = None, *,
                  max_rows: int = 8, slots: int = 1, max_ctx: int = 4096, page_tokens: int = 64,
                  n_pages: Optional[int] = None, row_hi: bool = False, moe_rows: int = 32, kv_dtype: str = "bf16",
@@ -808,17 +748,9 @@ class DS41Engine:
         self.inv_long = torch.tensor(rope_inv_freq(cfg.rope_long, cfg.rope_dim), dtype=F32, device=dev)
         self.inv_idx = torch.tensor(rope_inv_freq(cfg.rope_long, cfg.index_dim // 2), dtype=F32, device=dev)
         self.layer_prefix_plain = False   # drafter blocks use the plain rope
-        self.launches = 0
-        self.only = None
-        from ..utils.trace import ActivationTrace
-        self.layer_timer = None   # utils.trace.LayerTimer: device time per layer of eager passes
-        # DS41_NVTX=1: every launch sits in an NVTX range named after its kernel class (for timeline tools)
-        import os
-        self.nvtx = os.environ.get("DS41_NVTX", "") == "1"
-        self.activation_trace = ActivationTrace.from_env()
+        self._init_instruments()
         self._pass_hint = None    # (rows, highest position) of a single-request pass described by the last set_rows
         self.image_patch = None   # (image rows, pass-row ids) applied after the embedding lookup of the next pass
-        self.timeline = None   # set to a list to record (tag, start event, end event) per launch of eager passes
         # Engram memory layers: layer -> (EngramLayer, pinned host rows [max_rows * rows_per_token, row_bytes], device
         # text mask [max_rows] uint8).  A layer takes part in a pass only after set_engram_rows() filled its host rows.
         self.engram: Dict[int, tuple] = {}
@@ -868,31 +800,6 @@ class DS41Engine:
         """Split-K factor of a swap-AB projection: fill one wave of CTAs, counting the row tiles of long passes."""
         n_tiles = (rows + G.pick_bn(rows) - 1) // G.pick_bn(rows)
         return G.pick_splits(m, k, max_splits=self.max_splits, n_tiles=n_tiles)
-
-    def _run(self, tag, fn, *args, **kw):
-        """Launch one kernel; `self.only` (a set of tags) restricts a pass to some kernels for profiling."""
-        if self.only is not None and tag not in self.only:
-            return
-        self.launches += 1
-        if self.nvtx:
-            torch.cuda.nvtx.range_push(tag)
-            try:
-                err = fn(*args, **kw)
-            finally:
-                torch.cuda.nvtx.range_pop()
-            if err is not None:
-                lib.check(err, tag)
-            return
-        if self.timeline is not None:           # eager passes only: a CUDA event pair around every launch
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            err = fn(*args, **kw)
-            e1.record()
-            self.timeline.append((tag, e0, e1))
-        else:
-            err = fn(*args, **kw)
-        if err is not None:
-            lib.check(err, tag)
 
     def set_rows(self, tokens, positions, slots, row_hi=None, row_lo=None):
         """Host -> device copy of one pass's inputs (lists or CPU tensors).  `row_lo` (one position per row) puts a
@@ -1336,7 +1243,7 @@ class DS41Engine:
                 # the layer's output is merged into the streams by the next sublayer; the dump shows the streams as
                 # they stand plus the pending expert plane of this rank
                 self.activation_trace.dump(l, self.streams, self.row_pos, R)
-        self._pending = pending
+        self._pending, self._rows_run = pending, R
         if self._pass_hint is not None and self._pass_hint[1] >= 0:
             self._pass_hint = None        # a long pass's key count holds for that pass only; the static form stays until
                                           # the rows are described again (device-fed steps keep their slot)
@@ -1707,22 +1614,6 @@ class DS41Engine:
                       lib.ptr(self.extras), C.c_float(cfg.norm_eps), self.cache.row_bytes, st())
 
     # ------------------------------------------------------------------ convenience drivers
-    def prefill(self, slot: int, tokens: List[int], start: int = 0, chunk: Optional[int] = None) -> int:
-        """Run the prompt through the engine in chunks of up to max_rows rows; returns the greedy next token."""
-        chunk = chunk or self.max_rows
-        assert self.cache.ensure(slot, start + len(tokens) + 1)
-        nxt = -1
-        for c0 in range(0, len(tokens), chunk):
-            part = tokens[c0:c0 + chunk]
-            pos = list(range(start + c0, start + c0 + len(part)))
-            self.set_rows(part, pos, [slot] * len(part))
-            last = c0 + chunk >= len(tokens)
-            # a chunk may run padded up to the row-sharded granularity (the padding rows have no slot)
-            self.forward_rows(self.sp_rows(len(part)), head=last, head_row=len(part) - 1)
-            if last:
-                nxt = int(self.chosen[self.last_head_row].item())
-        return nxt
-
     def boundary_source(self, rows: int, layer: int, sources: bool = True):
         """Finish an encoder slice at `layer`: merge the pending sublayer into the streams, normalise layer `layer`'s
         input and run only its projection + compressor, so that its compressed source covers these rows.  Afterwards
@@ -1836,5 +1727,18 @@ class DS41Engine:
         dist.all_gather(parts, local, group=self.fabric.group)
         return torch.cat(parts, dim=1)
 
-    def check_status(self, what: str = "engine pass"):
-        lib.raise_on_status(self.status, what)
+    def logits_at(self, rows: List[int]) -> torch.Tensor:
+        """fp32 logits of any rows of the last pass, which ran with head=False (one rank); consumes the pass."""
+        assert self.world == 1 and self._sp_active is None
+        lw0 = self._lw_any
+        self._hc(self._rows_run, self._pending, lw0.hc_attn_fn, lw0.hc_attn_scale, lw0.hc_attn_base, self.w.final_norm)
+        self._pending = None
+        out = []
+        for i in range(0, len(rows), self.head_cap):
+            part = torch.tensor(list(rows[i:i + self.head_cap]), device=self.device)
+            x = self.xn.index_select(0, part)
+            self._run("gemm_head", G.gemm_raw, self.w.head, x, self.logits, self.V_local, len(part), self.cfg.hidden,
+                      lda=self.cfg.hidden, ldb=self.cfg.hidden, ldo=self.V_local, out_mode=3, status=self.status,
+                      static_operand=1)
+            out.append(self.logits[:len(part)].clone())
+        return torch.cat(out)

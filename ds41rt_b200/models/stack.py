@@ -1,0 +1,519 @@
+"""Execution of layer-stack models (stack_config.StackConfig) with the hand-written sm_100a kernels.
+
+`StackEngine` enqueues one pass over rows as a fixed sequence of launches: the residual step (csrc/kernels/stack_ops.cu)
+closes a sublayer and opens the next one, the mixers (`MIXERS`) and the feed-forward part run between.  Everything that
+depends on data stays on the device, so a decode pass is captured as a CUDA graph.  `dtype="bf16"` is the serving form
+(matrix products and activations in bf16 with fp32 accumulation; streams, norms, gates, attention weights and recurrent
+states in fp32); `dtype="f32"` keeps everything in true 32-bit.
+
+`StackCache` holds what a request leaves behind: paged latent rows of the attention layers that produce them (a layer that
+reads another layer's rows has none of its own) and one recurrent state per slot and recurrent layer.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import torch
+
+from ..config import rope_inv_freq
+from ..ops import lib
+from ..ops import stack as S
+from ..ops.stack import Matrix, Proj, ceil_to
+from ..stack_config import LatentAttentionSpec, MLSTMSpec, StackConfig
+from .base import RowsEngine
+from .paged import PagedSlots
+
+BF16, F32, I32 = torch.bfloat16, torch.float32, torch.int32
+DTYPES = {"bf16": BF16, "f32": F32}
+
+
+# ---------------------------------------------------------------------------------------------------- cache and states
+@dataclass
+class StackSnapshot:
+    """State of one request after `n_tokens` positions.  Full pages are shared by reference (they are never written
+    again); the rows of the partly filled last page and the recurrent states are copied."""
+    n_tokens: int
+    pages: List[int]
+    partial: Dict[int, torch.Tensor]
+    states: Dict[int, Tuple[torch.Tensor, ...]]
+
+    def nbytes(self) -> int:
+        ts = list(self.partial.values()) + [t for st in self.states.values() for t in st]
+        return sum(t.numel() * t.element_size() for t in ts)
+
+
+def latent_row_len(m: LatentAttentionSpec) -> Tuple[int, int]:
+    """(padded latent width, cache row length): [latent | rotated key part], both padded to 16 values."""
+    kv = ceil_to(m.kv_rank, 16)
+    return kv, kv + ceil_to(m.rot_dim, 16)
+
+
+def mlstm_state_shapes(m: MLSTMSpec) -> Tuple[Tuple[int, ...], ...]:
+    d, v = ceil_to(m.dim, 16), ceil_to(m.vdim, 16)
+    nb = -(-v // S.STATE_COLS)
+    return (m.heads, d, v), (m.heads, nb, d), (m.heads, nb)
+
+
+class StackCache(PagedSlots):
+    def __init__(self, cfg: StackConfig, slots: int, max_ctx: int, device, dtype=BF16, page_tokens: int = 64,
+                 n_pages: Optional[int] = None):
+        self.cfg, self.dtype = cfg, dtype
+        self._init_pages(slots, max_ctx, device, page_tokens, n_pages)
+        self.pools: Dict[int, torch.Tensor] = {}
+        for l in cfg.cache_layers():
+            row = latent_row_len(cfg.layers[l].mixer)[1]
+            self.pools[l] = torch.zeros(self.n_pages * page_tokens, row, dtype=dtype, device=device)
+        self.states: Dict[int, Tuple[torch.Tensor, ...]] = {
+            l: tuple(torch.zeros(slots, *shape, dtype=F32, device=device)
+                     for shape in mlstm_state_shapes(cfg.layers[l].mixer)) for l in cfg.state_layers()}
+
+    def snapshot(self, slot: int, n_tokens: int) -> StackSnapshot:
+        """Capture `slot`, whose last pass ended at position n_tokens - 1 (call it between passes, on the stream)."""
+        P = self.page_tokens
+        full, rem = n_tokens // P, n_tokens % P
+        mine = self.alloc.pages(slot)
+        pages = self.alloc.retain(slot, self._gen(slot), min(full, len(mine)))
+        partial = {}
+        if rem and full < len(mine):
+            at = mine[full] * P
+            partial = {l: t[at:at + rem].clone() for l, t in self.pools.items()}
+        return StackSnapshot(n_tokens, pages, partial,
+                             {l: tuple(t[slot].clone() for t in st) for l, st in self.states.items()})
+
+    def restore(self, slot: int, snap: StackSnapshot) -> bool:
+        """Continue a snapshot in an empty `slot`.  Returns False when no page is free for the partly filled page."""
+        gen = self._gen(slot)
+        assert self.alloc.page_count(slot) == 0, "restore needs an empty slot"
+        if snap.partial and self.alloc.free_pages == 0:
+            return False
+        self.alloc.share(slot, gen, snap.pages)
+        if snap.partial:
+            self.alloc.ensure(slot, gen, (len(snap.pages) + 1) * self.page_tokens)
+            at = self.alloc.pages(slot)[len(snap.pages)] * self.page_tokens
+            for l, t in snap.partial.items():
+                self.pools[l][at:at + t.shape[0]].copy_(t)
+        self._publish(slot)
+        for l, st in snap.states.items():
+            for mine, kept in zip(self.states[l], st):
+                mine[slot].copy_(kept)
+        return True
+
+    def restore_prefix(self, slot: int, snap: StackSnapshot, n_tokens: int) -> bool:
+        """Only a snapshot's whole length can be continued where recurrent states belong to it."""
+        return n_tokens == snap.n_tokens and self.restore(slot, snap)
+
+    def nbytes(self) -> int:
+        ts = list(self.pools.values()) + [t for st in self.states.values() for t in st]
+        return sum(t.numel() * t.element_size() for t in ts)
+
+
+# ---------------------------------------------------------------------------------------------------- mixers
+class LatentAttention:
+    """Weights of a latent-attention layer in kernel layout and its launch sequence.
+
+    Head widths are padded to 16 values.  Two forms of the same attention: `absorbed` multiplies the queries by W_uk and
+    attends over the latent rows themselves (decode, short portions, mixed passes); `expanded` makes keys and values of
+    every visible position of one request first (long prompt passes)."""
+
+    def __init__(self, spec: LatentAttentionSpec, cfg: StackConfig, t: Dict[str, torch.Tensor], gate: Dict[str, torch.Tensor],
+                 device, dtype):
+        self.spec, self.cfg = spec, cfg
+        H, W = spec.heads, cfg.hidden
+        self.dp, self.rp, self.vp = ceil_to(spec.dim, 16), ceil_to(spec.rot_dim, 16), ceil_to(spec.vdim, 16)
+        self.kvp, self.row_len = latent_row_len(spec)
+        self.hs = self.dp + self.rp
+        own = spec.kv_from is None
+        parts = [("dq", t["dq"])]
+        if own:
+            parts += [("kv", t["dkv"][:spec.kv_rank]), ("kr", t["dkv"][spec.kv_rank:])]
+        parts += [("g", S.pad_heads(t["g"], H, spec.vdim, self.vp))]
+        if gate:
+            parts += [("gate", gate["w"])]
+        self.w_in, self.at = S.stack_rows(parts, device, dtype)
+        f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
+        self.dq_norm, self.sink = f32(t["dq.norm"]), f32(t["sink"])
+        self.kv_norm = f32(t["dkv.norm"]) if own else None
+        uq = t["uq"].view(H, spec.dim + spec.rot_dim, spec.q_rank)
+        self.w_uq = Matrix(torch.cat([S.pad_heads(uq[:, :spec.dim].reshape(-1, spec.q_rank), H, spec.dim, self.dp)
+                                      .view(H, self.dp, -1),
+                                      S.pad_heads(uq[:, spec.dim:].reshape(-1, spec.q_rank), H, spec.rot_dim, self.rp)
+                                      .view(H, self.rp, -1)], 1).reshape(H * self.hs, spec.q_rank), device, dtype)
+        uk = S.pad_heads(t["uk"], H, spec.dim, self.dp)              # [H * dp, kv_rank]
+        uv = S.pad_heads(t["uv"], H, spec.vdim, self.vp)
+        z = lambda *shape: torch.zeros(*shape, dtype=dtype, device=device)
+        self.w_ukt = z(H, self.kvp, self.dp)                         # per head: latent value <- query value
+        self.w_ukt[:, :spec.kv_rank] = uk.view(H, self.dp, spec.kv_rank).transpose(1, 2).to(device=device, dtype=dtype)
+        ukv = z(H * (self.dp + self.vp), self.kvp)                   # keys of all heads, then values of all heads
+        ukv[:, :spec.kv_rank] = torch.cat([uk, uv], 0).to(device=device, dtype=dtype)
+        self.w_ukv = Matrix(ukv, device, dtype)
+        self.w_uv = self.w_ukv.w[H * self.dp:]
+        self.w_o = Matrix(S.pad_heads(t["o"].t().contiguous(), H, spec.vdim, self.vp).t(), device, dtype)
+        freq = rope_inv_freq(spec.rope, spec.rot_dim) if spec.rope is not None else [0.0] * (spec.rot_dim // 2)
+        self.freq = torch.tensor(freq or [0.0], dtype=F32, device=device)
+
+    def matrices(self):
+        return {"a": [(self.w_in.n, self.w_in.k)], "b": [(self.w_uq.n, self.w_uq.k), (self.w_o.n, self.w_o.k)]}
+
+    def run(self, e: "StackEngine", l: int, R: int, src: int) -> Tuple[Proj, Optional[Proj]]:
+        sp, k, H = self.spec, e.k, self.spec.heads
+        pin = e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
+        pool = e.cache.pools[src]
+        a = S.LatentPostArgs()
+        a.dq, a.dq_norm = pin.at(self.at["dq"]).args(), self.dq_norm.data_ptr()
+        a.cq, a.ld_cq, a.q_rank = e.cq.data_ptr(), e.cq.shape[1], sp.q_rank
+        if sp.kv_from is None:
+            a.kv, a.kr, a.kv_norm = pin.at(self.at["kv"]).args(), pin.at(self.at["kr"]).args(), self.kv_norm.data_ptr()
+            a.pool, a.freq, a.magnitude = pool.data_ptr(), self.freq.data_ptr(), sp.magnitude
+        a.page_table, a.row_pos, a.row_slot = e.cache.page_table.data_ptr(), e.row_pos.data_ptr(), e.row_slot.data_ptr()
+        a.eps, a.rows, a.kv_rank, a.kv_pad, a.rot_dim = self.cfg.norm_eps, R, sp.kv_rank, self.kvp, sp.rot_dim
+        a.row_len, a.max_pages, a.page_tokens, a.f32 = self.row_len, e.cache.max_pages, e.cache.page_tokens, e.f32
+        e._run("latent_post", k.ds41_latent_post, C.byref(a), lib.stream())
+        ldq = H * self.hs
+        q = e.project("gemm_uq", e.cq, e.cq.shape[1], R, self.w_uq, e.planes_b)
+        e._run("latent_query", k.ds41_latent_query, C.byref(q.args()), lib.ptr(e.row_pos), lib.ptr(self.freq),
+               C.c_float(sp.magnitude), R, H, self.dp, self.rp, sp.rot_dim, lib.ptr(e.q), ldq, e.f32, lib.stream())
+        self._absorbed(e, R, ldq, pool, pin.at(self.at["g"]))
+        y = e.project("gemm_o", e.act, H * self.vp, R, self.w_o, e.planes_b)
+        return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
+
+    def _absorbed(self, e: "StackEngine", R: int, ldq: int, pool, gate: Proj):
+        sp, k, H = self.spec, e.k, self.spec.heads
+        q = e.q.view(-1)
+        for r0 in range(0, R, e.attn_rows):
+            n = min(e.attn_rows, R - r0)
+            qr = q[r0 * ldq:]
+            e._run("absorb_q", S.per_head, qr, ldq, self.hs, n, H, self.w_ukt, self.kvp, self.dp, self.dp, e.q_abs,
+                   H * self.kvp, e.status)
+            splits = e.attn_splits(n, H)
+            a = S.LatentAttendArgs()
+            a.q_abs, a.ld_q_abs = e.q_abs.data_ptr(), H * self.kvp
+            a.q_rot, a.ld_q_rot, a.q_rot_stride = qr[self.dp:].data_ptr(), ldq, self.hs
+            a.pool, a.page_table = pool.data_ptr(), e.cache.page_table.data_ptr()
+            a.row_pos, a.row_slot = e.row_pos[r0:].data_ptr(), e.row_slot[r0:].data_ptr()
+            a.part_o, a.part_ml = e.part_o.data_ptr(), e.part_ml.data_ptr()
+            a.scale, a.rows, a.heads, a.kv_pad, a.row_len, a.n_splits = sp.scale, n, H, self.kvp, self.row_len, splits
+            a.max_pages, a.page_tokens, a.f32 = e.cache.max_pages, e.cache.page_tokens, e.f32
+            e._run("latent_attend", k.ds41_latent_attend, C.byref(a), lib.stream())
+            e._run("latent_merge", k.ds41_latent_merge, lib.ptr(e.part_o), lib.ptr(e.part_ml), lib.ptr(self.sink), splits, n,
+                   H, self.kvp, lib.ptr(e.o_lat), H * self.kvp, e.f32, lib.stream())
+            o = e.o_heads.view(-1)[r0 * H * self.vp:]
+            e._run("values", S.per_head, e.o_lat, H * self.kvp, self.kvp, n, H, self.w_uv, self.vp, self.kvp, self.kvp, o,
+                   H * self.vp, e.status)
+        y = Proj(e.o_heads, H * self.vp)
+        e._run("gate_mul", k.ds41_gate_mul, C.byref(y.args()), C.byref(gate.args()), R, H * self.vp, lib.ptr(e.act),
+               H * self.vp, e.f32, lib.stream())
+
+
+class MLSTM:
+    def __init__(self, spec: MLSTMSpec, cfg: StackConfig, t: Dict[str, torch.Tensor], gate: Dict[str, torch.Tensor],
+                 device, dtype):
+        self.spec, self.cfg = spec, cfg
+        H = spec.heads
+        self.dp, self.vp = ceil_to(spec.dim, 16), ceil_to(spec.vdim, 16)
+        parts = [("q", S.pad_heads(t["q"], H, spec.dim, self.dp)), ("k", S.pad_heads(t["k"], H, spec.dim, self.dp)),
+                 ("v", S.pad_heads(t["v"], H, spec.vdim, self.vp)), ("g", S.pad_heads(t["g"], H, spec.vdim, self.vp)),
+                 ("i", t["i"]), ("f", t["f"])]
+        if gate:
+            parts += [("gate", gate["w"])]
+        self.w_in, self.at = S.stack_rows(parts, device, dtype)
+        f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
+        self.bias_i, self.bias_f = f32(t["i.b"]), f32(t["f.b"])
+        self.norm = f32(S.pad_heads(t["norm"], H, spec.vdim, self.vp))
+        self.w_o = Matrix(S.pad_heads(t["o"].t().contiguous(), H, spec.vdim, self.vp).t(), device, dtype)
+
+    def matrices(self):
+        return {"a": [(self.w_in.n, self.w_in.k)], "b": [(self.w_o.n, self.w_o.k)]}
+
+    def run(self, e: "StackEngine", l: int, R: int, src: Optional[int]) -> Tuple[Proj, Optional[Proj]]:
+        sp, k, H = self.spec, e.k, self.spec.heads
+        pin = e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
+        ld = H * self.vp
+        s, n, m = e.cache.states[l]
+        a = S.MlstmArgs()
+        a.q, a.k, a.v = (pin.at(self.at[x]).args() for x in "qkv")
+        a.gate_i, a.gate_f = pin.at(self.at["i"]).args(), pin.at(self.at["f"]).args()
+        a.bias_i, a.bias_f = self.bias_i.data_ptr(), self.bias_f.data_ptr()
+        a.row_pos, a.row_slot = e.row_pos.data_ptr(), e.row_slot.data_ptr()
+        a.state_s, a.state_n, a.state_m, a.out = s.data_ptr(), n.data_ptr(), m.data_ptr(), e.o_heads.data_ptr()
+        a.gate_cap, a.q_scale, a.den_eps = sp.gate_cap, sp.dim ** -0.5, sp.den_eps
+        a.rows, a.heads, a.dim_pad, a.vdim_pad, a.slots, a.ld_out = R, H, self.dp, self.vp, e.cache.slots, ld
+        e._run("mlstm_step", k.ds41_mlstm_step, C.byref(a), lib.stream())
+        e._run("head_norm_gate", k.ds41_head_norm_gate, lib.ptr(e.o_heads), ld, C.byref(pin.at(self.at["g"]).args()),
+               lib.ptr(self.norm), R, H, sp.vdim, self.vp, C.c_float(self.cfg.norm_eps), lib.ptr(e.act), ld, e.f32,
+               lib.stream())
+        y = e.project("gemm_o", e.act, ld, R, self.w_o, e.planes_b)
+        return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
+
+
+MIXERS = {"latent_attention": LatentAttention, "mlstm": MLSTM}
+
+
+class DenseMLP:
+    def __init__(self, spec, cfg: StackConfig, t: Dict[str, torch.Tensor], gate: Dict[str, torch.Tensor], device, dtype):
+        assert spec.activation == "polynorm"
+        self.spec, self.cfg = spec, cfg
+        self.ffp = ceil_to(spec.ff, 8)
+        parts = [("up", t["up"])] + ([("gate", gate["w"])] if gate else [])
+        self.w_up, self.at = S.stack_rows(parts, device, dtype)
+        self.coef = t["act"].to(device=device, dtype=F32).contiguous()
+        self.w_down = Matrix(t["down"], device, dtype)
+
+    def matrices(self):
+        return {"a": [(self.w_up.n, self.w_up.k)], "b": [(self.w_down.n, self.w_down.k)]}
+
+    def run(self, e: "StackEngine", R: int) -> Tuple[Proj, Optional[Proj]]:
+        pin = e.project("gemm_up", e.h, e.ldh, R, self.w_up, e.planes_a)
+        e._run("polynorm", e.k.ds41_polynorm, C.byref(pin.at(self.at["up"]).args()), lib.ptr(self.coef), R, self.spec.ff,
+               C.c_float(self.cfg.norm_eps), lib.ptr(e.act), self.ffp, e.f32, lib.stream())
+        y = e.project("gemm_down", e.act, self.ffp, R, self.w_down, e.planes_b)
+        return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
+
+
+# ---------------------------------------------------------------------------------------------------- weights
+@dataclass
+class StackLayer:
+    mixer: object
+    norm1: torch.Tensor
+    norm1b: Optional[torch.Tensor]
+    bias1: Optional[torch.Tensor]
+    mlp: Optional[DenseMLP] = None
+    norm2: Optional[torch.Tensor] = None
+    norm2b: Optional[torch.Tensor] = None
+    bias2: Optional[torch.Tensor] = None
+    mix: Optional[torch.Tensor] = None
+
+
+class StackWeights:
+    """Kernel-layout weights built from a family's tensors: `get(l)` returns layer l's tensors under canonical names
+    (mixer tensors "mix.*", feed-forward "mlp.*", norms, "rg1" / "rg1.b" / "rg2" / "rg2.b", "dwa"); `top` has "embed",
+    "final.norm" and "head"."""
+
+    def __init__(self, cfg: StackConfig, get, top: Dict[str, torch.Tensor], device, dtype: str = "bf16"):
+        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
+        dt = DTYPES[dtype]
+        f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
+        self.embed = Matrix(top["embed"], device, BF16)
+        self.final_norm = f32(top["final.norm"])
+        self.head = Matrix(top["head"], device, dt)
+        self.layers: List[StackLayer] = []
+        for l, spec in enumerate(cfg.layers):
+            t = get(l)
+            part = lambda p: {n[len(p):]: x for n, x in t.items() if n.startswith(p)}
+            gate = lambda n: {"w": t[n]} if cfg.residual_gate else {}
+            bias = lambda n: f32(t[n]) if cfg.residual_gate else None
+            post = lambda n: f32(t[n]) if cfg.post_norm else None
+            lw = StackLayer(MIXERS[spec.mixer.kind](spec.mixer, cfg, part("mix."), gate("rg1"), device, dt),
+                            f32(t["norm1"]), post("norm1b"), bias("rg1.b"))
+            if spec.mlp is not None:
+                lw.mlp = DenseMLP(spec.mlp, cfg, part("mlp."), gate("rg2"), device, dt)
+                lw.norm2, lw.norm2b, lw.bias2 = f32(t["norm2"]), post("norm2b"), bias("rg2.b")
+            if cfg.depth_average:
+                lw.mix = f32(t["dwa"])
+            self.layers.append(lw)
+
+    def nbytes(self) -> int:
+        seen, total, todo = set(), 0, [self]
+        while todo:
+            o = todo.pop()
+            for v in (vars(o).values() if not isinstance(o, (list, tuple)) else o):
+                if isinstance(v, torch.Tensor):
+                    if v.untyped_storage().data_ptr() not in seen:
+                        seen.add(v.untyped_storage().data_ptr())
+                        total += v.untyped_storage().nbytes()
+                elif isinstance(v, (list, Matrix, StackLayer, DenseMLP) + tuple(MIXERS.values())):
+                    todo.append(v)
+        return total
+
+
+# ---------------------------------------------------------------------------------------------------- engine
+class StackEngine(RowsEngine):
+    partial_prefix = False        # recurrent states belong to a snapshot's whole length
+    replay_window = 1 << 30       # the prefix banks then never prefer a truncated snapshot
+    engram: dict = {}
+    taps = None
+
+    def __init__(self, cfg: StackConfig, weights: StackWeights, *, max_rows: int = 8, slots: int = 1, max_ctx: int = 4096,
+                 page_tokens: int = 64, n_pages: Optional[int] = None):
+        self.cfg, self.w, self.device = cfg, weights, weights.device
+        self.rank, self.world = 0, 1
+        self.max_rows = R = max_rows
+        self.n_layers = cfg.n_layers
+        self.k = lib.kernels()
+        self.f32 = 1 if weights.dtype == "f32" else 0
+        dev, dt = self.device, DTYPES[weights.dtype]
+        self.cache = StackCache(cfg, slots, max_ctx, dev, dt, page_tokens, n_pages)
+        z = lambda shape, d: torch.zeros(shape, dtype=d, device=dev)
+        W = cfg.hidden
+        # inputs
+        self.in_tokens, self.row_pos = z((R,), I32), z((R,), I32)
+        self.row_slot = torch.full((R,), -1, dtype=I32, device=dev)
+        # residual streams: the kept result of every layer (depth average) and the working rows
+        self.ldx = ceil_to(W, 4)
+        self.kept = z((cfg.n_layers + 1 if cfg.depth_average else 1, R, self.ldx), F32)
+        self.x_mid, self.x_avg = z((R, self.ldx), F32), z((R, self.ldx), F32)
+        self.ldh = ceil_to(W, 8)
+        self.h = z((R, self.ldh), dt)
+        # projections
+        need = {"a": 8, "b": 8}
+        act = heads = q = 8
+        q_rank = 8
+        lat = 0
+        self.attn_rows = min(R, 256)
+        cells = 1
+        for lw in weights.layers:
+            for m in (lw.mixer, lw.mlp):
+                if m is not None:
+                    for b, ms in m.matrices().items():
+                        for n, kk in ms:
+                            need[b] = max(need[b], S.plane_floats(R, n, kk))
+            mx = lw.mixer
+            heads = max(heads, mx.spec.heads * mx.vp)
+            if lw.mlp is not None:
+                act = max(act, lw.mlp.ffp)
+            if isinstance(mx, LatentAttention):
+                q = max(q, mx.spec.heads * mx.hs)
+                q_rank = max(q_rank, mx.spec.q_rank)
+                lat = max(lat, mx.spec.heads * mx.kvp)
+                for n in range(1, self.attn_rows + 1):
+                    cells = max(cells, n * self.attn_splits(n, mx.spec.heads) * mx.spec.heads * mx.kvp)
+        self.planes_a, self.planes_b = z((need["a"],), F32), z((need["b"],), F32)
+        self.act = z((R * max(act, heads),), dt)
+        self.o_heads = z((R * heads,), F32)
+        if lat:
+            self.cq = z((R, ceil_to(q_rank, 8)), dt)
+            self.q = z((R * q,), dt)
+            self.q_abs, self.o_lat = z((self.attn_rows * lat,), dt), z((self.attn_rows * lat,), dt)
+            self.part_o, self.part_ml = z((cells,), F32), z((cells // 8 + 2,), F32)
+        # head
+        self.head_cap = min(R, 64)
+        self.last_head_row = 0
+        self.logits = z((self.head_cap, cfg.vocab), F32)
+        self.picked, self.pick_idx = z((self.head_cap, self.ldh), dt), z((self.head_cap,), I32)
+        self.best_val, self.chosen = z((R,), F32), z((R,), I32)
+        self.head_mask = None
+        self.image_patch = None
+        self.status = lib.new_status(dev)
+        self._init_instruments()
+        self.on_layer = None      # callable (layer, streams [rows, width]) after every layer of an eager pass
+
+    # ------------------------------------------------------------------ helpers
+    def attn_splits(self, rows: int, heads: int) -> int:
+        """Key splits per row of the absorbed attention: enough blocks to fill the GPU about twice, static per batch
+        size (a captured pass replays while the context grows)."""
+        want = -(-2 * 148 // (rows * -(-heads // 16)))
+        return max(1, min(want, 32, -(-self.cache.max_ctx // 64)))
+
+    def project(self, tag: str, x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor) -> Proj:
+        out: List[Proj] = []
+        self._run(tag, lambda: out.append(S.project(x, ldx, rows, m, buf, self.status)))
+        return out[0] if out else S.Proj(buf, m.out_ld)
+
+    def _enter_rehearsal(self):
+        self.row_slot.fill_(-1)       # no row owns a slot: caches and states keep what they hold
+
+    def set_rows(self, tokens, positions, slots, row_hi=None, row_lo=None):
+        """Host -> device copy of one pass's inputs.  Rows of one slot are adjacent, at consecutive positions."""
+        assert row_lo is None and row_hi is None, "a layer stack has no window floor"
+        n = len(positions)
+        assert n <= self.max_rows
+        slots, positions, seen = list(slots), list(positions), set()
+        for i in range(n):
+            if slots[i] < 0:
+                continue
+            if i and slots[i] == slots[i - 1]:
+                assert positions[i] == positions[i - 1] + 1, "rows of a request must follow one another"
+            else:
+                assert slots[i] not in seen, "rows of a request must be adjacent"
+                seen.add(slots[i])
+        pad = self.max_rows - n
+        if tokens is not None:
+            assert len(tokens) == n
+            self.in_tokens.copy_(torch.tensor(list(tokens) + [0] * pad, dtype=I32), non_blocking=True)
+        self.row_pos.copy_(torch.tensor(positions + [0] * pad, dtype=I32), non_blocking=True)
+        self.row_slot.copy_(torch.tensor(slots + [-1] * pad, dtype=I32), non_blocking=True)
+
+    def _resid(self, R: int, *, y: Optional[Proj] = None, gate: Optional[Proj] = None, bias=None, post=None, x_in=None,
+               x_out=None, layer: Optional[int] = None, next_w=None):
+        a = S.ResidArgs()
+        cfg = self.cfg
+        a.y, a.gate = (y.args() if y is not None else S.NO_PROJ), (gate.args() if gate is not None else S.NO_PROJ)
+        a.gate_bias, a.post_w, a.next_w = lib.ptr(bias), lib.ptr(post), lib.ptr(next_w)
+        if x_in is None:
+            a.tokens, a.embed, a.embed_ld = lib.ptr(self.in_tokens), lib.ptr(self.w.embed.w), self.w.embed.ld
+        a.x_in, a.x_out = lib.ptr(x_in), lib.ptr(x_out)
+        if layer is not None:
+            a.mix, a.kept, a.kept_stride = lib.ptr(self.w.layers[layer].mix), lib.ptr(self.kept), self.kept.stride(0)
+            a.n_mix, a.x_avg = layer + 2, lib.ptr(self.x_avg)
+        a.h, a.ldh, a.ldx, a.vocab, a.rows, a.W = lib.ptr(self.h), self.ldh, self.ldx, cfg.vocab, R, cfg.hidden
+        a.norm_kind, a.eps, a.f32 = cfg.norm_kind, cfg.norm_eps, self.f32
+        self._run("resid_step", self.k.ds41_resid_step, C.byref(a), lib.stream())
+
+    # ------------------------------------------------------------------ one pass
+    def forward_rows(self, rows: int, *, head: bool = True, head_row: Optional[int] = None, sources: bool = True):
+        """One pass over the `rows` rows described by set_rows()."""
+        cfg, R, layers = self.cfg, rows, self.w.layers
+        if self.layer_timer is not None:
+            self.layer_timer.begin()
+        cur = self.kept[0]
+        self._resid(R, x_out=cur, next_w=layers[0].norm1)
+        for l, lw in enumerate(layers):
+            after = layers[l + 1].norm1 if l + 1 < len(layers) else self.w.final_norm
+            done = self.kept[l + 1] if cfg.depth_average else self.kept[0]
+            mix = l if cfg.depth_average else None
+            y, gate = lw.mixer.run(self, l, R, cfg.source_of(l))
+            if lw.mlp is None:
+                self._resid(R, y=y, gate=gate, bias=lw.bias1, post=lw.norm1b, x_in=cur, x_out=done, layer=mix, next_w=after)
+            else:
+                self._resid(R, y=y, gate=gate, bias=lw.bias1, post=lw.norm1b, x_in=cur, x_out=self.x_mid, next_w=lw.norm2)
+                y, gate = lw.mlp.run(self, R)
+                self._resid(R, y=y, gate=gate, bias=lw.bias2, post=lw.norm2b, x_in=self.x_mid, x_out=done, layer=mix,
+                            next_w=after)
+            cur = self.x_avg if cfg.depth_average else self.kept[0]
+            if self.layer_timer is not None:
+                self.layer_timer.mark()
+            if self.activation_trace is not None:
+                self.activation_trace.dump(l, cur[:, :cfg.hidden], self.row_pos, R)
+            if self.on_layer is not None:
+                self.on_layer(l, cur[:R, :cfg.hidden])
+        if head:
+            self.head_rows(R if head_row is None else head_row + 1)
+
+    def _head_gemm(self, x: torch.Tensor, rows: int):
+        m = self.w.head
+        if self.f32:
+            self._run("gemm_head", S.gemm_f32, x, m.w, self.logits, rows, m.n, m.k, self.ldh, m.ld, self.cfg.vocab)
+        else:
+            from ..ops import gemm as G
+            self._run("gemm_head", G.gemm_raw, m.w, x, self.logits, m.n, rows, m.k, lda=m.ld, ldb=self.ldh,
+                      ldo=self.cfg.vocab, out_mode=3, status=self.status, static_operand=1)
+
+    def head_rows(self, rows: int, mask: Optional[torch.Tensor] = None):
+        """Logits and greedy choice of the pass's rows; a long pass only needs its last row, whose logits land in row 0."""
+        if mask is None:
+            mask = self.head_mask
+        x, self.last_head_row = self.h, rows - 1
+        if rows > self.head_cap:
+            x, rows, self.last_head_row = self.h[rows - 1:rows], 1, 0
+        self._head_gemm(x, rows)
+        V = self.cfg.vocab
+        self._run("argmax_rows", self.k.ds41_argmax_rows, lib.ptr(self.logits), C.c_longlong(V), rows, V, 0, lib.ptr(mask),
+                  0 if mask is None else mask.shape[-1], lib.ptr(self.best_val), lib.ptr(self.chosen), lib.ptr(None),
+                  lib.stream())
+
+    def logits_rows(self, rows: int) -> torch.Tensor:
+        return self.logits[:rows].clone()
+
+    def logits_at(self, rows: Sequence[int]) -> torch.Tensor:
+        """fp32 logits of any rows of the last pass (run with head=False or True), [len(rows), vocab]."""
+        out = []
+        for i in range(0, len(rows), self.head_cap):
+            part = list(rows[i:i + self.head_cap])
+            n = len(part)
+            self.pick_idx[:n].copy_(torch.tensor(part, dtype=I32))
+            self._run("gather_rows", self.k.ds41_gather_rows, lib.ptr(self.h), self.ldh, lib.ptr(self.pick_idx),
+                      self.max_rows, n, self.cfg.hidden, lib.ptr(self.picked), self.f32, lib.stream())
+            self._head_gemm(self.picked, n)
+            out.append(self.logits[:n].clone())
+        return torch.cat(out) if out else torch.empty(0, self.cfg.vocab, device=self.device)

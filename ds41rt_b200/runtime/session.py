@@ -16,12 +16,12 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..models.ds41 import DS41Engine
+from ..models.base import RowsEngine
 from ..ops import lib
 
 
 class DecodeSession:
-    def __init__(self, engine: DS41Engine, use_graphs: bool = True):
+    def __init__(self, engine: RowsEngine, use_graphs: bool = True):
         self.e = engine
         self.use_graphs = use_graphs and engine.device.type == "cuda"
         self.graphs: Dict[tuple, torch.cuda.CUDAGraph] = {}
@@ -46,20 +46,9 @@ class DecodeSession:
         if not self.use_graphs:
             return None
         if key not in self.graphs:
-            # one eager pass first: sets function attributes and warms every code path
-            snapshot = (self.e.in_tokens.clone(), self.e.row_pos.clone())
-            self._enqueue(rows, feedback)
-            torch.cuda.synchronize()
-            self.e.in_tokens.copy_(snapshot[0])
-            self.e.row_pos.copy_(snapshot[1])
             before = self.e.launches
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                self._enqueue(rows, feedback)
-            self.launches_per_graph[key] = self.e.launches - before
-            self.e.in_tokens.copy_(snapshot[0])
-            self.e.row_pos.copy_(snapshot[1])
-            self.graphs[key] = g
+            self.graphs[key] = self.e.capture(lambda: self._enqueue(rows, feedback))
+            self.launches_per_graph[key] = (self.e.launches - before) // 2      # an eager rehearsal, then the capture
         return self.graphs[key]
 
     # ------------------------------------------------------------------ stepping

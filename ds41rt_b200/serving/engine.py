@@ -164,7 +164,9 @@ class NativeBackend(Backend):
         self.e, self.eos = engine, eos
         # prompt passes use the encoder / decoder-replay split when the model has a boundary (config.ced_on)
         self.ced = ced
-        self.partial_reuse = True     # snapshots that share only a leading part with a prompt contribute that part
+        # snapshots that share only a leading part with a prompt contribute that part (not where a recurrent state
+        # belongs to the snapshot's whole length)
+        self.partial_reuse = engine.partial_prefix
         self.spec = None
         self.policy = None
         # runtime.engram.EngramPipeline or None.  Every pass hands its token ids to the pipeline first (hashes, page
@@ -187,7 +189,7 @@ class NativeBackend(Backend):
         self.lanes = K.Lanes(2)
         # Prompt and turn banks: the radix (csrc/core/prefix.cc) owns ids, reuse scores and the per-bank LRU; this map
         # holds what an id stands for: (token tuple, KVSnapshot, logits after the last token or None)
-        self.prefix = K.PrefixBanks(prompt_snapshots, turn_snapshots, engine.cfg.window)
+        self.prefix = K.PrefixBanks(prompt_snapshots, turn_snapshots, engine.replay_window)
         self.snapshots: Dict[int, tuple] = {}
         # pinned-host tier behind the banks: a snapshot that leaves the device (bank eviction, page pressure) is copied
         # there and comes back when a prompt extends it (runtime/hosttier.py)
@@ -427,7 +429,7 @@ class NativeBackend(Backend):
         first_new = reused
         if replay_from is not None:
             # a truncated snapshot: its compressed rows reach up to the common prefix's even boundary
-            first_new = replay_from + e.cfg.window
+            first_new = replay_from + e.replay_window
         req.events.put(Event("ready", usage={"prompt_tokens": len(req.prompt_ids), "prompt_cache_hit_tokens": reused}))
         self.totals["requests"] += 1
         self.totals["prompt_tokens"] += len(req.prompt_ids)
@@ -455,7 +457,7 @@ class NativeBackend(Backend):
         if hit is not None or part is not None:
             dev = self.prefix.lookup(prompt)
             if dev is not None and dev["id"] in self.snapshots:
-                dev_n = dev["frontier"] if dev["exact"] else max(0, dev["common"] // 2 * 2 - self.e.cfg.window)
+                dev_n = dev["frontier"] if dev["exact"] else max(0, dev["common"] // 2 * 2 - self.e.replay_window)
         if part is not None and part[1] > dev_n:
             # only a leading part is shared: its rows come back from the host, the last window before the cut is replayed
             sid, n = part
@@ -499,7 +501,7 @@ class NativeBackend(Backend):
                 break
             self.prefix.remove(hit["id"])                 # the map was cleared behind the radix: forget the id, look again
         toks, snap, logits = ent
-        window = e.cfg.window
+        window = e.replay_window
         n = len(toks)
         exact = hit["exact"] and n <= len(prompt) and not (n == len(prompt) and logits is None)
         score = n if exact else min(hit["common"], len(prompt) - 1) // 2 * 2 - window
@@ -575,7 +577,7 @@ class NativeBackend(Backend):
         cuts = [(c0, min(hi, c0 + step), hi == end) for lo, hi in ((first, start), (start, end))
                 for c0 in range(lo, hi, step)]
         taps_above = (self.spec is None or min(e.cfg.dspark.tap_layers) >= e.cfg.ced_boundary) \
-            and e.cfg.ced_replay >= e.cfg.window        # stored snapshots must hold complete decoder windows
+            and e.cfg.ced_replay >= e.replay_window        # stored snapshots must hold complete decoder windows
         if self.ced and first < end and not req.images and taps_above and e.ced_usable(first, end - first):
             pf.ced, pf.r0 = True, e.ced_replay_start(first, end)
             pf.passes = [("enc", c0, c1, fresh) for c0, c1, fresh in cuts]
@@ -886,19 +888,9 @@ class NativeBackend(Backend):
     # ------------------------------------------------------------------ decode rounds
     def _graph_for(self, rows: int):
         """Captured launch sequence of one `rows`-row decode pass (made on first use of a batch size)."""
-        import torch
         g = self._graphs.get(rows)
         if g is None:
-            e = self.e
-            keep = (e.in_tokens.clone(), e.row_pos.clone(), e.row_slot.clone())
-            e.forward_rows(rows)                      # eager pass first: kernel attributes, every code path warm
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                e.forward_rows(rows)
-            e.in_tokens.copy_(keep[0])
-            e.row_pos.copy_(keep[1])
-            e.row_slot.copy_(keep[2])
+            g = self.e.capture(lambda: self.e.forward_rows(rows))
             self._graphs[rows] = g
         return g
 

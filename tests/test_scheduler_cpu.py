@@ -8,12 +8,13 @@ import pytest
 import torch
 
 from ds41rt_b200.config import ModelConfig
+from ds41rt_b200.models.base import RowsEngine
 from ds41rt_b200.models.ds41 import KVCache
 from ds41rt_b200.serving.engine import GenRequest, NativeBackend
 from ds41rt_b200.serving.protocol import Sampling
 
 
-class FakeEngine:
+class FakeEngine(RowsEngine):
     def __init__(self, slots=2, max_ctx=512, n_pages=None, max_rows=64):
         self.cfg = ModelConfig.tiny()
         self.device = torch.device("cpu")
