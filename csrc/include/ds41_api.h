@@ -519,6 +519,21 @@ int ds41_latent_attend(const ds41_latent_attend_args* args, void* stream);
 int ds41_latent_merge(const float* part_o, const float* part_ml, const float* sink, int n_splits, int rows, int heads,
                       int kv_pad, void* out, int ld_out, int f32, void* stream);
 
+// Long prompt pass of one request over expanded keys and values (latent_prefill.cu): pass row r stands at position pos0 + r.
+typedef struct ds41_latent_prefill_args {
+  const void* q;                  // bf16 [rows][ld_q]: head h at h * (dim_pad + rot_pad): [unrotated | rotated]
+  const void* kv;                 // bf16 [n_keys][ld_kv]: unrotated keys of all heads, then values of all heads
+  const void* rot;                // bf16 [n_keys][rot_pad]: rotated key part shared by the heads
+  const float* sink;              // [heads] or NULL
+  void* out;                      // bf16 [rows][ld_out]: attention output (x sigmoid(gate) when given)
+  int* status;
+  ds41_proj gate;                 // [rows][heads * vdim_pad] or absent
+  long long ld_q, ld_kv;
+  float scale;
+  int rows, heads, dim_pad, rot_pad, vdim_pad, n_keys, pos0, ld_out;
+} ds41_latent_prefill_args;
+int ds41_latent_prefill(const ds41_latent_prefill_args* args, void* stream);
+
 typedef struct ds41_mlstm_args {
   ds41_proj q, k, v, gate_i, gate_f;     // q, k: heads x dim_pad; v: heads x vdim_pad; gates: heads
   const float* bias_i;
@@ -533,6 +548,8 @@ typedef struct ds41_mlstm_args {
   int rows, heads, dim_pad, vdim_pad, slots, ld_out;
 } ds41_mlstm_args;
 int ds41_mlstm_step(const ds41_mlstm_args* args, void* stream);
+// Long pass of one request (row 0's slot; adjacent rows), dim_pad <= 512; q, k, v are bf16 with 16-byte aligned rows.
+int ds41_mlstm_chunk(const ds41_mlstm_args* args, void* stream);
 
 int ds41_gemm_f32(const float* A, const float* B, float* out, int M, int N, int K, long long lda, long long ldb,
                   long long ldo, int batch, long long a_batch_stride, long long b_batch_stride,

@@ -8,6 +8,7 @@
 //  latent_attend : causal attention over the cache with absorbed queries (q W_uk, so that the latent row itself is key and
 //                  value), partial results per key split
 //  latent_merge  : sums the splits; the softmax denominator also contains exp(sink) per head
+#include "ds41_mma.cuh"
 #include "ds41_stack.cuh"
 
 namespace ds41 {
@@ -183,6 +184,221 @@ __global__ void __launch_bounds__(128) latent_attend_plain_kernel(ds41_latent_at
   }
 }
 
+// bf16 form on the warp-level tensor cores: one CTA per (row, MT x 16 heads, split) walks its keys 64 at a time through two
+// shared-memory buffers; the key tile is the value tile as well.  Four warps per 16 heads: each scores 16 of the 64 keys,
+// then accumulates a quarter of the latent columns (NP pairs of 8 columns).
+constexpr int kKeyTile = 64;
+constexpr int kProbStride = kKeyTile + 8;
+
+template <int MT, int NP>
+__global__ void __launch_bounds__(MT * 128) latent_attend_mma_kernel(ds41_latent_attend_args p) {
+  extern __shared__ __align__(16) uint8_t la_smem[];
+  const int RL = p.row_len, RS = RL + 8;
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(la_smem);              // [MT * 16][RS]
+  __nv_bfloat16* sk = sq + MT * 16 * RS;                                      // [2][64][RS]
+  __nv_bfloat16* sp = sk + 2 * kKeyTile * RS;                                 // [MT][16][72]
+  float* tops = reinterpret_cast<float*>(sp + MT * 16 * kProbStride);         // [MT][4][16] maxima, then sums
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, mt = warp >> 2, w = warp & 3;
+  const int g = lane >> 2, q2 = 2 * (lane & 3);
+  const int split = blockIdx.x, r = blockIdx.y, h0 = blockIdx.z * MT * 16;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slot = p.row_slot[r];
+  const int n_keys = slot < 0 ? 0 : p.row_pos[r] + 1;
+  const int per = ((n_keys + kKeyTile - 1) / kKeyTile + p.n_splits - 1) / p.n_splits * kKeyTile;
+  const int k0 = split * per, k1 = min(n_keys, k0 + per);
+  const long long cell0 = (1ll * r * p.n_splits + split) * p.heads;
+  if (k0 >= k1) {
+    for (int h = tid; h < MT * 16; h += MT * 128)
+      if (h0 + h < p.heads) {
+        p.part_ml[2 * (cell0 + h0 + h)] = -INFINITY;
+        p.part_ml[2 * (cell0 + h0 + h) + 1] = 0.f;
+      }
+    return;
+  }
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  auto load = [&](int key0, int buf) {
+    __nv_bfloat16* dst = sk + buf * kKeyTile * RS;
+    for (int i = warp; i < kKeyTile; i += MT * 4) {
+      const __nv_bfloat16* src = key0 + i < k1 ? cache_row(static_cast<__nv_bfloat16*>(p.pool), p.page_table, p.max_pages,
+                                                           p.page_tokens, RL, slot, key0 + i)
+                                               : nullptr;
+      for (int d = lane * 8; d < RL; d += 256) {
+        if (src != nullptr) cp_async_16(dst + i * RS + d, src + d);
+        else *reinterpret_cast<uint4*>(dst + i * RS + d) = zero;
+      }
+    }
+    cp_async_commit();
+  };
+  for (int i = warp; i < MT * 16; i += MT * 4) {
+    const int h = h0 + i;
+    const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.q_abs) + r * p.ld_q_abs + 1ll * h * p.kv_pad;
+    const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(p.q_rot) + r * p.ld_q_rot + 1ll * h * p.q_rot_stride;
+    for (int d = lane * 8; d < RL; d += 256) {
+      if (h < p.heads) cp_async_16(sq + i * RS + d, d < p.kv_pad ? qa + d : qr + (d - p.kv_pad));
+      else *reinterpret_cast<uint4*>(sq + i * RS + d) = zero;
+    }
+  }
+  load(k0, 0);
+  float acc[NP][2][4];
+#pragma unroll
+  for (int i = 0; i < NP; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float scale2 = p.scale * 1.4426950408889634f;
+  const int n_pairs = p.kv_pad / 16;
+  int buf = 0;
+  for (int t0 = k0; t0 < k1; t0 += kKeyTile, buf ^= 1) {
+    if (t0 + kKeyTile < k1) {
+      load(t0 + kKeyTile, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* kt = sk + buf * kKeyTile * RS;
+    float s[2][4] = {};
+    {
+      const __nv_bfloat16* arow = sq + (mt * 16 + (lane & 15)) * RS + (lane >> 4) * 8;
+      const __nv_bfloat16* brow = kt + (w * 16 + (lane & 7) + (lane >> 4) * 8) * RS + ((lane >> 3) & 1) * 8;
+#pragma unroll 4
+      for (int k = 0; k < RL; k += 16) {
+        uint32_t a[4], b[4];
+        ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
+        ldmatrix_x4(b[0], b[1], b[2], b[3], brow + k);
+        mma_bf16_16816(s[0], a, b[0], b[1]);
+        mma_bf16_16816(s[1], a, b[2], b[3]);
+      }
+    }
+    float top[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = t0 + w * 16 + 8 * j + q2 + (e & 1);
+        s[j][e] = key < k1 ? s[j][e] * scale2 : -INFINITY;
+        top[e >> 1] = fmaxf(top[e >> 1], s[j][e]);
+      }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      top[u] = fmaxf(top[u], __shfl_xor_sync(0xffffffffu, top[u], 1));
+      top[u] = fmaxf(top[u], __shfl_xor_sync(0xffffffffu, top[u], 2));
+      if ((lane & 3) == 0) tops[(mt * 4 + w) * 16 + g + 8 * u] = top[u];
+    }
+    __syncthreads();
+    float keep[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      float x = m[u];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x = fmaxf(x, tops[(mt * 4 + i) * 16 + g + 8 * u]);
+      keep[u] = m[u] == -INFINITY ? 0.f : ex2_approx(m[u] - x);
+      m[u] = x;
+      l[u] *= keep[u];
+    }
+    // the tile holds at least one visible key, so m is finite here
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float x = ex2_approx(s[j][2 * u] - m[u]), y = ex2_approx(s[j][2 * u + 1] - m[u]);
+        l[u] += x + y;
+        *reinterpret_cast<uint32_t*>(sp + (mt * 16 + g + 8 * u) * kProbStride + w * 16 + 8 * j + q2) = pack_bf16(x, y);
+      }
+#pragma unroll
+    for (int i = 0; i < NP; ++i)
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][j][e] *= keep[e >> 1];
+    __syncthreads();
+    const __nv_bfloat16* prow = sp + (mt * 16 + (lane & 15)) * kProbStride + (lane >> 4) * 8;
+#pragma unroll
+    for (int k = 0; k < kKeyTile; k += 16) {
+      uint32_t a[4];
+      ldmatrix_x4(a[0], a[1], a[2], a[3], prow + k);
+      const __nv_bfloat16* brow = kt + (k + (lane & 15)) * RS + (lane >> 4) * 8;
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int pair = w + 4 * i;
+        if (pair < n_pairs) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(b[0], b[1], b[2], b[3], brow + 16 * pair);
+          mma_bf16_16816(acc[i][0], a, b[0], b[1]);
+          mma_bf16_16816(acc[i][1], a, b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    l[u] += __shfl_xor_sync(0xffffffffu, l[u], 1);
+    l[u] += __shfl_xor_sync(0xffffffffu, l[u], 2);
+    if ((lane & 3) == 0) tops[(mt * 4 + w) * 16 + g + 8 * u] = l[u];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int h = h0 + mt * 16 + g + 8 * u;
+    if (h >= p.heads) continue;
+    const long long cell = cell0 + h;
+    if (w == 0 && (lane & 3) == 0) {
+      float x = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x += tops[(mt * 4 + i) * 16 + g + 8 * u];
+      p.part_ml[2 * cell] = m[u] * 0.6931471805599453f;       // natural-log units, like the plain kernel
+      p.part_ml[2 * cell + 1] = x;
+    }
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int pair = w + 4 * i;
+      if (pair < n_pairs)
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+          *reinterpret_cast<float2*>(p.part_o + cell * p.kv_pad + 16 * pair + 8 * j + q2) =
+              make_float2(acc[i][j][2 * u], acc[i][j][2 * u + 1]);
+    }
+  }
+}
+
+template <int MT, int NP>
+static int launch_attend_mma(const ds41_latent_attend_args& a, cudaStream_t st) {
+  const int smem = (MT * 16 + 2 * kKeyTile) * (a.row_len + 8) * 2 + MT * 16 * kProbStride * 2 + MT * 64 * 4;
+  static int allowed = 47 * 1024;
+  if (smem > allowed) {
+    const cudaError_t e = cudaFuncSetAttribute(latent_attend_mma_kernel<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    allowed = smem;
+  }
+  const dim3 grid(a.n_splits, a.rows, (a.heads + MT * 16 - 1) / (MT * 16));
+  return launch_pdl(latent_attend_mma_kernel<MT, NP>, grid, dim3(MT * 128), smem, st, a);
+}
+
+template <int MT>
+static int dispatch_attend_mma(const ds41_latent_attend_args& a, cudaStream_t st) {
+  if (a.kv_pad <= 64) return launch_attend_mma<MT, 1>(a, st);
+  if (a.kv_pad <= 128) return launch_attend_mma<MT, 2>(a, st);
+  if (a.kv_pad <= 256) return launch_attend_mma<MT, 4>(a, st);
+  return launch_attend_mma<MT, 8>(a, st);
+}
+
+// heads per CTA of the tensor-core form for this row length (0: it does not fit, the plain form runs)
+static int attend_mma_heads(const ds41_latent_attend_args& a) {
+  if (a.f32 || a.kv_pad > 512 || (a.kv_pad & 15) || (a.row_len & 15) || (a.ld_q_abs & 7) || (a.ld_q_rot & 7) ||
+      (a.q_rot_stride & 7) || ((reinterpret_cast<uintptr_t>(a.q_abs) | reinterpret_cast<uintptr_t>(a.q_rot) |
+                                reinterpret_cast<uintptr_t>(a.pool)) & 15))
+    return 0;
+  auto fits = [&](int mt) {
+    return (mt * 16 + 2 * kKeyTile) * (a.row_len + 8) * 2 + mt * 16 * kProbStride * 2 + mt * 256 <= 226 * 1024;
+  };
+  if (a.heads > 16 && fits(2)) return 32;
+  return fits(1) ? 16 : 0;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* part_o, const float* part_ml, const float* sink,
                                                            int n_splits, int heads, int kv_pad, T* out, int ld_out) {
@@ -276,6 +492,9 @@ extern "C" int ds41_latent_attend(const ds41_latent_attend_args* a, void* stream
       a->row_pos == nullptr || a->row_slot == nullptr || a->part_o == nullptr || a->part_ml == nullptr)
     return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int mma_heads = attend_mma_heads(*a);
+  if (mma_heads == 32) return dispatch_attend_mma<2>(*a, st);
+  if (mma_heads == 16) return dispatch_attend_mma<1>(*a, st);
   const size_t smem = (1ull * a->row_len + a->kv_pad + 32) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const dim3 grid(a->heads, a->n_splits, a->rows);

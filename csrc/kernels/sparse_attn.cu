@@ -12,6 +12,7 @@
 // decode batch sizes, each CTA touching 64 gathered 1 KiB rows.
 #include "ds41_api.h"
 #include "ds41_launch.cuh"
+#include "ds41_mma.cuh"
 #include "ds41_ptx.cuh"
 
 namespace ds41 {
@@ -498,31 +499,6 @@ __global__ void __launch_bounds__(1024) candidate_select_kernel(CandParams p) {
 }
 
 // ---------------------------------------------------------------------------------------- attention
-__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, const void* smem_row) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];"
-               : "=r"(r0), "=r"(r1)
-               : "r"(smem_u32(smem_row)));
-}
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3,
-                                            const void* smem_row) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3)
-               : "r"(smem_u32(smem_row)));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3,
-                                                  const void* smem_row) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3)
-               : "r"(smem_u32(smem_row)));
-}
-
 struct AttendParams {
   const __nv_bfloat16* q;      // [rows][ldq]; local head h at column q_off + h*D
   long long ldq;
@@ -565,13 +541,6 @@ __device__ __forceinline__ uint4 expand_fp4_chunk(const uint8_t* row8, int D, in
 
 constexpr int kKeysPerCta = 64;
 constexpr int kHeadsPerCta = 16;
-
-__device__ __forceinline__ void cp_async_16(void* smem_dst, const void* gsrc) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem_dst)), "l"(gsrc) : "memory");
-}
-__device__ __forceinline__ void cp_async_wait_all() {
-  asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
-}
 
 // grid (n_splits, rows, ceil(heads/16)), 128 threads: one CTA = 16 heads x the 64-key tiles split, split + n_splits, ...
 // of one row, folded with a running softmax; n_splits = number of tiles gives one tile per CTA (decode), a small

@@ -36,14 +36,29 @@ import sys
 import time
 
 
-def _config(args):
-    from .config import ModelConfig
+def _family(args):
+    """(model family, configuration) that the command line names: --config, else the checkpoint's own config.json where a
+    family reads it, else the preset --model."""
+    from .models import registry
     if args.config:
-        with open(args.config) as f:
-            return ModelConfig.from_official_json(json.load(f))
-    if args.model == "flash":
-        return ModelConfig.flash(args.layers or 4)
-    return ModelConfig.small() if args.model == "small" else ModelConfig.tiny()
+        return registry.config_from_file(args.config)
+    ckpt = getattr(args, "checkpoint", "")
+    if ckpt and os.path.exists(os.path.join(ckpt, "config.json")):
+        fam, cfg = registry.config_from_file(ckpt)
+        if fam.name != "ds41":           # a ds41 checkpoint keeps to --model / --config (layer counts can be cut there)
+            return fam, cfg
+    return registry.preset(args.model, args.layers)
+
+
+def _config(args):
+    return _family(args)[1]
+
+
+def _only_ds41(args, what: str):
+    fam, cfg = _family(args)
+    if fam.name != "ds41":
+        raise SystemExit(f"{what} reads the tensor catalog of ds41 models; {cfg.name} is a {fam.name} model")
+    return cfg
 
 
 def cmd_build(args) -> int:
@@ -56,7 +71,16 @@ def cmd_build(args) -> int:
 
 def cmd_info(args) -> int:
     from .loader.catalog import expected_tensors
-    cfg = _config(args)
+    fam, cfg = _family(args)
+    if fam.name != "ds41":
+        import math
+        from .models import genesun
+        shapes = genesun.tensor_shapes(cfg)
+        print(json.dumps({"model": cfg.name, "family": fam.name, "layers": cfg.n_layers, "hidden": cfg.hidden,
+                          "mixers": [l.mixer.kind for l in cfg.layers], "vocab": cfg.vocab,
+                          "checkpoint_tensors": len(shapes), "cache_rows_of_layers": cfg.cache_layers(),
+                          "parameters": sum(math.prod(x) for x in shapes.values()), "dtypes": list(fam.dtypes)}))
+        return 0
     n = len(expected_tensors(cfg)) if args.model == "flash" and not args.layers else None
     expert = 3 * cfg.hidden * cfg.inter
     print(json.dumps({"model": cfg.name, "layers": cfg.n_layers, "hidden": cfg.hidden, "experts": cfg.n_experts,
@@ -119,7 +143,19 @@ def cmd_doctor(args) -> int:
 def cmd_inspect_model(args) -> int:
     """Catalog summary (reference: `ds41rt inspect-model`, rust/crates/ds41rt-loader/src/v41_catalog.rs:478-637)."""
     from .loader.catalog import Catalog, expected_tensors, official_templates
-    cfg = _config(args)
+    fam, cfg = _family(args)
+    if fam.name != "ds41":
+        import math
+        from .loader.stack import StackCheckpoint
+        from .models import genesun
+        shapes = genesun.tensor_shapes(cfg)
+        rep = {"model": cfg.name, "family": fam.name, "tensors": len(shapes),
+               "total_gb": round(2 * sum(math.prod(x) for x in shapes.values()) / 2 ** 30, 3)}
+        if args.checkpoint:
+            rep["checkpoint"] = {"directory": args.checkpoint,
+                                 "validated_tensors": len(StackCheckpoint(args.checkpoint, shapes).where)}
+        print(json.dumps(rep, indent=1))
+        return 0
     specs = expected_tensors(cfg, variant=args.variant)
     by_dtype, by_class = {}, {}
     import math
@@ -164,7 +200,7 @@ def cmd_load_tensors(args) -> int:
     """Read tensors of a checkpoint through the strict catalog (reference: `ds41rt load-tensors`)."""
     import fnmatch
     from .loader.catalog import Catalog
-    cfg = _config(args)
+    cfg = _only_ds41(args, "load-tensors")
     t0 = time.time()
     cat = Catalog(args.checkpoint, cfg, variant=args.variant)
     t_open = time.time() - t0
@@ -236,7 +272,7 @@ def cmd_make_loadplan(args) -> int:
     """Per-rank load plan (reference: `ds41rt make-loadplan`, rust/crates/ds41rt-loader/src/v41_catalog.rs:215-273)."""
     import math
     from .loader.catalog import Catalog, expected_tensors
-    cfg = _config(args)
+    cfg = _only_ds41(args, "make-loadplan")
     sizes = {"BF16": 2, "F32": 4, "F8_E4M3": 1, "F8_E8M0": 1, "I8": 1, "U8": 1}
     if args.checkpoint:
         cat = Catalog(args.checkpoint, cfg, variant=args.variant)
@@ -439,7 +475,6 @@ def _vision_tower(args, cfg, dev):
 
 def cmd_serve(args) -> int:
     import torch
-    from .models.ds41 import DS41Engine, EngineWeights
     from .serving.engine import NativeBackend
     from .serving.http import ApiServer
     from .serving.tokenizer import ByteTokenizer, HFTokenizer
@@ -448,7 +483,15 @@ def cmd_serve(args) -> int:
         return 2
     from .parallel.fabric import Fabric
     from .serving.distributed import LeaderEngine, follower_loop, make_control_group
-    cfg = _config(args)
+    fam, cfg = _family(args)
+    if fam.name != "ds41":
+        wanted = [o for o, on in (("--vision", args.vision), ("--speculative", args.speculative),
+                                  ("--engram-table", args.engram_table), ("--engram-random-rows", args.engram_random_rows),
+                                  ("--host-cache-gb", args.host_cache_gb), ("--kv-dtype", args.kv_dtype != "bf16"),
+                                  ("more than one rank", int(os.environ.get("WORLD_SIZE", "1")) > 1)) if on]
+        if wanted:
+            print(f"{cfg.name}: {', '.join(wanted)} not available for {fam.name} models", file=sys.stderr)
+            return 2
     fabric = Fabric.create() if "WORLD_SIZE" in os.environ else Fabric.single(torch.device("cuda", args.device))
     rank, world, dev = fabric.rank, fabric.world, fabric.device
     ctl = make_control_group(fabric)
@@ -456,11 +499,9 @@ def cmd_serve(args) -> int:
     tk = HFTokenizer(args.tokenizer) if args.tokenizer else \
         ByteTokenizer(vocab_size=cfg.vocab, extra_specials=image_marks if args.vision else ())
     t0 = time.time()
-    if args.checkpoint:
-        from .loader.official import load_engine_weights
-        weights = load_engine_weights(args.checkpoint, cfg, rank, world, dev, expert_dtype=args.expert_dtype)
-    else:
-        weights = EngineWeights.random(cfg, rank, world, dev, seed=args.seed, expert_dtype=args.expert_dtype)
+    make = dict(rank=rank, world=world, expert_dtype=args.expert_dtype)
+    weights = fam.load_weights(args.checkpoint, cfg, dev, **make) if args.checkpoint else \
+        fam.random_weights(cfg, dev, seed=args.seed, **make)
     # KV pool: what the request slots want at full context, cut to what is free beside the weights
     from .runtime.memory import plan_pool
     torch.cuda.synchronize()
@@ -472,7 +513,7 @@ def cmd_serve(args) -> int:
     if n_pages < (args.max_context + 63) // 64 + 1:
         print(f"rank {rank}: only {n_pages} KV pages fit; lower --max-context or --concurrency", file=sys.stderr)
         return 2
-    eng = DS41Engine(cfg, weights, fabric, max_rows=max(8, args.concurrency, args.prefill_chunk), slots=args.concurrency,
+    eng = fam.engine(cfg, weights, fabric, max_rows=max(8, args.concurrency, args.prefill_chunk), slots=args.concurrency,
                      max_ctx=args.max_context, kv_dtype=args.kv_dtype, n_pages=n_pages)
     engram_layers = _attach_engram(args, cfg, eng, dev)
     hb = None
@@ -544,9 +585,10 @@ def main(argv=None) -> int:
     sub = ap.add_subparsers(dest="cmd", required=True)
 
     def model_args(p):
-        p.add_argument("--model", default="tiny", choices=["tiny", "small", "flash"])
-        p.add_argument("--layers", type=int, default=0, help="flash: number of layers to instantiate")
-        p.add_argument("--config", default="", help="official config.json (overrides --model)")
+        from .models.registry import PRESETS
+        p.add_argument("--model", default="tiny", choices=PRESETS)
+        p.add_argument("--layers", type=int, default=0, help="flash, genesun: number of layers to instantiate")
+        p.add_argument("--config", default="", help="config.json of any model family (overrides --model)")
 
     sub.add_parser("build")
     pi = sub.add_parser("info")
@@ -599,7 +641,8 @@ def main(argv=None) -> int:
                     help="pinned host memory for snapshots that leave the device banks (0 = off; one-rank serving)")
     ps.add_argument("--reserve-gb", type=int, default=0, help="device memory to leave untouched by the KV pool")
     ps.add_argument("--peer-timeout", type=float, default=10.0, help="seconds without a heartbeat before a rank counts as gone")
-    ps.add_argument("--checkpoint", default="", help="directory with model.safetensors.index.json (official layout)")
+    ps.add_argument("--checkpoint", default="", help="directory with the model's safetensors files (ds41: official layout with an index; genesun: config.json "
+                         "beside model.safetensors)")
     ps.add_argument("--tokenizer", default="", help="tokenizer.json; default: byte-level tokenizer")
     ps.add_argument("--expert-dtype", default="mxfp8", choices=["mxfp8", "mxfp4", "nvfp4", "bf16"])
     ps.add_argument("--host", default="127.0.0.1")

@@ -153,12 +153,18 @@ class LatentAttention:
         freq = rope_inv_freq(spec.rope, spec.rot_dim) if spec.rope is not None else [0.0] * (spec.rot_dim // 2)
         self.freq = torch.tensor(freq or [0.0], dtype=F32, device=device)
 
+        # the expanded form keeps two query tiles, a key tile and a value tile of 128 rows in shared memory
+        chunks = -(-self.dp // 64) + -(-self.rp // 64)
+        self.expandable = dtype == BF16 and self.vp <= 128 and 3 * chunks + -(-self.vp // 64) <= 14
+
     def matrices(self):
         return {"a": [(self.w_in.n, self.w_in.k)], "b": [(self.w_uq.n, self.w_uq.k), (self.w_o.n, self.w_o.k)]}
 
     def run(self, e: "StackEngine", l: int, R: int, src: int) -> Tuple[Proj, Optional[Proj]]:
         sp, k, H = self.spec, e.k, self.spec.heads
-        pin = e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
+        long = e.long_keys if self.expandable else 0
+        pin = e.project_wide("gemm_mix_in", R, self.w_in) if long else \
+            e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
         pool = e.cache.pools[src]
         a = S.LatentPostArgs()
         a.dq, a.dq_norm = pin.at(self.at["dq"]).args(), self.dq_norm.data_ptr()
@@ -171,12 +177,36 @@ class LatentAttention:
         a.row_len, a.max_pages, a.page_tokens, a.f32 = self.row_len, e.cache.max_pages, e.cache.page_tokens, e.f32
         e._run("latent_post", k.ds41_latent_post, C.byref(a), lib.stream())
         ldq = H * self.hs
-        q = e.project("gemm_uq", e.cq, e.cq.shape[1], R, self.w_uq, e.planes_b)
+        if long:
+            q = Proj(e.q, ldq)
+            e._run("gemm_uq", S.project_bf16, e.cq, e.cq.shape[1], R, self.w_uq, e.q, ldq, e.status)
+        else:
+            q = e.project("gemm_uq", e.cq, e.cq.shape[1], R, self.w_uq, e.planes_b)
         e._run("latent_query", k.ds41_latent_query, C.byref(q.args()), lib.ptr(e.row_pos), lib.ptr(self.freq),
                C.c_float(sp.magnitude), R, H, self.dp, self.rp, sp.rot_dim, lib.ptr(e.q), ldq, e.f32, lib.stream())
-        self._absorbed(e, R, ldq, pool, pin.at(self.at["g"]))
+        if long:
+            self._expanded(e, R, ldq, pool, src, pin.at(self.at["g"]))
+        else:
+            self._absorbed(e, R, ldq, pool, pin.at(self.at["g"]))
         y = e.project("gemm_o", e.act, H * self.vp, R, self.w_o, e.planes_b)
         return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
+
+    def _expanded(self, e: "StackEngine", R: int, ldq: int, pool, src: int, gate: Proj):
+        sp, k, H, n = self.spec, e.k, self.spec.heads, e.long_keys
+        lat, rot, kv = e.key_space(n, self.kvp, self.rp, self.w_ukv.n)
+        if e.gathered != (src, n):           # a layer that reads the same rows finds them in place
+            e._run("latent_gather", k.ds41_latent_gather, lib.ptr(pool), lib.ptr(e.cache.page_table), e.cache.max_pages,
+                   e.cache.page_tokens, self.row_len, self.kvp, 0, lib.ptr(e.row_slot), n, lib.ptr(lat), lib.ptr(rot), 0,
+                   lib.stream())
+            e.gathered = (src, n)
+        ldkv = self.w_ukv.n
+        e._run("expand_kv", S.project_bf16, lat, self.kvp, n, self.w_ukv, kv, ldkv, e.status)
+        a = S.LatentPrefillArgs()
+        a.q, a.kv, a.rot, a.sink, a.out = (x.data_ptr() for x in (e.q, kv, rot, self.sink, e.act))
+        a.status, a.gate, a.ld_q, a.ld_kv, a.scale = e.status.data_ptr(), gate.args(), ldq, ldkv, sp.scale
+        a.rows, a.heads, a.dim_pad, a.rot_pad, a.vdim_pad = R, H, self.dp, self.rp, self.vp
+        a.n_keys, a.pos0, a.ld_out = n, n - R, H * self.vp
+        e._run("latent_prefill", k.ds41_latent_prefill, C.byref(a), lib.stream())
 
     def _absorbed(self, e: "StackEngine", R: int, ldq: int, pool, gate: Proj):
         sp, k, H = self.spec, e.k, self.spec.heads
@@ -213,11 +243,14 @@ class MLSTM:
         H = spec.heads
         self.dp, self.vp = ceil_to(spec.dim, 16), ceil_to(spec.vdim, 16)
         parts = [("q", S.pad_heads(t["q"], H, spec.dim, self.dp)), ("k", S.pad_heads(t["k"], H, spec.dim, self.dp)),
-                 ("v", S.pad_heads(t["v"], H, spec.vdim, self.vp)), ("g", S.pad_heads(t["g"], H, spec.vdim, self.vp)),
-                 ("i", t["i"]), ("f", t["f"])]
+                 ("v", S.pad_heads(t["v"], H, spec.vdim, self.vp)), ("g", S.pad_heads(t["g"], H, spec.vdim, self.vp))]
         if gate:
             parts += [("gate", gate["w"])]
-        self.w_in, self.at = S.stack_rows(parts, device, dtype)
+        self.w_in, self.at = S.stack_rows(parts + [("i", t["i"]), ("f", t["f"])], device, dtype)
+        # long passes take the log gates in fp32 from a product of their own and everything else in bf16
+        self.w_main = self.w_in.rows(0, self.at["i"])
+        self.w_gates = self.w_in.rows(self.at["i"], self.w_in.n)
+        self.chunked = dtype == BF16 and self.dp <= 512
         f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
         self.bias_i, self.bias_f = f32(t["i.b"]), f32(t["f.b"])
         self.norm = f32(S.pad_heads(t["norm"], H, spec.vdim, self.vp))
@@ -228,18 +261,28 @@ class MLSTM:
 
     def run(self, e: "StackEngine", l: int, R: int, src: Optional[int]) -> Tuple[Proj, Optional[Proj]]:
         sp, k, H = self.spec, e.k, self.spec.heads
-        pin = e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
+        long = e.long_keys > 0 and self.chunked
+        if long:
+            pin = e.project_wide("gemm_mix_in", R, self.w_main)
+            log_gates: List[Proj] = []
+            e._run("gemm_gates", lambda: log_gates.append(S.project_few(e.h, e.ldh, R, self.w_gates, e.planes_a, e.status)))
+            gates = (log_gates[0] if log_gates else Proj(e.planes_a, self.w_gates.out_ld)).at(-self.at["i"])
+        else:
+            pin = gates = e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
         ld = H * self.vp
         s, n, m = e.cache.states[l]
         a = S.MlstmArgs()
         a.q, a.k, a.v = (pin.at(self.at[x]).args() for x in "qkv")
-        a.gate_i, a.gate_f = pin.at(self.at["i"]).args(), pin.at(self.at["f"]).args()
+        a.gate_i, a.gate_f = gates.at(self.at["i"]).args(), gates.at(self.at["f"]).args()
         a.bias_i, a.bias_f = self.bias_i.data_ptr(), self.bias_f.data_ptr()
         a.row_pos, a.row_slot = e.row_pos.data_ptr(), e.row_slot.data_ptr()
         a.state_s, a.state_n, a.state_m, a.out = s.data_ptr(), n.data_ptr(), m.data_ptr(), e.o_heads.data_ptr()
         a.gate_cap, a.q_scale, a.den_eps = sp.gate_cap, sp.dim ** -0.5, sp.den_eps
         a.rows, a.heads, a.dim_pad, a.vdim_pad, a.slots, a.ld_out = R, H, self.dp, self.vp, e.cache.slots, ld
-        e._run("mlstm_step", k.ds41_mlstm_step, C.byref(a), lib.stream())
+        if long:
+            e._run("mlstm_chunk", k.ds41_mlstm_chunk, C.byref(a), lib.stream())
+        else:
+            e._run("mlstm_step", k.ds41_mlstm_step, C.byref(a), lib.stream())
         e._run("head_norm_gate", k.ds41_head_norm_gate, lib.ptr(e.o_heads), ld, C.byref(pin.at(self.at["g"]).args()),
                lib.ptr(self.norm), R, H, sp.vdim, self.vp, C.c_float(self.cfg.norm_eps), lib.ptr(e.act), ld, e.f32,
                lib.stream())
@@ -264,7 +307,8 @@ class DenseMLP:
         return {"a": [(self.w_up.n, self.w_up.k)], "b": [(self.w_down.n, self.w_down.k)]}
 
     def run(self, e: "StackEngine", R: int) -> Tuple[Proj, Optional[Proj]]:
-        pin = e.project("gemm_up", e.h, e.ldh, R, self.w_up, e.planes_a)
+        pin = e.project_wide("gemm_up", R, self.w_up) if e.long_keys else \
+            e.project("gemm_up", e.h, e.ldh, R, self.w_up, e.planes_a)
         e._run("polynorm", e.k.ds41_polynorm, C.byref(pin.at(self.at["up"]).args()), lib.ptr(self.coef), R, self.spec.ff,
                C.c_float(self.cfg.norm_eps), lib.ptr(e.act), self.ffp, e.f32, lib.stream())
         y = e.project("gemm_down", e.act, self.ffp, R, self.w_down, e.planes_b)
@@ -379,6 +423,14 @@ class StackEngine(RowsEngine):
                 for n in range(1, self.attn_rows + 1):
                     cells = max(cells, n * self.attn_splits(n, mx.spec.heads) * mx.spec.heads * mx.kvp)
         self.planes_a, self.planes_b = z((need["a"],), F32), z((need["b"],), F32)
+        # long passes: one request's rows with everything but the log gates and sublayer results in bf16
+        self.long_rows = 64
+        self.long_keys = 0            # > 0 during a long pass: positions its last row sees
+        self.gathered = None
+        wide = max(S.ceil_to(n, 8) for lw in weights.layers for m in (lw.mixer, lw.mlp) if m is not None
+                   for n, _ in m.matrices()["a"])
+        self.wide = z((R * wide if R >= self.long_rows and not self.f32 else 8,), BF16)
+        self._keys = [z((8,), BF16) for _ in range(3)]
         self.act = z((R * max(act, heads),), dt)
         self.o_heads = z((R * heads,), F32)
         if lat:
@@ -393,7 +445,7 @@ class StackEngine(RowsEngine):
         self.picked, self.pick_idx = z((self.head_cap, self.ldh), dt), z((self.head_cap,), I32)
         self.best_val, self.chosen = z((R,), F32), z((R,), I32)
         self.head_mask = None
-        self.image_patch = None
+        self._hint = None
         self.status = lib.new_status(dev)
         self._init_instruments()
         self.on_layer = None      # callable (layer, streams [rows, width]) after every layer of an eager pass
@@ -409,6 +461,19 @@ class StackEngine(RowsEngine):
         out: List[Proj] = []
         self._run(tag, lambda: out.append(S.project(x, ldx, rows, m, buf, self.status)))
         return out[0] if out else S.Proj(buf, m.out_ld)
+
+    def project_wide(self, tag: str, rows: int, m: Matrix) -> Proj:
+        """bf16 result of a projection of self.h in a long pass."""
+        self._run(tag, S.project_bf16, self.h, self.ldh, rows, m, self.wide, m.out_ld, self.status)
+        return Proj(self.wide, m.out_ld)
+
+    def key_space(self, n: int, kv_pad: int, rot_pad: int, width: int):
+        """Buffers for one request's gathered latent rows, rotated key parts and expanded keys / values (they grow)."""
+        for i, w in enumerate((kv_pad, rot_pad, width)):
+            if self._keys[i].numel() < n * w:
+                self.gathered = None
+                self._keys[i] = torch.zeros(ceil_to(n, 1024) * w, dtype=BF16, device=self.device)
+        return self._keys
 
     def _enter_rehearsal(self):
         self.row_slot.fill_(-1)       # no row owns a slot: caches and states keep what they hold
@@ -427,6 +492,9 @@ class StackEngine(RowsEngine):
             else:
                 assert slots[i] not in seen, "rows of a request must be adjacent"
                 seen.add(slots[i])
+        # what the host knows about the pass it just described: a long pass of one request
+        one = n >= self.long_rows and len(seen) == 1 and min(slots) >= 0 and not self.f32
+        self._hint = (n, positions[-1] + 1) if one else None
         pad = self.max_rows - n
         if tokens is not None:
             assert len(tokens) == n
@@ -454,6 +522,8 @@ class StackEngine(RowsEngine):
     def forward_rows(self, rows: int, *, head: bool = True, head_row: Optional[int] = None, sources: bool = True):
         """One pass over the `rows` rows described by set_rows()."""
         cfg, R, layers = self.cfg, rows, self.w.layers
+        self.long_keys = self._hint[1] if self._hint is not None and self._hint[0] == R else 0
+        self._hint = self.gathered = None
         if self.layer_timer is not None:
             self.layer_timer.begin()
         cur = self.kept[0]

@@ -130,6 +130,7 @@ def dir_functions():
         "ds41_attend_tc", "ds41_attend_merge", "ds41_engram_dequant_nvfp4", "ds41_wire_encode", "ds41_wire_decode",
         "ds41_resid_step", "ds41_polynorm", "ds41_gate_mul", "ds41_head_norm_gate", "ds41_gather_rows",
         "ds41_latent_post", "ds41_latent_query", "ds41_latent_gather", "ds41_latent_attend", "ds41_latent_merge",
+        "ds41_latent_prefill", "ds41_mlstm_chunk",
         "ds41_mlstm_step", "ds41_gemm_f32",
     ]
 

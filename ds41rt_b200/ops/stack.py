@@ -50,6 +50,13 @@ class LatentAttendArgs(C.Structure):
                 ("n_splits", C.c_int), ("max_pages", C.c_int), ("page_tokens", C.c_int), ("f32", C.c_int)]
 
 
+class LatentPrefillArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("kv", C.c_void_p), ("rot", C.c_void_p), ("sink", C.c_void_p), ("out", C.c_void_p),
+                ("status", C.c_void_p), ("gate", ProjArgs), ("ld_q", C.c_longlong), ("ld_kv", C.c_longlong),
+                ("scale", C.c_float), ("rows", C.c_int), ("heads", C.c_int), ("dim_pad", C.c_int), ("rot_pad", C.c_int),
+                ("vdim_pad", C.c_int), ("n_keys", C.c_int), ("pos0", C.c_int), ("ld_out", C.c_int)]
+
+
 class MlstmArgs(C.Structure):
     _fields_ = [("q", ProjArgs), ("k", ProjArgs), ("v", ProjArgs), ("gate_i", ProjArgs), ("gate_f", ProjArgs),
                 ("bias_i", C.c_void_p), ("bias_f", C.c_void_p), ("row_pos", C.c_void_p), ("row_slot", C.c_void_p),
@@ -88,6 +95,12 @@ class Matrix:
         self.ld = ceil_to(self.k, 8)
         self.w = torch.zeros(self.n, self.ld, dtype=dtype, device=device)
         self.w[:, :self.k] = w.to(device=device, dtype=dtype)
+
+    def rows(self, lo: int, hi: int) -> "Matrix":
+        """Some of the rows, sharing the storage."""
+        m = object.__new__(Matrix)
+        m.n, m.k, m.ld, m.w = hi - lo, self.k, self.ld, self.w[lo:hi]
+        return m
 
     @property
     def out_ld(self) -> int:
@@ -145,12 +158,21 @@ def project(x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor, 
     return Proj(buf, ldo)
 
 
-def project_bf16(x: torch.Tensor, ldx: int, rows: int, m: Matrix, out: torch.Tensor, ldo: int, status) -> Proj:
+def project_bf16(x: torch.Tensor, ldx: int, rows: int, m: Matrix, out: torch.Tensor, ldo: int, status) -> None:
     """The same with a bf16 result (long passes: half the bytes for the consumer)."""
-    assert rows > SWAP_ROWS and x.dtype == BF16
     G.gemm_raw(x, m.w, out, rows, m.n, m.k, lda=ldx, ldb=m.ld, ldo=ldo,
                out_mode=6 if m.n >= 64 and ldo % 8 == 0 else 0, bn=_wide_bn(m.n), status=status, static_operand=2)
-    return Proj(out, ldo)
+
+
+def project_few(x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor, status) -> Proj:
+    """fp32 result of a matrix with few rows, for any number of activation rows (weights as the 128-row operand)."""
+    n_tiles = -(-rows // 128)
+    s = G.pick_splits(m.n, m.k, max_splits=16, n_tiles=n_tiles)
+    while s > 1 and s * rows * m.out_ld > buf.numel():
+        s -= 1
+    G.gemm_raw(m.w, x, buf if s == 1 else None, m.n, rows, m.k, lda=m.ld, ldb=ldx, ldo=m.out_ld, out_mode=3, k_splits=s,
+               split_workspace=buf if s > 1 else None, bn=G.pick_bn(rows), status=status, static_operand=1)
+    return Proj(buf, m.out_ld, s, rows * m.out_ld)
 
 
 def _wide_bn(n: int) -> int:

@@ -13,6 +13,7 @@ from dataclasses import dataclass, asdict
 from typing import Optional
 
 from ..config import ModelConfig
+from ..stack_config import StackConfig
 from . import core as K
 
 HEADROOM_BYTES = 2 << 30
@@ -45,16 +46,34 @@ def kv_row_bytes(cfg: ModelConfig, kv_dtype: str) -> tuple:
     return fp8, (D // 2 + D // 16 + 15) // 16 * 16
 
 
+def stack_page_bytes(cfg: StackConfig, page_tokens: int, elem: int = 2) -> int:
+    from ..models.stack import latent_row_len
+    return sum(page_tokens * latent_row_len(cfg.layers[l].mixer)[1] * elem for l in cfg.cache_layers())
+
+
+def stack_state_bytes(cfg: StackConfig) -> int:
+    """fp32 recurrent state of one request."""
+    import math
+    from ..models.stack import mlstm_state_shapes
+    return sum(4 * math.prod(s) for l in cfg.state_layers() for s in mlstm_state_shapes(cfg.layers[l].mixer))
+
+
 def plan_pool(cfg: ModelConfig, *, n_layers: int, slots: int, max_context: int, free_bytes: int, kv_dtype: str = "bf16",
               page_tokens: int = 64, retained: int = 40, ring_rows: Optional[int] = None,
               reserve_bytes: int = 0) -> PoolPlan:
-    win_row, comp_row = kv_row_bytes(cfg, kv_dtype)
-    per_page = 0
-    for src, ratio in cfg.source_layers.items():
-        if src < n_layers:
-            per_page += (page_tokens // ratio) * (comp_row + 2 * cfg.index_dim)
-    ring = ring_rows if ring_rows is not None else cfg.window + 16
-    ring_bytes = n_layers * slots * ring * win_row
+    if isinstance(cfg, StackConfig):
+        # latent rows of the layers that produce them; recurrent states (one per slot, and per retained snapshot) stand
+        # where the other models have their window rings
+        per_page, state = stack_page_bytes(cfg, page_tokens), stack_state_bytes(cfg)
+        ring_bytes = state * (slots + retained)
+    else:
+        win_row, comp_row = kv_row_bytes(cfg, kv_dtype)
+        per_page = 0
+        for src, ratio in cfg.source_layers.items():
+            if src < n_layers:
+                per_page += (page_tokens // ratio) * (comp_row + 2 * cfg.index_dim)
+        ring = ring_rows if ring_rows is not None else cfg.window + 16
+        ring_bytes = n_layers * slots * ring * win_row
     budget = max(0, free_bytes - ring_bytes - reserve_bytes - HEADROOM_BYTES)
     wanted = (max_context + page_tokens - 1) // page_tokens * (slots + 2) + slots + 2 * retained
     pages = wanted if per_page == 0 else K.plan_kv_groups(max_context, page_tokens, slots, retained, per_page, budget)
