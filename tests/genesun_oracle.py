@@ -10,6 +10,18 @@ import math
 import torch
 
 
+_noise = None      # a torch.Generator while `rounding_spread` measures how far bf16 rounding carries
+
+
+def _shake(x):
+    """What storing x in bf16 may do to it: a random relative change of up to one part in 2^8."""
+    return x if _noise is None else x * (1 + (torch.rand(x.shape, generator=_noise, dtype=x.dtype) - 0.5) * 2 ** -7)
+
+
+def linear(x, w):
+    return _shake(_shake(x) @ w.T)
+
+
 def rms_unit(x, eps):
     return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
 
@@ -70,20 +82,20 @@ def latent_attention(h, pos, w, p, mx, eps, shared):
     """`shared`: (latent, rotated key) of the layer named by kv_from, or None.  -> (output, (latent, rotated key))."""
     H, D, R, V = mx["heads"], mx["dim"], mx["rot_dim"], mx["vdim"]
     T = h.shape[0]
-    cq = rms_unit(h @ w[p + "dq"].T, eps) * w[p + "dq.norm"]
-    q = (cq @ w[p + "uq"].T).view(T, H, D + R)
+    cq = rms_unit(linear(h, w[p + "dq"]), eps) * w[p + "dq.norm"]
+    q = linear(cq, w[p + "uq"]).view(T, H, D + R)
     if shared is None:
-        kv = h @ w[p + "dkv"].T
+        kv = linear(h, w[p + "dkv"])
         lat = rms_unit(kv[:, :mx["kv_rank"]], eps) * w[p + "dkv.norm"]
         kr = rotate_pairs(kv[:, mx["kv_rank"]:], pos, mx["rot"])
         shared = (lat, kr)
     lat, kr = shared
     qr = rotate_pairs(q[..., D:], pos, mx["rot"])
-    k = torch.cat([(lat @ w[p + "uk"].T).view(T, H, D), kr[:, None, :].expand(T, H, R)], -1)
-    v = (lat @ w[p + "uv"].T).view(T, H, V)
+    k = torch.cat([linear(lat, w[p + "uk"]).view(T, H, D), kr[:, None, :].expand(T, H, R)], -1)
+    v = linear(lat, w[p + "uv"]).view(T, H, V)
     o = sink_softmax_attention(torch.cat([q[..., :D], qr], -1), k, v, mx["scale"], w[p + "sink"])
-    o = o.reshape(T, H * V) * torch.sigmoid(h @ w[p + "g"].T)
-    return o @ w[p + "o"].T, shared
+    o = o.reshape(T, H * V) * torch.sigmoid(linear(h, w[p + "g"]))
+    return linear(o, w[p + "o"]), shared
 
 
 def mlstm_scan(q, k, v, i, f):
@@ -107,22 +119,22 @@ def mlstm_scan(q, k, v, i, f):
 def mlstm(h, w, p, mx, eps):
     H, D, V, cap = mx["heads"], mx["dim"], mx["vdim"], mx["gate_cap"]
     T = h.shape[0]
-    q = (h @ w[p + "q"].T).view(T, H, D) * D ** -0.5
-    k = (h @ w[p + "k"].T).view(T, H, D)
-    v = (h @ w[p + "v"].T).view(T, H, V)
-    i = cap * torch.tanh((h @ w[p + "i"].T + w[p + "i.b"]) / cap)
-    f = torch.nn.functional.logsigmoid(cap * torch.tanh((h @ w[p + "f"].T + w[p + "f.b"]) / cap))
+    q = linear(h, w[p + "q"]).view(T, H, D) * D ** -0.5
+    k = linear(h, w[p + "k"]).view(T, H, D)
+    v = linear(h, w[p + "v"]).view(T, H, V)
+    i = cap * torch.tanh((linear(h, w[p + "i"]) + w[p + "i.b"]) / cap)
+    f = torch.nn.functional.logsigmoid(cap * torch.tanh((linear(h, w[p + "f"]) + w[p + "f.b"]) / cap))
     o = rms_unit(mlstm_scan(q, k, v, i, f), eps).reshape(T, H * V) * w[p + "norm"]
-    return (o * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+    return linear(o * torch.sigmoid(linear(h, w[p + "g"])), w[p + "o"])
 
 
 def dense_polynorm_mlp(h, w, p, eps):
-    return polynorm(h @ w[p + "up"].T, w[p + "act"], eps) @ w[p + "down"].T
+    return linear(polynorm(linear(h, w[p + "up"]), w[p + "act"], eps), w[p + "down"])
 
 
 def gated_normed(y, h, gate_w, gate_b, norm_w, eps):
     """Sublayer result y of input h: sigmoid gate from h, then the norm that follows the sublayer."""
-    return layer_norm(y * torch.sigmoid(h @ gate_w.T + gate_b), norm_w, eps)
+    return layer_norm(y * torch.sigmoid(linear(h, gate_w) + gate_b), norm_w, eps)
 
 
 class GenesunOracle:
@@ -154,4 +166,100 @@ class GenesunOracle:
             kept.append(x)
             x = sum(c * t for c, t in zip(w[p + "dwa"], kept))
             after.append(x)
-        return layer_norm(x, w["final.norm"], eps) @ w["head"].T, after
+        return linear(layer_norm(x, w["final.norm"], eps), w["head"]), after
+
+
+def position_error(got, want):
+    """Root mean square difference per position, relative to the spread of all values."""
+    return (got.double() - want.double()).pow(2).mean(-1).sqrt() / want.double().std()
+
+
+def rounding_spread(oracle, tokens, trials=4):
+    """How far bf16-sized rounding of every stored activation moves each position, -> (logits, [per layer])."""
+    global _noise
+    want, layers = oracle.forward(tokens)
+    worst = [torch.zeros(len(tokens), dtype=torch.float64) for _ in range(1 + len(layers))]
+    try:
+        for t in range(trials):
+            _noise = torch.Generator().manual_seed(t)
+            got, after = oracle.forward(tokens)
+            for i, (a, b) in enumerate(zip([got, *after], [want, *layers])):
+                worst[i] = torch.maximum(worst[i], position_error(a, b))
+    finally:
+        _noise = None
+    return worst[0], worst[1:]
+
+
+# ---------------------------------------------------------------------------------------------------- test models
+def attention_mixer(heads, dim, rot_dim, vdim, q_rank, kv_rank, scale=None, base=10000.0, scaling=None, kv_from=None):
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank,
+             scale=(dim + rot_dim) ** -0.5 if scale is None else scale, rot=dict(base=base, dims=rot_dim))
+    if scaling is not None:
+        m["rot"]["scaling"] = scaling
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return m
+
+
+def make_doc(width, vocab, layers, eps=1e-6):
+    """`layers`: (type, mixer, ff or None)."""
+    return {"architecture": "Genesun", "width": width, "vocab": vocab, "norm": {"eps": eps},
+            "layers": [{"type": t, "mixer": m, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+                       for t, m, ff in layers]}
+
+
+def make_weights(doc, seed=0):
+    """Random weights whose every mechanism shows in the logits, rounded to bf16 (returned as fp32)."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = doc["width"], doc["vocab"]
+    n = lambda *s, std=1.0: torch.randn(*s, generator=g) * std
+    lin = lambda o, i: n(o, i, std=i ** -0.5)
+    one = lambda k: 1.0 + n(k, std=0.2)
+    w = {"embed": n(V, W), "final.norm": one(W), "head": lin(V, W)}
+    for l, d in enumerate(doc["layers"]):
+        p, m = f"l{l}.", d["mixer"]
+        w.update({p + "norm1": one(W), p + "norm1b": one(W), p + "rg1": lin(W, W), p + "rg1.b": n(W, std=0.5),
+                  p + "dwa": n(l + 2, std=0.3)})
+        w[p + "dwa"][-1] += 0.7
+        if d["type"] == "mlstm":
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            w.update({p + "mix.q": 2 * lin(hd, W), p + "mix.k": lin(hd, W), p + "mix.v": lin(hv, W), p + "mix.g": lin(hv, W),
+                      p + "mix.o": lin(W, hv), p + "mix.norm": one(hv), p + "mix.i": 2 * lin(m["heads"], W),
+                      p + "mix.i.b": n(m["heads"]), p + "mix.f": lin(m["heads"], W), p + "mix.f.b": 3 + 2 * n(m["heads"])})
+        else:
+            hv = m["heads"] * m["vdim"]
+            w.update({p + "mix.dq": lin(m["q_rank"], W), p + "mix.dq.norm": 2 * one(m["q_rank"]),
+                      p + "mix.uq": 2 * lin(m["heads"] * (m["dim"] + m["rot_dim"]), m["q_rank"]),
+                      p + "mix.uk": lin(m["heads"] * m["dim"], m["kv_rank"]), p + "mix.uv": lin(hv, m["kv_rank"]),
+                      p + "mix.sink": n(m["heads"]) + 1.0, p + "mix.g": lin(hv, W), p + "mix.o": lin(W, hv)})
+            if "kv_from" not in m:
+                w.update({p + "mix.dkv": lin(m["kv_rank"] + m["rot_dim"], W), p + "mix.dkv.norm": one(m["kv_rank"])})
+        if d["mlp"] is not None:
+            ff = d["mlp"]["ff"]
+            w.update({p + "norm2": one(W), p + "norm2b": one(W), p + "rg2": lin(W, W), p + "rg2.b": n(W, std=0.5),
+                      p + "mlp.up": lin(ff, W), p + "mlp.down": lin(W, ff),
+                      p + "mlp.act": torch.tensor([0.6, 0.4, 0.3, 0.1]) + n(4, std=0.1)})
+    return {k: v.to(torch.bfloat16).float() for k, v in w.items()}
+
+
+YARN = dict(factor=5.0, original=96, fast=8.0, slow=1.0)
+
+MODELS = {
+    # widths that are no multiple of the tile sizes, shared cache rows over several layers, feed-forward after a recurrence
+    "odd": make_doc(88, 131, [
+        ("latent_attention", attention_mixer(3, 20, 6, 24, 56, 40, scaling=YARN), 100),
+        ("mlstm", dict(heads=3, dim=24, vdim=40, gate_cap=7.0), 60),
+        ("latent_attention", attention_mixer(5, 12, 6, 36, 40, 40, scale=0.3, base=500.0, kv_from=0), None),
+        ("latent_attention", attention_mixer(2, 20, 6, 24, 24, 40, scaling=YARN, kv_from=0), 36)]),
+    # head counts and ranks of one tile or less, no scaling, recurrences first and last
+    "plain": make_doc(64, 96, [
+        ("mlstm", dict(heads=1, dim=16, vdim=16, gate_cap=5.0), None),
+        ("latent_attention", attention_mixer(1, 32, 2, 16, 16, 16, scale=0.5), None),
+        ("mlstm", dict(heads=2, dim=64, vdim=32, gate_cap=20.0), None)]),
+    # sizes that fill whole tensor-core tiles, more heads than one tile holds
+    "tiles": make_doc(256, 320, [
+        ("latent_attention", attention_mixer(20, 64, 64, 128, 64, 192, base=2000.0, scaling=dict(YARN, original=512)), 512),
+        ("mlstm", dict(heads=2, dim=128, vdim=192, gate_cap=11.0), None),
+        ("latent_attention", attention_mixer(18, 80, 64, 48, 96, 192, base=2000.0, scaling=dict(YARN, original=512),
+                                             kv_from=0), 256)]),
+}
