@@ -544,12 +544,14 @@ typedef struct ds41_mlstm_args {
   float* state_n;                 // [slots][heads][ceil(vdim_pad / 32)][dim_pad]
   float* state_m;                 // [slots][heads][ceil(vdim_pad / 32)]
   float* out;                     // [rows][ld_out]
+  float* work;                    // mlstm_chunk: ds41_mlstm_chunk_work() bytes, 16-byte aligned
   float gate_cap, q_scale, den_eps;
   int rows, heads, dim_pad, vdim_pad, slots, ld_out;
 } ds41_mlstm_args;
 int ds41_mlstm_step(const ds41_mlstm_args* args, void* stream);
 // Long pass of one request (row 0's slot; adjacent rows), dim_pad <= 512; q, k, v are bf16 with 16-byte aligned rows.
 int ds41_mlstm_chunk(const ds41_mlstm_args* args, void* stream);
+long long ds41_mlstm_chunk_work(int rows, int heads);
 
 int ds41_gemm_f32(const float* A, const float* B, float* out, int M, int N, int K, long long lda, long long ldb,
                   long long ldo, int batch, long long a_batch_stride, long long b_batch_stride,

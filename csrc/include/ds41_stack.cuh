@@ -17,6 +17,44 @@ __device__ __forceinline__ float proj_at(const ds41_proj& a, long long row, int 
   return s;
 }
 
+// Four neighbouring elements at a column that is a multiple of 4 (rows and planes 16-byte aligned).
+__device__ __forceinline__ float4 proj_at4(const ds41_proj& a, long long row, int col) {
+  const long long i = row * a.ld + a.col + col;
+  if (a.bf16) {
+    const uint2 v = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(a.data) + i);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+  }
+  const float* p = static_cast<const float*>(a.data) + i;
+  float4 s = *reinterpret_cast<const float4*>(p);
+#pragma unroll 4
+  for (int k = 1; k < a.splits; ++k) {
+    const float4 t = *reinterpret_cast<const float4*>(p + k * a.plane);
+    s.x += t.x;
+    s.y += t.y;
+    s.z += t.z;
+    s.w += t.w;
+  }
+  return s;
+}
+inline bool proj_ok(const ds41_proj& p) {
+  return p.data != nullptr && p.ld > 0 && p.splits >= 1 && p.col >= 0 && (p.splits == 1 || (p.plane > 0 && !p.bf16));
+}
+inline bool proj_vec4(const ds41_proj& p) {
+  return !(p.ld & 3) && !(p.col & 3) && !(p.plane & 3) && !(reinterpret_cast<uintptr_t>(p.data) & 15);
+}
+
+// Four values of a vector of which `valid` exist (the rest read as zero).
+__device__ __forceinline__ float4 load4(const float* p, int valid) {
+  if (valid >= 4) return *reinterpret_cast<const float4*>(p);
+  return make_float4(valid > 0 ? p[0] : 0.f, valid > 1 ? p[1] : 0.f, valid > 2 ? p[2] : 0.f, 0.f);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
 template <typename T>
 __device__ __forceinline__ T from_f32(float v);
 template <>

@@ -217,19 +217,27 @@ __global__ void __launch_bounds__(MT * 128) latent_attend_mma_kernel(ds41_latent
     return;
   }
   const uint4 zero = make_uint4(0, 0, 0, 0);
-  auto load = [&](int key0, int buf) {
-    __nv_bfloat16* dst = sk + buf * kKeyTile * RS;
-    for (int i = warp; i < kKeyTile; i += MT * 4) {
-      const __nv_bfloat16* src = key0 + i < k1 ? cache_row(static_cast<__nv_bfloat16*>(p.pool), p.page_table, p.max_pages,
-                                                           p.page_tokens, RL, slot, key0 + i)
-                                               : nullptr;
+  // lane i knows where the warp's i-th key of a tile lies; looked up one tile ahead of the copies
+  constexpr int kMine = kKeyTile / (MT * 4);
+  auto locate = [&](int key0) {
+    const int key = key0 + warp + (lane % kMine) * MT * 4;
+    return key < k1 ? cache_row(static_cast<__nv_bfloat16*>(p.pool), p.page_table, p.max_pages, p.page_tokens, RL, slot, key)
+                    : nullptr;
+  };
+  auto load = [&](__nv_bfloat16* where, int buf) {
+    __nv_bfloat16* dst = sk + buf * kKeyTile * RS + warp * RS;
+#pragma unroll 4
+    for (int i = 0; i < kMine; ++i) {
+      const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(
+          __shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(where), i));
       for (int d = lane * 8; d < RL; d += 256) {
-        if (src != nullptr) cp_async_16(dst + i * RS + d, src + d);
-        else *reinterpret_cast<uint4*>(dst + i * RS + d) = zero;
+        if (src != nullptr) cp_async_16(dst + i * MT * 4 * RS + d, src + d);
+        else *reinterpret_cast<uint4*>(dst + i * MT * 4 * RS + d) = zero;
       }
     }
     cp_async_commit();
   };
+  __nv_bfloat16* where = locate(k0);
   for (int i = warp; i < MT * 16; i += MT * 4) {
     const int h = h0 + i;
     const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.q_abs) + r * p.ld_q_abs + 1ll * h * p.kv_pad;
@@ -239,7 +247,8 @@ __global__ void __launch_bounds__(MT * 128) latent_attend_mma_kernel(ds41_latent
       else *reinterpret_cast<uint4*>(sq + i * RS + d) = zero;
     }
   }
-  load(k0, 0);
+  load(where, 0);
+  where = locate(k0 + kKeyTile);
   float acc[NP][2][4];
 #pragma unroll
   for (int i = 0; i < NP; ++i)
@@ -253,19 +262,32 @@ __global__ void __launch_bounds__(MT * 128) latent_attend_mma_kernel(ds41_latent
   int buf = 0;
   for (int t0 = k0; t0 < k1; t0 += kKeyTile, buf ^= 1) {
     if (t0 + kKeyTile < k1) {
-      load(t0 + kKeyTile, buf ^ 1);
+      load(where, buf ^ 1);
+      where = locate(t0 + 2 * kKeyTile);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
     const __nv_bfloat16* kt = sk + buf * kKeyTile * RS;
-    float s[2][4] = {};
+    float s[2][4] = {}, s_odd[2][4] = {};       // two chains: consecutive products into one accumulator wait for each other
     {
       const __nv_bfloat16* arow = sq + (mt * 16 + (lane & 15)) * RS + (lane >> 4) * 8;
       const __nv_bfloat16* brow = kt + (w * 16 + (lane & 7) + (lane >> 4) * 8) * RS + ((lane >> 3) & 1) * 8;
-#pragma unroll 4
-      for (int k = 0; k < RL; k += 16) {
+      int k = 0;
+#pragma unroll 3
+      for (; k + 32 <= RL; k += 32) {
+        uint32_t a[4], b[4], c[4], d[4];
+        ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
+        ldmatrix_x4(b[0], b[1], b[2], b[3], brow + k);
+        ldmatrix_x4(c[0], c[1], c[2], c[3], arow + k + 16);
+        ldmatrix_x4(d[0], d[1], d[2], d[3], brow + k + 16);
+        mma_bf16_16816(s[0], a, b[0], b[1]);
+        mma_bf16_16816(s[1], a, b[2], b[3]);
+        mma_bf16_16816(s_odd[0], c, d[0], d[1]);
+        mma_bf16_16816(s_odd[1], c, d[2], d[3]);
+      }
+      if (k < RL) {
         uint32_t a[4], b[4];
         ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
         ldmatrix_x4(b[0], b[1], b[2], b[3], brow + k);
@@ -279,7 +301,7 @@ __global__ void __launch_bounds__(MT * 128) latent_attend_mma_kernel(ds41_latent
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = t0 + w * 16 + 8 * j + q2 + (e & 1);
-        s[j][e] = key < k1 ? s[j][e] * scale2 : -INFINITY;
+        s[j][e] = key < k1 ? (s[j][e] + s_odd[j][e]) * scale2 : -INFINITY;
         top[e >> 1] = fmaxf(top[e >> 1], s[j][e]);
       }
 #pragma unroll
@@ -427,10 +449,6 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* part_o, 
 }  // namespace ds41
 
 using namespace ds41;
-
-static bool proj_ok(const ds41_proj& p) {
-  return p.data != nullptr && p.ld > 0 && p.splits >= 1 && p.col >= 0 && (p.splits == 1 || (p.plane > 0 && !p.bf16));
-}
 
 extern "C" int ds41_latent_post(const ds41_latent_post_args* a, void* stream) {
   if (a == nullptr || a->rows <= 0 || !proj_ok(a->dq) || a->cq == nullptr || a->dq_norm == nullptr || a->q_rank <= 0 ||

@@ -6,7 +6,8 @@
 // A block owns 32 value columns of one head.  Every column block carries its own copy of n and m, so blocks never wait for
 // one another.  A request's state starts at zero where its rows start at position 0.
 //
-//  mlstm_step : one block walks the adjacent rows of a request token by token (decode rows, 32-bit passes)
+//  mlstm_step : one block walks the adjacent rows of a request token by token (decode rows, 32-bit passes), the state in
+//               registers, or in shared memory where it is too large for them
 //  mlstm_chunk: one request's rows, 64 at a time, on the tensor cores.  With F the running sum of f inside a chunk and m0
 //               the maximum before it, m_t = F_t + max(m0, max_{s<=t}(i_s - F_s)) is the same maximum the walk would find, and
 //                 S'^T q_t = exp(F_t + m0 - m_t) S^T q_t + sum_{s<=t} exp(F_t - F_s + i_s - m_t) (k_s . q_t) v_s
@@ -103,19 +104,206 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(ds41_mlstm_args p) {
   if (tid == 0) *gm = m;
 }
 
+// The same walk with the state in registers: thread (warp, lane) holds rows d = 32 i + 4 warp + lane / 8 and the four columns
+// 4 (lane % 8), i < NR.
+template <int NR>
+__global__ void __launch_bounds__(256) mlstm_walk_kernel(ds41_mlstm_args p) {
+  constexpr int D = NR * 32;
+  __shared__ float qs[D], ks[D];
+  __shared__ float n[D];
+  __shared__ __align__(16) float part[8][kStateCols];
+  __shared__ __align__(16) float vs[kStateCols];
+  __shared__ float red[33];
+  __shared__ float gates[2];
+  const int vb = blockIdx.x, h = blockIdx.y;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  pdl_launch_dependents();
+  pdl_wait();
+  int r = blockIdx.z;
+  if (!segment_start(p.row_slot, r)) return;
+  const int slot = p.row_slot[r];
+  if (slot >= p.slots) return;
+  const int nb = gridDim.x, col0 = vb * kStateCols, c4 = col0 + 4 * (lane & 7), d0 = 4 * warp + (lane >> 3);
+  const bool live = c4 < p.vdim_pad;                 // vdim_pad is a multiple of 4
+  const bool fresh = p.row_pos[r] == 0;
+  const long long head = 1ll * slot * p.heads + h;
+  float* gS = p.state_s + head * p.dim_pad * p.vdim_pad + c4;
+  float* gn = p.state_n + (head * nb + vb) * p.dim_pad;
+  float* gm = p.state_m + head * nb + vb;
+  float4 st[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = 32 * i + d0;
+    st[i] = !fresh && live && d < p.dim_pad ? *reinterpret_cast<const float4*>(gS + 1ll * d * p.vdim_pad)
+                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  for (int d = tid; d < D; d += 256) n[d] = !fresh && d < p.dim_pad ? gn[d] : 0.f;
+  float m = fresh ? 0.f : *gm;
+  for (; r < p.rows && p.row_slot[r] == slot; ++r) {
+    __syncthreads();
+    for (int d = tid; d < D; d += 256) {
+      const bool in = d < p.dim_pad;
+      qs[d] = in ? proj_at(p.q, r, h * p.dim_pad + d) * p.q_scale : 0.f;
+      ks[d] = in ? proj_at(p.k, r, h * p.dim_pad + d) : 0.f;
+    }
+    if (tid < kStateCols) vs[tid] = col0 + tid < p.vdim_pad ? proj_at(p.v, r, h * p.vdim_pad + col0 + tid) : 0.f;
+    if (tid == 32) {
+      const GateValues g = mlstm_gates(p, r, h);
+      gates[0] = g.i;
+      gates[1] = g.f;
+    }
+    __syncthreads();
+    const float m_new = fmaxf(gates[1] + m, gates[0]);
+    const float keep = expf(gates[1] + m - m_new), add = expf(gates[0] - m_new);
+    m = m_new;
+    float nq = 0.f;
+    for (int d = tid; d < D; d += 256) {
+      const float t = keep * n[d] + add * ks[d];
+      n[d] = t;
+      nq += t * qs[d];
+    }
+    float4 v = *reinterpret_cast<const float4*>(vs + 4 * (lane & 7));
+    v.x *= add;
+    v.y *= add;
+    v.z *= add;
+    v.w *= add;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const float k = ks[32 * i + d0], q = qs[32 * i + d0];
+      st[i].x = keep * st[i].x + k * v.x;
+      st[i].y = keep * st[i].y + k * v.y;
+      st[i].z = keep * st[i].z + k * v.z;
+      st[i].w = keep * st[i].w + k * v.w;
+      o.x += st[i].x * q;
+      o.y += st[i].y * q;
+      o.z += st[i].z * q;
+      o.w += st[i].w * q;
+    }
+#pragma unroll
+    for (int x = 8; x <= 16; x <<= 1) {
+      o.x += __shfl_xor_sync(0xffffffffu, o.x, x);
+      o.y += __shfl_xor_sync(0xffffffffu, o.y, x);
+      o.z += __shfl_xor_sync(0xffffffffu, o.z, x);
+      o.w += __shfl_xor_sync(0xffffffffu, o.w, x);
+    }
+    if (lane < 8) *reinterpret_cast<float4*>(&part[warp][4 * lane]) = o;
+    nq = block_sum(nq, red);                // also orders `part`
+    if (warp == 0 && col0 + lane < p.vdim_pad) {
+      float t = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) t += part[w][lane];
+      p.out[1ll * r * p.ld_out + h * p.vdim_pad + col0 + lane] = t / (fmaxf(fabsf(nq), expf(-m)) + p.den_eps);
+    }
+  }
+  if (live)
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = 32 * i + d0;
+      if (d < p.dim_pad) *reinterpret_cast<float4*>(gS + 1ll * d * p.vdim_pad) = st[i];
+    }
+  for (int d = tid; d < p.dim_pad; d += 256) gn[d] = n[d];
+  if (tid == 0) *gm = m;
+}
+
 constexpr int kChunk = 64;
 constexpr int kPStride = kChunk + 8;          // bf16 per row of the decayed scores
 constexpr int kVStride = kStateCols + 8;      // bf16 per row of a value tile
 constexpr int kRedStride = kStateCols + 1;
+// What the gates of one (chunk, head) come to, as the chunk kernel wants it: five rows of 64 values and four scalars.
+//   [0] e_t = (F_t - m_t) log2(e)   [1] a_s = (i_s - F_s) log2(e)   [2] weight of key s in the state after the chunk
+//   [3] q_scale exp(F_t + m0 - m_t)  [4] exp(-m_t)                   scalars: factor on the old state, m after the chunk
+constexpr int kGateFloats = 5 * kChunk + 4;
+
+// One block per head: the gates of every chunk, then the maxima from chunk to chunk.
+__global__ void __launch_bounds__(1024) mlstm_gates_kernel(ds41_mlstm_args p) {
+  extern __shared__ float mg_smem[];          // [n_chunks][3]: F at the end, largest i - F, m before the chunk
+  const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slot = p.row_slot[0];
+  if (slot < 0 || slot >= p.slots) return;
+  const int n_chunks = (p.rows + kChunk - 1) / kChunk;
+  constexpr float kLog2e = 1.4426950408889634f;
+  float F[2], a[2], top[2];
+  auto scan = [&](int c) {
+    float gi[2], gf[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = c * kChunk + 2 * lane + u;
+      gi[u] = -INFINITY;
+      gf[u] = 0.f;
+      if (r < p.rows) {
+        const GateValues g = mlstm_gates(p, r, h);
+        gi[u] = g.i;
+        gf[u] = g.f;
+      }
+    }
+    F[1] = gf[0] + gf[1];                     // running sum up to row 2 lane + 1
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, F[1], o);
+      if (lane >= o) F[1] += x;
+    }
+    F[0] = __shfl_up_sync(0xffffffffu, F[1], 1);
+    F[0] = (lane == 0 ? 0.f : F[0]) + gf[0];
+    a[0] = gi[0] - F[0];
+    a[1] = gi[1] - F[1];
+    top[1] = fmaxf(a[0], a[1]);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, top[1], o);
+      if (lane >= o) top[1] = fmaxf(top[1], x);
+    }
+    top[0] = __shfl_up_sync(0xffffffffu, top[1], 1);
+    top[0] = fmaxf(lane == 0 ? -INFINITY : top[0], a[0]);
+  };
+  for (int c = warp; c < n_chunks; c += 32) {
+    scan(c);
+    if (lane == 31) {
+      mg_smem[3 * c] = F[1];
+      mg_smem[3 * c + 1] = top[1];
+    }
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    const int nb = (p.vdim_pad + kStateCols - 1) / kStateCols;
+    float m = p.row_pos[0] == 0 ? 0.f : p.state_m[(1ll * slot * p.heads + h) * nb];
+    for (int c = 0; c < n_chunks; ++c) {
+      mg_smem[3 * c + 2] = m;
+      m = mg_smem[3 * c] + fmaxf(m, mg_smem[3 * c + 1]);
+    }
+  }
+  __syncthreads();
+  for (int c = warp; c < n_chunks; c += 32) {
+    if (n_chunks > 32) scan(c);               // one chunk per warp keeps its values
+    const float F_end = mg_smem[3 * c], m0 = mg_smem[3 * c + 2], end = fmaxf(m0, mg_smem[3 * c + 1]);
+    float* out = p.work + (1ll * c * p.heads + h) * kGateFloats;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = 2 * lane + u;
+      const float mx = fmaxf(top[u], m0);     // m_t - F_t
+      out[t] = -mx * kLog2e;
+      out[kChunk + t] = a[u] * kLog2e;
+      out[2 * kChunk + t] = expf(a[u] - end);
+      out[3 * kChunk + t] = p.q_scale * expf(m0 - mx);
+      out[4 * kChunk + t] = expf(-(F[u] + mx));
+    }
+    if (lane == 0) {
+      out[5 * kChunk] = expf(m0 - end);
+      out[5 * kChunk + 1] = F_end + end;
+    }
+  }
+}
 
 template <int NTD>
 struct ChunkSmem {
   static constexpr int D = NTD * 32;
   static constexpr int kStride = D + 8;                            // bf16 per row of a q / k tile
   static constexpr int kTile = kChunk * kStride * 2;               // bytes
-  static constexpr int kStage = 2 * kTile + kChunk * kVStride * 2;
-  static constexpr int kFixed = 2 * kChunk * kPStride * 2 + 2 * kChunk * kVStride * 2 + 4 * kChunk * kRedStride * 4 +
-                                D * 4 + 7 * kChunk * 4 + 64;
+  static constexpr int kStage = 2 * kTile + kChunk * kVStride * 2 + kGateFloats * 4;
+  static constexpr int kFixed = 2 * kChunk * kPStride * 2 + 2 * kChunk * kVStride * 2 + 8 * kStride * 2 +
+                                4 * kChunk * kRedStride * 4 + D * 4 + 4 * kChunk * 4;
   static constexpr int kStages = 2 * kStage + kFixed <= 226 * 1024 ? 2 : 1;
   static constexpr int kBytes = kStages * kStage + kFixed;
 };
@@ -132,15 +320,12 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
   __nv_bfloat16* p_lo = p_hi + kChunk * kPStride;
   __nv_bfloat16* w_hi = p_lo + kChunk * kPStride;
   __nv_bfloat16* w_lo = w_hi + kChunk * kVStride;
-  float* red = reinterpret_cast<float*>(w_lo + kChunk * kVStride);     // [4][64][33]
+  __nv_bfloat16* n_rows = w_lo + kChunk * kVStride;                    // [8][D + 8]: n as high and low parts, zero rows
+  float* red = reinterpret_cast<float*>(n_rows + 8 * Sm::kStride);     // [4][64][33]
   float* nv = red + 4 * kChunk * kRedStride;                           // [D]
-  float* g_e = nv + D;                 // F_t - m_t
-  float* g_a = g_e + kChunk;           // i_s - F_s
-  float* g_m = g_a + kChunk;           // m_t
-  float* g_w = g_m + kChunk;           // weight of key s in the state after the chunk
-  float* nq = g_w + kChunk;            // n . q_t before the chunk
+  float* nq = nv + D;                  // n . q_t before the chunk
   float* rs = nq + kChunk;             // [2][64] sums of the decayed scores
-  float* carry = rs + 2 * kChunk;      // factor on the state, new m
+  float* inv = rs + 2 * kChunk;        // 1 / denominator
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int vb = blockIdx.x, h = blockIdx.y;
   const int nt = warp & 1, dq = warp >> 1, g = lane >> 2, q2 = 2 * (lane & 3);
@@ -153,8 +338,44 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
   const long long head = 1ll * slot * p.heads + h;
   float* gS = p.state_s + head * p.dim_pad * p.vdim_pad;
   float* gn = p.state_n + (head * nb + vb) * p.dim_pad;
-  float* gm = p.state_m + head * nb + vb;
 
+  const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(p.q.data) + p.q.col + h * p.dim_pad;
+  const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad;
+  const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(p.v.data) + p.v.col + h * p.vdim_pad + col0;
+  const int n_chunks = (p.rows + kChunk - 1) / kChunk;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  auto load = [&](int c, int stage) {
+    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(mc_smem + stage * Sm::kStage);
+    __nv_bfloat16* sk = sq + kChunk * Sm::kStride;
+    __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
+    const int live = p.rows - c * kChunk;
+    constexpr int kPer = D / 8;                       // 16-byte pieces of a row
+    constexpr int kRows = kPer <= 256 ? 256 / kPer : 1;
+    if (kPer * kRows == 256 || tid < kPer * kRows) {
+      const int d = (tid % kPer) * 8;
+      const __nv_bfloat16* q = gq + (1ll * c * kChunk + tid / kPer) * p.q.ld + d;
+      const __nv_bfloat16* k = gk + (1ll * c * kChunk + tid / kPer) * p.k.ld + d;
+      for (int t = tid / kPer; t < kChunk; t += kRows, q += 1ll * kRows * p.q.ld, k += 1ll * kRows * p.k.ld) {
+        if (t < live && d < p.dim_pad) {
+          cp_async_16(sq + t * Sm::kStride + d, q);
+          cp_async_16(sk + t * Sm::kStride + d, k);
+        } else {
+          *reinterpret_cast<uint4*>(sq + t * Sm::kStride + d) = zero;
+          *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
+        }
+      }
+    }
+    {
+      const int t = tid >> 2, d = (tid & 3) * 8;
+      if (t < live && col0 + d < p.vdim_pad) cp_async_16(sv + t * kVStride + d, gv + (1ll * c * kChunk + t) * p.v.ld + d);
+      else *reinterpret_cast<uint4*>(sv + t * kVStride + d) = zero;
+    }
+    if (tid < kGateFloats / 4)
+      cp_async_16(reinterpret_cast<float*>(sv + kChunk * kVStride) + 4 * tid,
+                  p.work + (1ll * c * p.heads + h) * kGateFloats + 4 * tid);
+    cp_async_commit();
+  };
+  load(0, 0);
   // transposed state: tile j holds columns d = dq DQ + 8 j + q2 + {0, 1} of rows nt 16 + g and + 8
   float st[NTD][4];
 #pragma unroll
@@ -164,48 +385,16 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       const int d = dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
       st[j][e] = !fresh && d < p.dim_pad && c < p.vdim_pad ? gS[1ll * d * p.vdim_pad + c] : 0.f;
     }
-  for (int d = tid; d < D; d += 256) nv[d] = !fresh && d < p.dim_pad ? gn[d] : 0.f;
-  float m0 = fresh ? 0.f : *gm;
-
-  const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(p.q.data) + p.q.col + h * p.dim_pad;
-  const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad;
-  const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(p.v.data) + p.v.col + h * p.vdim_pad + col0;
-  const int n_chunks = (p.rows + kChunk - 1) / kChunk;
-  auto load = [&](int c, int stage) {
-    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(mc_smem + stage * Sm::kStage);
-    __nv_bfloat16* sk = sq + kChunk * Sm::kStride;
-    __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
-    const uint4 zero = make_uint4(0, 0, 0, 0);
-    for (int i = tid; i < kChunk * (D / 8); i += 256) {
-      const int t = i / (D / 8), d = (i - t * (D / 8)) * 8, r = c * kChunk + t;
-      if (r < p.rows && d < p.dim_pad) {
-        cp_async_16(sq + t * Sm::kStride + d, gq + 1ll * r * p.q.ld + d);
-        cp_async_16(sk + t * Sm::kStride + d, gk + 1ll * r * p.k.ld + d);
-      } else {
-        *reinterpret_cast<uint4*>(sq + t * Sm::kStride + d) = zero;
-        *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
-      }
-    }
-    {
-      const int t = tid >> 2, d = (tid & 3) * 8, r = c * kChunk + t;
-      if (r < p.rows && col0 + d < p.vdim_pad) cp_async_16(sv + t * kVStride + d, gv + 1ll * r * p.v.ld + d);
-      else *reinterpret_cast<uint4*>(sv + t * kVStride + d) = zero;
-    }
-    cp_async_commit();
-  };
-  // raw gates of the next chunk travel in registers of warp 0 (rows 2 lane and 2 lane + 1)
-  float raw_i[2], raw_f[2];
-  auto load_gates = [&](int c) {
-    if (warp == 0)
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int r = c * kChunk + 2 * lane + u;
-        raw_i[u] = r < p.rows ? proj_at(p.gate_i, r, h) + p.bias_i[h] : 0.f;
-        raw_f[u] = r < p.rows ? proj_at(p.gate_f, r, h) + p.bias_f[h] : 0.f;
-      }
-  };
-  load(0, 0);
-  load_gates(0);
+  for (int i = tid; i < 8 * Sm::kStride; i += 256) n_rows[i] = __float2bfloat16_rn(0.f);
+  __syncthreads();
+  for (int d = tid; d < D; d += 256) {
+    const float x = !fresh && d < p.dim_pad ? gn[d] : 0.f;
+    const __nv_bfloat16 hi = __float2bfloat16_rn(x);
+    nv[d] = x;
+    n_rows[d] = hi;
+    n_rows[Sm::kStride + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
+  }
+  float m_end = 0.f;
   for (int c = 0; c < n_chunks; ++c) {
     const int stage = Sm::kStages == 2 ? (c & 1) : 0;
     if (Sm::kStages == 2 && c + 1 < n_chunks) {
@@ -217,56 +406,17 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
     const __nv_bfloat16* sq = reinterpret_cast<const __nv_bfloat16*>(mc_smem + stage * Sm::kStage);
     const __nv_bfloat16* sk = sq + kChunk * Sm::kStride;
     const __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
-    if (warp == 0) {
-      float gi[2], gf[2];
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const bool live = c * kChunk + 2 * lane + u < p.rows;
-        gi[u] = live ? p.gate_cap * tanhf(raw_i[u] / p.gate_cap) : -INFINITY;
-        gf[u] = live ? log_sigmoid_f32(p.gate_cap * tanhf(raw_f[u] / p.gate_cap)) : 0.f;
-      }
-      float F1 = gf[0] + gf[1];                       // running sum up to row 2 lane + 1
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, F1, o);
-        if (lane >= o) F1 += x;
-      }
-      float F0 = __shfl_up_sync(0xffffffffu, F1, 1);
-      F0 = (lane == 0 ? 0.f : F0) + gf[0];
-      const float a0 = gi[0] - F0, a1 = gi[1] - F1;
-      float top1 = fmaxf(a0, a1);
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, top1, o);
-        if (lane >= o) top1 = fmaxf(top1, x);
-      }
-      float top0 = __shfl_up_sync(0xffffffffu, top1, 1);
-      top0 = fmaxf(lane == 0 ? m0 : fmaxf(top0, m0), a0);
-      top1 = fmaxf(top1, m0);
-      const float F_end = __shfl_sync(0xffffffffu, F1, 31), top_end = __shfl_sync(0xffffffffu, top1, 31);
-      g_e[2 * lane] = -top0;                          // F_t - m_t
-      g_e[2 * lane + 1] = -top1;
-      g_a[2 * lane] = a0;
-      g_a[2 * lane + 1] = a1;
-      g_m[2 * lane] = F0 + top0;
-      g_m[2 * lane + 1] = F1 + top1;
-      g_w[2 * lane] = expf(a0 - top_end);
-      g_w[2 * lane + 1] = expf(a1 - top_end);
-      if (lane == 0) {
-        carry[0] = expf(m0 - top_end);
-        carry[1] = F_end + top_end;
-      }
-      if (c + 1 < n_chunks) load_gates(c + 1);
-    }
+    const float* gates = reinterpret_cast<const float*>(sv + kChunk * kVStride);
     __syncthreads();
 
-    // ---- decayed scores: 16 rows x 32 keys per warp
+    // ---- decayed scores, 16 rows x 32 keys per warp; the warps of the first keys also take n . q_t
     {
       const int tm = warp >> 1, sh = warp & 1;
-      float acc[4][4] = {};
+      float acc[4][4] = {}, na[4] = {};
+      const __nv_bfloat16* arow = sq + (tm * 16 + (lane & 15)) * Sm::kStride + (lane >> 4) * 8;
+      const __nv_bfloat16* brow = sk + (sh * 32 + (lane & 7) + (lane >> 4) * 8) * Sm::kStride + ((lane >> 3) & 1) * 8;
+      const __nv_bfloat16* nrow = n_rows + (lane & 7) * Sm::kStride + (lane >> 3) * 8;
       if (sh * 32 <= tm * 16 + 15) {
-        const __nv_bfloat16* arow = sq + (tm * 16 + (lane & 15)) * Sm::kStride + (lane >> 4) * 8;
-        const __nv_bfloat16* brow = sk + (sh * 32 + (lane & 7) + (lane >> 4) * 8) * Sm::kStride + ((lane >> 3) & 1) * 8;
 #pragma unroll 4
         for (int k = 0; k < D; k += 16) {
           uint32_t a[4], b[8];
@@ -277,16 +427,32 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
           for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[j], a, b[2 * j], b[2 * j + 1]);
         }
       }
+      if (sh == 0) {
+#pragma unroll 2
+        for (int k = 0; k < D; k += 32) {
+          uint32_t a[4], b[4];
+          ldmatrix_x4(b[0], b[1], b[2], b[3], nrow + k);
+          ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
+          mma_bf16_16816(na, a, b[0], b[1]);
+          ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k + 16);
+          mma_bf16_16816(na, a, b[2], b[3]);
+        }
+        if ((lane & 3) == 0) {
+          nq[tm * 16 + g] = na[0] + na[1];
+          nq[tm * 16 + g + 8] = na[2] + na[3];
+        }
+      }
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
         const int t = tm * 16 + g + 8 * u;
-        const float e = g_e[t];
+        const float e = gates[t];
         float sum = 0.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int s = sh * 32 + 8 * j + q2;
-          const float x = s <= t ? acc[j][2 * u] * p.q_scale * expf(e + g_a[s]) : 0.f;
-          const float y = s + 1 <= t ? acc[j][2 * u + 1] * p.q_scale * expf(e + g_a[s + 1]) : 0.f;
+          const float2 as = *reinterpret_cast<const float2*>(gates + kChunk + s);
+          const float x = s <= t ? acc[j][2 * u] * p.q_scale * ex2_approx(e + as.x) : 0.f;
+          const float y = s + 1 <= t ? acc[j][2 * u + 1] * p.q_scale * ex2_approx(e + as.y) : 0.f;
           sum += x + y;
           const uint32_t hi = pack_bf16(x, y);
           *reinterpret_cast<uint32_t*>(p_hi + t * kPStride + s) = hi;
@@ -297,27 +463,21 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
         if ((lane & 3) == 0) rs[sh * kChunk + t] = sum;
       }
     }
-    // ---- decayed values, n . q
+    // ---- decayed values
     {
       const int s = tid >> 2, d = (tid & 3) * 8;
-      const float w = g_w[s];
+      const float w = gates[2 * kChunk + s];
+      const uint4 v4 = *reinterpret_cast<const uint4*>(sv + s * kVStride + d);
+      const uint32_t v[4] = {v4.x, v4.y, v4.z, v4.w};
+      uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int i = 0; i < 8; i += 2) {
-        const float x = __bfloat162float(sv[s * kVStride + d + i]) * w, y = __bfloat162float(sv[s * kVStride + d + i + 1]) * w;
-        const uint32_t hi = pack_bf16(x, y);
-        *reinterpret_cast<uint32_t*>(w_hi + s * kVStride + d + i) = hi;
-        *reinterpret_cast<uint32_t*>(w_lo + s * kVStride + d + i) = pack_bf16_rest(x, y, hi);
+      for (int i = 0; i < 4; ++i) {
+        const float x = __uint_as_float(v[i] << 16) * w, y = __uint_as_float(v[i] & 0xffff0000u) * w;
+        hi[i] = pack_bf16(x, y);
+        lo[i] = pack_bf16_rest(x, y, hi[i]);
       }
-#pragma unroll 2
-      for (int t = warp * 8; t < warp * 8 + 8; ++t) {
-        float x = 0.f;
-        for (int i = 2 * lane; i < D; i += 64) {
-          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sq + t * Sm::kStride + i));
-          x += nv[i] * f.x + nv[i + 1] * f.y;
-        }
-        x = warp_sum(x);
-        if (lane == 0) nq[t] = x * p.q_scale;
-      }
+      *reinterpret_cast<uint4*>(w_hi + s * kVStride + d) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(w_lo + s * kVStride + d) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
     __syncthreads();
 
@@ -346,12 +506,11 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        const int t = 8 * j + q2;
-        const float x = p.q_scale * expf(g_e[t] + m0), y = p.q_scale * expf(g_e[t + 1] + m0);
-        o[j][0] *= x;
-        o[j][1] *= y;
-        o[j][2] *= x;
-        o[j][3] *= y;
+        const float2 f = *reinterpret_cast<const float2*>(gates + 3 * kChunk + 8 * j + q2);
+        o[j][0] *= f.x;
+        o[j][1] *= f.y;
+        o[j][2] *= f.x;
+        o[j][3] *= f.y;
       }
       uint32_t a[4];
       ldmatrix_x4_trans(a[0], a[1], a[2], a[3],
@@ -373,9 +532,13 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) dst[(8 * j + q2 + (e & 1)) * kRedStride + (e >> 1) * 8] = o[j][e];
     }
+    if (tid < kChunk)
+      inv[tid] = 1.0f / (fmaxf(fabsf(gates[3 * kChunk + tid] * nq[tid] + rs[tid] + rs[kChunk + tid]), gates[4 * kChunk + tid]) +
+                         p.den_eps);
     // ---- state after the chunk
     {
-      const float keep = carry[0];
+      const float keep = gates[5 * kChunk];
+      m_end = gates[5 * kChunk + 1];
 #pragma unroll
       for (int j = 0; j < NTD; ++j)
 #pragma unroll
@@ -397,31 +560,61 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
           mma_bf16_16816(st[2 * j + 1], lo, b[2], b[3]);
         }
       }
-      for (int d = 2 * tid; d < D; d += 512) {
-        float x = nv[d] * keep, y = nv[d + 1] * keep;
-#pragma unroll 8
-        for (int s = 0; s < kChunk; ++s) {
-          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sk + s * Sm::kStride + d));
-          x += g_w[s] * f.x;
-          y += g_w[s] * f.y;
+      // n: one row of weights (high parts in row 0, low parts in row 1 of the left operand) times the keys; the two warps
+      // of a quarter take half of its columns each
+      uint32_t wf[4][2];
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float2 w = *reinterpret_cast<const float2*>(gates + 2 * kChunk + 16 * k + 8 * e + q2);
+          const uint32_t hi = pack_bf16(w.x, w.y);
+          wf[k][e] = g == 0 ? hi : (g == 1 ? pack_bf16_rest(w.x, w.y, hi) : 0u);
         }
-        nv[d] = x;
-        nv[d + 1] = y;
+#pragma unroll
+      for (int j = nt; j < NTD / 2; j += 2) {
+        float x[4] = {}, y[4] = {};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          uint32_t b[4];
+          const uint32_t a[4] = {wf[k][0], 0u, wf[k][1], 0u};
+          ldmatrix_x4_trans(b[0], b[1], b[2], b[3], brow + 16 * k * Sm::kStride + 16 * j);
+          mma_bf16_16816(x, a, b[0], b[1]);
+          mma_bf16_16816(y, a, b[2], b[3]);
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          x[e] += __shfl_down_sync(0xffffffffu, x[e], 4);       // rows 0 and 1 of a column meet in row 0's lanes
+          y[e] += __shfl_down_sync(0xffffffffu, y[e], 4);
+        }
+        if (g == 0) {
+          const int d = dq * DQ + 16 * j + q2;
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const int at = d + 8 * u;
+            const float n0 = nv[at] * keep + (u == 0 ? x[0] : y[0]), n1 = nv[at + 1] * keep + (u == 0 ? x[1] : y[1]);
+            nv[at] = n0;
+            nv[at + 1] = n1;
+            const uint32_t hi = pack_bf16(n0, n1);
+            *reinterpret_cast<uint32_t*>(n_rows + at) = hi;
+            *reinterpret_cast<uint32_t*>(n_rows + Sm::kStride + at) = pack_bf16_rest(n0, n1, hi);
+          }
+        }
       }
     }
     __syncthreads();
+    if (col0 + lane < p.vdim_pad) {
+      const int t0 = warp * 8, live = min(8, p.rows - c * kChunk - t0);
+      float* dst = p.out + (1ll * c * kChunk + t0) * p.ld_out + h * p.vdim_pad + col0 + lane;
+      const float* src = red + t0 * kRedStride + lane;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int t = warp * 8 + i, r = c * kChunk + t;
-      if (r < p.rows && col0 + lane < p.vdim_pad) {
+      for (int i = 0; i < 8; ++i) {
         float x = 0.f;
 #pragma unroll
-        for (int w = 0; w < 4; ++w) x += red[(w * kChunk + t) * kRedStride + lane];
-        const float dot = expf(g_e[t] + m0) * nq[t] + rs[t] + rs[kChunk + t];
-        p.out[1ll * r * p.ld_out + h * p.vdim_pad + col0 + lane] = x / (fmaxf(fabsf(dot), expf(-g_m[t])) + p.den_eps);
+        for (int w = 0; w < 4; ++w) x += src[(w * kChunk + i) * kRedStride];
+        if (i < live) dst[1ll * i * p.ld_out] = x * inv[t0 + i];
       }
     }
-    m0 = carry[1];
     __syncthreads();
     if (Sm::kStages == 1 && c + 1 < n_chunks) load(c + 1, 0);
   }
@@ -433,7 +626,7 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       if (d < p.dim_pad && cc < p.vdim_pad) gS[1ll * d * p.vdim_pad + cc] = st[j][e];
     }
   for (int d = tid; d < p.dim_pad; d += 256) gn[d] = nv[d];
-  if (tid == 0) *gm = m0;
+  if (tid == 0) p.state_m[head * nb + vb] = m_end;
 }
 
 template <int NTD>
@@ -445,6 +638,10 @@ static int launch_chunk(const ds41_mlstm_args& a, cudaStream_t st) {
     if (e != cudaSuccess) return e;
     ready = true;
   }
+  const size_t gate_smem = 3ull * ((a.rows + kChunk - 1) / kChunk) * sizeof(float);
+  if (gate_smem > 48 * 1024) return cudaErrorInvalidValue;
+  const cudaError_t e = launch_pdl(mlstm_gates_kernel, dim3(a.heads), dim3(1024), gate_smem, st, a);
+  if (e != cudaSuccess) return e;
   const dim3 grid((a.vdim_pad + kStateCols - 1) / kStateCols, a.heads);
   return launch_pdl(mlstm_chunk_kernel<NTD>, grid, dim3(256), ChunkSmem<NTD>::kBytes, st, a);
 }
@@ -452,10 +649,6 @@ static int launch_chunk(const ds41_mlstm_args& a, cudaStream_t st) {
 }  // namespace ds41
 
 using namespace ds41;
-
-static bool proj_ok(const ds41_proj& p) {
-  return p.data != nullptr && p.ld > 0 && p.splits >= 1 && p.col >= 0 && (p.splits == 1 || (p.plane > 0 && !p.bf16));
-}
 
 static bool mlstm_args_ok(const ds41_mlstm_args* a) {
   return a != nullptr && a->rows > 0 && a->rows <= 65535 && a->heads > 0 && a->heads <= 65535 && a->dim_pad > 0 &&
@@ -467,6 +660,15 @@ static bool mlstm_args_ok(const ds41_mlstm_args* a) {
 
 extern "C" int ds41_mlstm_step(const ds41_mlstm_args* a, void* stream) {
   if (!mlstm_args_ok(a)) return cudaErrorInvalidValue;
+  if (!(a->vdim_pad & 3) && a->dim_pad <= 512 && !(reinterpret_cast<uintptr_t>(a->state_s) & 15)) {
+    const dim3 grid((a->vdim_pad + kStateCols - 1) / kStateCols, a->heads, a->rows);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a->dim_pad <= 32) return launch_pdl(mlstm_walk_kernel<1>, grid, dim3(256), 0, st, *a);
+    if (a->dim_pad <= 64) return launch_pdl(mlstm_walk_kernel<2>, grid, dim3(256), 0, st, *a);
+    if (a->dim_pad <= 128) return launch_pdl(mlstm_walk_kernel<4>, grid, dim3(256), 0, st, *a);
+    if (a->dim_pad <= 256) return launch_pdl(mlstm_walk_kernel<8>, grid, dim3(256), 0, st, *a);
+    return launch_pdl(mlstm_walk_kernel<16>, grid, dim3(256), 0, st, *a);
+  }
   const size_t smem = (1ull * a->dim_pad * (kStateCols + 3) + kStateCols * 9) * sizeof(float);
   static size_t allowed = 48 * 1024 - 512;
   if (smem > allowed) {
@@ -484,7 +686,7 @@ extern "C" int ds41_mlstm_chunk(const ds41_mlstm_args* a, void* stream) {
   if (!mlstm_args_ok(a)) return cudaErrorInvalidValue;
   for (const ds41_proj* x : {&a->q, &a->k, &a->v})
     if (!x->bf16 || (x->ld & 7) || (x->col & 7) || (reinterpret_cast<uintptr_t>(x->data) & 15)) return cudaErrorInvalidValue;
-  if ((a->dim_pad & 15) || (a->vdim_pad & 15)) return cudaErrorInvalidValue;
+  if ((a->dim_pad & 15) || (a->vdim_pad & 15) || a->work == nullptr || (reinterpret_cast<uintptr_t>(a->work) & 15)) return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a->dim_pad <= 64) return launch_chunk<2>(*a, st);
   if (a->dim_pad <= 128) return launch_chunk<4>(*a, st);
@@ -493,4 +695,8 @@ extern "C" int ds41_mlstm_chunk(const ds41_mlstm_args* a, void* stream) {
   if (a->dim_pad <= 384) return launch_chunk<12>(*a, st);
   if (a->dim_pad <= 512) return launch_chunk<16>(*a, st);
   return cudaErrorInvalidValue;
+}
+
+extern "C" long long ds41_mlstm_chunk_work(int rows, int heads) {
+  return rows <= 0 || heads <= 0 ? 0 : 4ll * kGateFloats * heads * ((rows + kChunk - 1) / kChunk);
 }

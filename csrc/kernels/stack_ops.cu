@@ -47,88 +47,146 @@ __device__ __forceinline__ Moments merge_moments(Moments own, float* slot) {
   }
 }
 
-// Norm factors of a row held in shared memory: layer norm (subtract the mean) or RMS norm (mean of squares).
-template <int CL>
-__device__ __forceinline__ float2 row_norm(const float* v, int n, int W, int kind, float eps, float* red, float* slot) {
+// Subtrahend and factor of a row's norm - layer norm (subtract the mean) or RMS norm (mean of squares) - from the pieces of
+// four columns that the threads hold; `n` columns of the row are in this CTA, piece i covers columns 4 (tid + i blockDim).
+template <int CL, int NI>
+__device__ __forceinline__ float2 row_norm(const float4 (&v)[NI], int n, int W, int kind, float eps, float* red, float* slot) {
   float mean = 0.f;
   if (kind == 0) {
-    float s = 0.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) s += v[i];
+    float s = 0.f;                       // columns beyond the row hold zeros
+#pragma unroll
+    for (int i = 0; i < NI; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
     mean = n > 0 ? block_sum(s, red) / n : 0.f;
   }
   float q = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float d = v[i] - mean;
-    q += d * d;
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int live = n - 4 * (threadIdx.x + i * blockDim.x);
+    const float a = v[i].x - mean, b = v[i].y - mean, c = v[i].z - mean, d = v[i].w - mean;
+    q += (live > 0 ? a * a : 0.f) + (live > 1 ? b * b : 0.f) + (live > 2 ? c * c : 0.f) + (live > 3 ? d * d : 0.f);
   }
   q = block_sum(q, red);
-  if (kind == 0) {
-    const Moments t = merge_moments<CL>({mean, q, static_cast<float>(n)}, slot);
-    return make_float2(t.mean, 1.0f / sqrtf(t.m2 / W + eps));
-  }
-  // the means of squares add up: reuse the exchange with zero means
-  const Moments t = merge_moments<CL>({0.f, q, static_cast<float>(n)}, slot);
-  return make_float2(0.f, 1.0f / sqrtf(t.m2 / W + eps));
+  // the means of squares add up: an RMS norm goes through the same exchange with zero means
+  const Moments t = merge_moments<CL>({mean, q, static_cast<float>(n)}, slot);
+  return make_float2(t.mean, 1.0f / sqrtf(t.m2 / W + eps));
 }
 
-template <typename T, int CL>
-__global__ void __launch_bounds__(512) resid_step_kernel(ds41_resid_args p) {
-  extern __shared__ float row_smem[];
+template <typename T, int CL, int NI>
+__global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_kernel(ds41_resid_args p) {
   __shared__ float red[33];
   __shared__ float slots[2][3];
-  const int per = (p.W + CL - 1) / CL;
+  const int per = ((p.W + CL - 1) / CL + 3) / 4 * 4;
   const int part = CL > 1 ? blockIdx.x % CL : 0;
   const int r = CL > 1 ? blockIdx.x / CL : blockIdx.x;
   const int c0 = min(p.W, part * per), n = min(p.W, c0 + per) - c0;
-  float* x = row_smem;
-  float* y = row_smem + per;
   pdl_launch_dependents();
   pdl_wait();
+  float4 x[NI];
+  int at[NI], live[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    at[i] = 4 * (threadIdx.x + i * blockDim.x);
+    live[i] = n - at[i];
+    x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   if (p.tokens != nullptr) {
     const int tok = p.tokens[r];
-    const bool ok = tok >= 0 && tok < p.vocab;
-    const __nv_bfloat16* e = static_cast<const __nv_bfloat16*>(p.embed) + (ok ? tok : 0) * p.embed_ld + c0;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) x[i] = ok ? __bfloat162float(e[i]) : 0.f;
+    const ds41_proj e{p.embed, 0, static_cast<int>(p.embed_ld), 1, 1, c0};
+    if (tok >= 0 && tok < p.vocab)
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+        if (live[i] > 0) x[i] = proj_at4(e, tok, at[i]);
   } else {
     const float* in = p.x_in + r * p.ldx + c0;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) x[i] = in[i];
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      if (live[i] > 0) x[i] = *reinterpret_cast<const float4*>(in + at[i]);
   }
+  auto clip = [&](float4& v, int i) {         // columns beyond the row hold zeros
+    if (live[i] < 4) v.w = 0.f;
+    if (live[i] < 3) v.z = 0.f;
+    if (live[i] < 2) v.y = 0.f;
+  };
   if (p.y.data != nullptr) {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      float v = proj_at(p.y, r, c0 + i);
-      if (p.gate.data != nullptr) v *= sigmoid_f32(proj_at(p.gate, r, c0 + i) + p.gate_bias[c0 + i]);
-      y[i] = v;
+    float4 y[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (live[i] > 0) {
+        y[i] = proj_at4(p.y, r, c0 + at[i]);
+        if (p.gate.data != nullptr) {
+          const float4 g = proj_at4(p.gate, r, c0 + at[i]), b = load4(p.gate_bias + c0 + at[i], live[i]);
+          y[i].x *= sigmoid_f32(g.x + b.x);
+          y[i].y *= sigmoid_f32(g.y + b.y);
+          y[i].z *= sigmoid_f32(g.z + b.z);
+          y[i].w *= sigmoid_f32(g.w + b.w);
+        }
+        clip(y[i], i);
+      }
     }
-    if (p.post_w != nullptr) {
-      const float2 s = row_norm<CL>(y, n, p.W, p.norm_kind, p.eps, red, slots[0]);
-      for (int i = threadIdx.x; i < n; i += blockDim.x) x[i] += (y[i] - s.x) * s.y * p.post_w[c0 + i];
-    } else {
-      for (int i = threadIdx.x; i < n; i += blockDim.x) x[i] += y[i];
-    }
+    float2 s = make_float2(0.f, 1.f);
+    if (p.post_w != nullptr) s = row_norm<CL, NI>(y, n, p.W, p.norm_kind, p.eps, red, slots[0]);
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      if (live[i] > 0) {
+        const float4 w = p.post_w != nullptr ? load4(p.post_w + c0 + at[i], live[i]) : make_float4(1.f, 1.f, 1.f, 1.f);
+        x[i].x += (y[i].x - s.x) * s.y * w.x;
+        x[i].y += (y[i].y - s.x) * s.y * w.y;
+        x[i].z += (y[i].z - s.x) * s.y * w.z;
+        x[i].w += (y[i].w - s.x) * s.y * w.w;
+      }
   }
+#pragma unroll
+  for (int i = 0; i < NI; ++i) clip(x[i], i);
   if (p.x_out != nullptr) {
     float* o = p.x_out + r * p.ldx + c0;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) o[i] = x[i];
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      if (live[i] > 0) store4(o + at[i], x[i]);
   }
   if (p.mix != nullptr) {
     // weighted sum of the kept streams; the newest one is the row this block holds
     const float* k0 = p.kept + r * p.ldx + c0;
     const float last = p.mix[p.n_mix - 1];
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      float s = last * x[i];
-#pragma unroll 8
-      for (int j = 0; j < p.n_mix - 1; ++j) s += p.mix[j] * k0[j * p.kept_stride + i];
-      x[i] = s;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      x[i].x *= last;
+      x[i].y *= last;
+      x[i].z *= last;
+      x[i].w *= last;
     }
+#pragma unroll 4
+    for (int j = 0; j < p.n_mix - 1; ++j) {
+      const float c = p.mix[j];
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+        if (live[i] > 0) {
+          const float4 k = *reinterpret_cast<const float4*>(k0 + j * p.kept_stride + at[i]);
+          x[i].x += c * k.x;
+          x[i].y += c * k.y;
+          x[i].z += c * k.z;
+          x[i].w += c * k.w;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NI; ++i) clip(x[i], i);
     if (p.x_avg != nullptr) {
       float* o = p.x_avg + r * p.ldx + c0;
-      for (int i = threadIdx.x; i < n; i += blockDim.x) o[i] = x[i];
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+        if (live[i] > 0) store4(o + at[i], x[i]);
     }
   }
   if (p.next_w != nullptr) {
-    const float2 s = row_norm<CL>(x, n, p.W, p.norm_kind, p.eps, red, slots[1]);
-    T* h = static_cast<T*>(p.h) + r * p.ldh + c0;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) h[i] = from_f32<T>((x[i] - s.x) * s.y * p.next_w[c0 + i]);
+    const float2 s = row_norm<CL, NI>(x, n, p.W, p.norm_kind, p.eps, red, slots[1]);
+    T* h = static_cast<T*>(p.h) + 1ll * r * p.ldh + c0;
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      if (live[i] > 0) {
+        const float4 w = load4(p.next_w + c0 + at[i], live[i]);
+        store4(h + at[i], make_float4((x[i].x - s.x) * s.y * w.x, (x[i].y - s.x) * s.y * w.y, (x[i].z - s.x) * s.y * w.z,
+                                      (x[i].w - s.x) * s.y * w.w));
+      }
   }
   if constexpr (CL > 1) cg::this_cluster().sync();      // peers may still read this CTA's moments
 }
@@ -142,21 +200,33 @@ __global__ void __launch_bounds__(512) polynorm_kernel(ds41_proj z, const float*
   pdl_launch_dependents();
   pdl_wait();
   float s2 = 0.f, s4 = 0.f, s6 = 0.f;
-  for (int i = threadIdx.x; i < ff; i += blockDim.x) {
-    const float v = proj_at(z, r, i), q = v * v;
-    zrow[i] = v;
+  auto add = [&](float v) {
+    const float q = v * v;
     s2 += q;
     s4 += q * q;
     s6 += q * q * q;
+  };
+#pragma unroll 4
+  for (int i = 4 * threadIdx.x; i < ff; i += 4 * blockDim.x) {
+    float4 v = proj_at4(z, r, i);
+    if (i + 3 >= ff) v.w = 0.f;            // columns beyond ff add nothing to the sums
+    if (i + 2 >= ff) v.z = 0.f;
+    if (i + 1 >= ff) v.y = 0.f;
+    *reinterpret_cast<float4*>(zrow + i) = v;
+    add(v.x);
+    add(v.y);
+    add(v.z);
+    add(v.w);
   }
   s2 = block_sum(s2, red);
   s4 = block_sum(s4, red);
   s6 = block_sum(s6, red);
   const float a = coef[0] / sqrtf(s2 / ff + eps), b = coef[1] / sqrtf(s4 / ff + eps), c = coef[2] / sqrtf(s6 / ff + eps);
   const float e = coef[3];
-  for (int i = threadIdx.x; i < ff; i += blockDim.x) {
-    const float v = zrow[i];
-    out[1ll * r * ld_out + i] = from_f32<T>(((c * v + b) * v + a) * v + e);
+  auto act = [&](float v) { return ((c * v + b) * v + a) * v + e; };
+  for (int i = 4 * threadIdx.x; i < ff; i += 4 * blockDim.x) {
+    const float4 v = *reinterpret_cast<const float4*>(zrow + i);
+    store4(out + 1ll * r * ld_out + i, make_float4(act(v.x), act(v.y), act(v.z), act(v.w)));
   }
 }
 
@@ -199,34 +269,26 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const T* src, int ld, 
   dst[1ll * r * ld + i] = s >= 0 && s < n_src ? src[1ll * s * ld + i] : from_f32<T>(0.f);
 }
 
+template <typename T, int CL, int NI>
+static cudaError_t launch_resid_ni(const ds41_resid_args& a, int threads, cudaStream_t st) {
+  if constexpr (CL == 1) return launch_pdl(resid_step_kernel<T, CL, NI>, dim3(a.rows), dim3(threads), 0, st, a);
+  else return launch_pdl_cluster(resid_step_kernel<T, CL, NI>, dim3(a.rows * CL), dim3(threads), CL, 0, st, a);
+}
+
 template <typename T, int CL>
 static cudaError_t launch_resid(const ds41_resid_args& a, cudaStream_t st) {
-  const int per = (a.W + CL - 1) / CL;
-  const size_t smem = 2ull * per * sizeof(float);
-  static size_t allowed = 48 * 1024 - 512;
-  if (smem > allowed) {
-    if (smem > 226 * 1024) return cudaErrorInvalidValue;
-    const cudaError_t e = cudaFuncSetAttribute(resid_step_kernel<T, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               static_cast<int>(smem));
-    if (e != cudaSuccess) return e;
-    allowed = smem;
-  }
-  int threads = (per + 31) / 32 * 32;
-  threads = threads < 64 ? 64 : (threads > 512 ? 512 : threads);
-  if constexpr (CL == 1) {
-    return launch_pdl(resid_step_kernel<T, CL>, dim3(a.rows), dim3(threads), smem, st, a);
-  } else {
-    return launch_pdl_cluster(resid_step_kernel<T, CL>, dim3(a.rows * CL), dim3(threads), CL, smem, st, a);
-  }
+  const int pieces = ((a.W + CL - 1) / CL + 3) / 4;
+  const auto width = [&](int ni) { return ((pieces + ni - 1) / ni + 31) / 32 * 32; };
+  if (width(1) <= 256) return launch_resid_ni<T, CL, 1>(a, width(1), st);
+  if (width(2) <= 256) return launch_resid_ni<T, CL, 2>(a, width(2), st);
+  if (width(4) <= 256) return launch_resid_ni<T, CL, 4>(a, width(4), st);
+  if (width(8) <= 1024) return launch_resid_ni<T, CL, 8>(a, width(8), st);
+  return cudaErrorInvalidValue;
 }
 
 }  // namespace ds41
 
 using namespace ds41;
-
-static bool proj_ok(const ds41_proj& p) {
-  return p.data != nullptr && p.ld > 0 && p.splits >= 1 && p.col >= 0 && (p.splits == 1 || (p.plane > 0 && !p.bf16));
-}
 
 extern "C" int ds41_resid_step(const ds41_resid_args* a, void* stream) {
   if (a == nullptr || a->rows <= 0 || a->W <= 0 || a->ldx < a->W) return cudaErrorInvalidValue;
@@ -235,7 +297,11 @@ extern "C" int ds41_resid_step(const ds41_resid_args* a, void* stream) {
   if (a->y.data != nullptr && !proj_ok(a->y)) return cudaErrorInvalidValue;
   if (a->gate.data != nullptr && (!proj_ok(a->gate) || a->gate_bias == nullptr)) return cudaErrorInvalidValue;
   if (a->mix != nullptr && (a->n_mix < 1 || (a->n_mix > 1 && a->kept == nullptr))) return cudaErrorInvalidValue;
-  if (a->next_w != nullptr && (a->h == nullptr || a->ldh < a->W)) return cudaErrorInvalidValue;
+  if (a->next_w != nullptr && (a->h == nullptr || a->ldh < a->W || (a->ldh & 3))) return cudaErrorInvalidValue;
+  // rows are walked in pieces of four columns
+  if ((a->ldx & 3) || (a->kept_stride & 3) || (a->tokens != nullptr && (a->embed_ld & 3)) ||
+      (a->y.data != nullptr && !proj_vec4(a->y)) || (a->gate.data != nullptr && !proj_vec4(a->gate)))
+    return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // few rows: a cluster of eight CTAs shares a row, so that its loads do not queue on one SM
   const bool wide = a->rows <= 32 && a->W >= 1024;
@@ -246,7 +312,7 @@ extern "C" int ds41_resid_step(const ds41_resid_args* a, void* stream) {
 template <typename T>
 static int launch_polynorm(const ds41_proj& z, const float* coef, int rows, int ff, int ld_out, float eps, void* out,
                            cudaStream_t st) {
-  const size_t smem = 1ull * ff * sizeof(float);
+  const size_t smem = (1ull * ff + 3) / 4 * 16;
   static size_t allowed = 48 * 1024 - 512;
   if (smem > allowed) {
     if (smem > 226 * 1024) return cudaErrorInvalidValue;
@@ -261,7 +327,8 @@ static int launch_polynorm(const ds41_proj& z, const float* coef, int rows, int 
 
 extern "C" int ds41_polynorm(const ds41_proj* z, const float* coef, int rows, int ff, float eps, void* out, int ld_out,
                              int f32, void* stream) {
-  if (z == nullptr || !proj_ok(*z) || coef == nullptr || out == nullptr || rows <= 0 || ff <= 0 || ld_out < ff)
+  if (z == nullptr || !proj_ok(*z) || !proj_vec4(*z) || coef == nullptr || out == nullptr || rows <= 0 || ff <= 0 ||
+      ld_out < ff || (ld_out & 3) || z->ld < z->col + (ff + 3) / 4 * 4)
     return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return f32 ? launch_polynorm<float>(*z, coef, rows, ff, ld_out, eps, out, st)

@@ -279,6 +279,7 @@ class MLSTM:
         a.state_s, a.state_n, a.state_m, a.out = s.data_ptr(), n.data_ptr(), m.data_ptr(), e.o_heads.data_ptr()
         a.gate_cap, a.q_scale, a.den_eps = sp.gate_cap, sp.dim ** -0.5, sp.den_eps
         a.rows, a.heads, a.dim_pad, a.vdim_pad, a.slots, a.ld_out = R, H, self.dp, self.vp, e.cache.slots, ld
+        a.work = e.recurrence_work.data_ptr()
         if long:
             e._run("mlstm_chunk", k.ds41_mlstm_chunk, C.byref(a), lib.stream())
         else:
@@ -430,6 +431,8 @@ class StackEngine(RowsEngine):
         wide = max(S.ceil_to(n, 8) for lw in weights.layers for m in (lw.mixer, lw.mlp) if m is not None
                    for n, _ in m.matrices()["a"])
         self.wide = z((R * wide if R >= self.long_rows and not self.f32 else 8,), BF16)
+        heads_rec = max([lw.mixer.spec.heads for lw in weights.layers if isinstance(lw.mixer, MLSTM)], default=0)
+        self.recurrence_work = z((S.mlstm_chunk_work(R, heads_rec) // 4 + 4,), F32)
         self._keys = [z((8,), BF16) for _ in range(3)]
         self.act = z((R * max(act, heads),), dt)
         self.o_heads = z((R * heads,), F32)
@@ -454,7 +457,7 @@ class StackEngine(RowsEngine):
     def attn_splits(self, rows: int, heads: int) -> int:
         """Key splits per row of the absorbed attention: enough blocks to fill the GPU about twice, static per batch
         size (a captured pass replays while the context grows)."""
-        want = -(-2 * 148 // (rows * -(-heads // 16)))
+        want = 2 * 148 // (rows * -(-heads // 32))
         return max(1, min(want, 32, -(-self.cache.max_ctx // 64)))
 
     def project(self, tag: str, x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor) -> Proj:

@@ -61,8 +61,15 @@ class MlstmArgs(C.Structure):
     _fields_ = [("q", ProjArgs), ("k", ProjArgs), ("v", ProjArgs), ("gate_i", ProjArgs), ("gate_f", ProjArgs),
                 ("bias_i", C.c_void_p), ("bias_f", C.c_void_p), ("row_pos", C.c_void_p), ("row_slot", C.c_void_p),
                 ("state_s", C.c_void_p), ("state_n", C.c_void_p), ("state_m", C.c_void_p), ("out", C.c_void_p),
-                ("gate_cap", C.c_float), ("q_scale", C.c_float), ("den_eps", C.c_float), ("rows", C.c_int),
+                ("work", C.c_void_p), ("gate_cap", C.c_float), ("q_scale", C.c_float), ("den_eps", C.c_float), ("rows", C.c_int),
                 ("heads", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int), ("slots", C.c_int), ("ld_out", C.c_int)]
+
+
+def mlstm_chunk_work(rows: int, heads: int) -> int:
+    """Bytes of workspace of the chunked recurrence."""
+    fn = lib.kernels().ds41_mlstm_chunk_work
+    fn.restype = C.c_longlong
+    return fn(rows, heads)
 
 
 STATE_COLS = 32       # value columns per state block of the mLSTM kernels (kStateCols)

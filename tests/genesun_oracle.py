@@ -246,7 +246,7 @@ YARN = dict(factor=5.0, original=96, fast=8.0, slow=1.0)
 
 MODELS = {
     # widths that are no multiple of the tile sizes, shared cache rows over several layers, feed-forward after a recurrence
-    "odd": make_doc(88, 131, [
+    "odd": make_doc(90, 131, [
         ("latent_attention", attention_mixer(3, 20, 6, 24, 56, 40, scaling=YARN), 100),
         ("mlstm", dict(heads=3, dim=24, vdim=40, gate_cap=7.0), 60),
         ("latent_attention", attention_mixer(5, 12, 6, 36, 40, 40, scale=0.3, base=500.0, kv_from=0), None),

@@ -158,7 +158,7 @@ def test_a_planted_mistake_shows_in_the_logits():
     assert moved(change_w=lambda x: x.update({"l0.mix.sink": torch.full((3,), -100.0)})) > 5e-3
     assert moved(change_w=lambda x: x.update({"l2.dwa": torch.tensor([0.0, 0.0, 0.0, 1.0])})) > 5e-3
     assert moved(change_w=lambda x: x.update({"l0.mlp.act": w["l0.mlp.act"] * torch.tensor([1.0, 1.0, 0.0, 1.0])})) > 5e-3
-    assert moved(change_w=lambda x: x.update({"l1.rg1.b": torch.zeros(88)})) > 5e-3
+    assert moved(change_w=lambda x: x.update({"l1.rg1.b": torch.zeros(90)})) > 5e-3
     assert moved(lambda d: d["layers"][0]["mixer"]["rot"].pop("scaling")) > 5e-3
     assert moved(lambda d: d["layers"][1]["mixer"].update(gate_cap=70.0)) > 5e-3
     assert moved(lambda d: d["layers"][3]["mixer"].update(scale=0.1)) > 5e-3

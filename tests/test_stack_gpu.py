@@ -68,7 +68,7 @@ def feed(e, slot, toks, start, sizes):
 def limit(dtype, spread):
     """Allowed difference at a position whose bf16 rounding spread is known: a floor plus a multiple of what rounding does
     there (a 32-bit pass rounds 2^16 times finer; the factor leaves room for sums over many terms)."""
-    return 2e-5 + 2e-4 * spread if dtype == "f32" else 0.03 + 3 * spread
+    return 2e-5 + 4e-4 * spread if dtype == "f32" else 0.03 + 3 * spread
 
 
 def close(got, want, dtype, spread):
@@ -303,7 +303,8 @@ def _ok(err):
     assert err == 0, f"cudaError {err}"
 
 
-@pytest.mark.parametrize("rows,W,kind", [(3, 52, 0), (33, 1032, 0), (5, 1032, 1), (2, 4096, 0)])
+@pytest.mark.parametrize("rows,W,kind", [(3, 52, 0), (4, 90, 0), (33, 1032, 0), (5, 1032, 1), (3, 1501, 0), (2, 4096, 0),
+                                         (40, 4096, 0), (40, 9000, 1)])
 def test_residual_step(rows, W, kind):
     lib, S, k = _stack()
     g = gen(W)
@@ -314,41 +315,51 @@ def test_residual_step(rows, W, kind):
     d = lambda t: t.double()
     full = d(x) + norm(d(y).sum(0) * torch.sigmoid(d(gt).sum(0) + d(b)), d(pw), eps)
     avg = sum(m * t for m, t in zip(d(mix), [*d(kept), full]))
-    cu = lambda t: t.contiguous().cuda()
-    Y, GT, B, PW, NW, X, KEPT, MIX = map(cu, (y, gt, b, pw, nw, x, kept, mix))
-    out, x_avg, h = torch.zeros(rows, W).cuda(), torch.zeros(rows, W).cuda(), torch.zeros(rows, W).cuda()
+    L = S.ceil_to(W, 8)
+
+    def wide(t):                    # rows padded with values that must not count
+        o = torch.full(t.shape[:-1] + (L,), float("nan"), device="cuda")
+        o[..., :W] = t.cuda()
+        return o
+
+    Y, GT, X, KEPT = map(wide, (y, gt, x, kept))
+    B, PW, NW, MIX = (t.cuda() for t in (b, pw, nw, mix))
+    out, x_avg, h = (torch.zeros(rows, L).cuda() for _ in range(3))
     a = S.ResidArgs()
-    a.y, a.gate = S.Proj(Y, W, 2, rows * W).args(), S.Proj(GT, W, 2, rows * W).args()
+    a.y, a.gate = S.Proj(Y, L, 2, rows * L).args(), S.Proj(GT, L, 2, rows * L).args()
     a.gate_bias, a.post_w, a.next_w, a.x_in, a.x_out = (lib.ptr(t) for t in (B, PW, NW, X, out))
-    a.mix, a.kept, a.kept_stride, a.n_mix, a.x_avg = lib.ptr(MIX), lib.ptr(KEPT), rows * W, 4, lib.ptr(x_avg)
-    a.h, a.ldh, a.ldx, a.rows, a.W, a.norm_kind, a.eps, a.f32 = lib.ptr(h), W, W, rows, W, kind, eps, 1
+    a.mix, a.kept, a.kept_stride, a.n_mix, a.x_avg = lib.ptr(MIX), lib.ptr(KEPT), rows * L, 4, lib.ptr(x_avg)
+    a.h, a.ldh, a.ldx, a.rows, a.W, a.norm_kind, a.eps, a.f32 = lib.ptr(h), L, L, rows, W, kind, eps, 1
     _ok(k.ds41_resid_step(C.byref(a), lib.stream()))
-    torch.testing.assert_close(out.cpu().double(), full, rtol=2e-5, atol=2e-5)
-    torch.testing.assert_close(x_avg.cpu().double(), avg, rtol=2e-5, atol=2e-5)
-    torch.testing.assert_close(h.cpu().double(), norm(avg, d(nw), eps), rtol=2e-5, atol=5e-5)
+    torch.testing.assert_close(out[:, :W].cpu().double(), full, rtol=2e-5, atol=2e-5)
+    torch.testing.assert_close(x_avg[:, :W].cpu().double(), avg, rtol=2e-5, atol=2e-5)
+    torch.testing.assert_close(h[:, :W].cpu().double(), norm(avg, d(nw), eps), rtol=2e-5, atol=5e-5)
     # start from the embedding, bf16 output
     E = r(17, W).to(BF16)
     toks = torch.randint(0, 17, (rows,), generator=g)
     a = S.ResidArgs()
     a.y = a.gate = S.NO_PROJ
-    te, tt, hb = E.cuda(), toks.int().cuda(), torch.zeros(rows, W, dtype=BF16).cuda()
-    a.tokens, a.embed, a.embed_ld, a.vocab, a.x_out, a.next_w = lib.ptr(tt), lib.ptr(te), W, 17, lib.ptr(out), lib.ptr(NW)
-    a.h, a.ldh, a.ldx, a.rows, a.W, a.norm_kind, a.eps = lib.ptr(hb), W, W, rows, W, kind, eps
+    te, tt, hb = wide(E).to(BF16), toks.int().cuda(), torch.zeros(rows, L, dtype=BF16).cuda()
+    a.tokens, a.embed, a.embed_ld, a.vocab, a.x_out, a.next_w = lib.ptr(tt), lib.ptr(te), L, 17, lib.ptr(out), lib.ptr(NW)
+    a.h, a.ldh, a.ldx, a.rows, a.W, a.norm_kind, a.eps = lib.ptr(hb), L, L, rows, W, kind, eps
     _ok(k.ds41_resid_step(C.byref(a), lib.stream()))
-    assert torch.equal(out.cpu(), E[toks].float())
-    torch.testing.assert_close(hb.cpu().double(), norm(d(E[toks]), d(nw), eps), rtol=1e-2, atol=1e-2)
+    assert torch.equal(out[:, :W].cpu(), E[toks].float())
+    torch.testing.assert_close(hb[:, :W].cpu().double(), norm(d(E[toks]), d(nw), eps), rtol=1e-2, atol=1e-2)
 
 
 @pytest.mark.parametrize("ff", [37, 640, 5000])
 def test_polynorm_and_gates(ff):
     lib, S, k = _stack()
     g = gen(ff)
-    z, coef = torch.randn(2, 4, ff, generator=g), torch.tensor([0.7, -0.4, 0.3, 0.2])
-    out = torch.zeros(4, ff).cuda()
-    Z, Cf = z.cuda(), coef.cuda()
-    _ok(k.ds41_polynorm(C.byref(S.Proj(Z, ff, 2, 4 * ff).args()), lib.ptr(Cf), 4, ff, C.c_float(1e-5), lib.ptr(out), ff, 1,
+    z, coef, ld = torch.randn(2, 4, ff, generator=g), torch.tensor([0.7, -0.4, 0.3, 0.2]), S.ceil_to(ff, 8)
+    out = torch.zeros(4, ld).cuda()
+    Z, Cf = torch.full((2, 4, ld), float("nan")).cuda(), coef.cuda()        # what lies beyond the row does not count
+    Z[..., :ff] = z.cuda()
+    _ok(k.ds41_polynorm(C.byref(S.Proj(Z, ld, 2, 4 * ld).args()), lib.ptr(Cf), 4, ff, C.c_float(1e-5), lib.ptr(out), ld, 1,
                         lib.stream()))
-    torch.testing.assert_close(out.cpu().double(), polynorm(z.double().sum(0), coef.double(), 1e-5), rtol=3e-5, atol=3e-5)
+    torch.testing.assert_close(out[:, :ff].cpu().double(), polynorm(z.double().sum(0), coef.double(), 1e-5), rtol=3e-5,
+                               atol=3e-5)
+    Z, out = z.cuda(), torch.zeros(4, ff).cuda()
     _ok(k.ds41_gate_mul(C.byref(S.Proj(Z[0], ff).args()), C.byref(S.Proj(Z[1], ff).args()), 4, ff, lib.ptr(out), ff, 1,
                         lib.stream()))
     torch.testing.assert_close(out.cpu(), z[0] * torch.sigmoid(z[1]), rtol=1e-5, atol=1e-6)
@@ -556,6 +567,7 @@ class Recurrence:
         x = torch.cat([q, kk, v], 1).to(dtype).cuda()
         gates = torch.cat([self.i, self.f], 1).float().cuda()
         bi, bf = self.bi.float().cuda(), self.bf.float().cuda()
+        work = torch.zeros(S.mlstm_chunk_work(self.T, self.H) // 4).cuda()
         outs, at, n_call = [], 0, 0
         while at < self.T:
             n = min(sizes[min(n_call, len(sizes) - 1)], self.T - at)
@@ -566,7 +578,7 @@ class Recurrence:
             a = S.MlstmArgs()
             a.q, a.k, a.v = px.args(), px.at(self.H * dp).args(), px.at(2 * self.H * dp).args()
             a.gate_i, a.gate_f, a.bias_i, a.bias_f = pg.args(), pg.at(self.H).args(), lib.ptr(bi), lib.ptr(bf)
-            a.row_pos, a.row_slot, a.out = lib.ptr(pos), lib.ptr(sl), lib.ptr(out)
+            a.row_pos, a.row_slot, a.out, a.work = lib.ptr(pos), lib.ptr(sl), lib.ptr(out), lib.ptr(work)
             a.state_s, a.state_n, a.state_m = (lib.ptr(t) for t in st)
             a.gate_cap, a.q_scale, a.den_eps = self.cap, self.D ** -0.5, 1e-6
             a.rows, a.heads, a.dim_pad, a.vdim_pad, a.slots, a.ld_out = n, self.H, dp, vp, slots, self.H * vp
@@ -580,7 +592,7 @@ class Recurrence:
         return torch.cat(outs)
 
 
-@pytest.mark.parametrize("shape", [(2, 24, 40), (1, 16, 16), (3, 64, 96)])
+@pytest.mark.parametrize("shape", [(2, 24, 40), (1, 16, 16), (3, 64, 96), (1, 100, 32), (1, 200, 64), (1, 400, 16), (1, 600, 48)])
 @pytest.mark.parametrize("sizes", [[300], [1], [2, 65, 1, 63]])
 def test_recurrence_token_by_token(shape, sizes):
     c = Recurrence(150, *shape, seed=shape[1])
