@@ -18,6 +18,7 @@ snapshot, 1024 output tokens, paged FP8 KV rows; 5 = speculative C1 decode over 
 vocabulary mask on the target's choices.
 
   python bench.py --gpus N --steps K --warmup W          (N > 1: launched by torch.distributed.run)
+  python bench.py --stack genesun-1b,genesun-7b          (layer-stack models beside ds41 models of equal size; one GPU)
   python bench.py --impl reference ...                   (prints the reference arm's availability line)
 
 Prints ONE JSON line on rank 0.  `value` is device-timed (CUDA events on the launching stream, barrier and
@@ -387,6 +388,25 @@ def concurrent_bench(args, fabric, cfg, n_layers):
     return 0
 
 
+def stack_bench(args, fabric):
+    """Prompt and decode throughput of layer-stack presets beside ds41 models of equal size (utils/stack_bench.py): one
+    JSON line whose `value` is the first preset's prompt throughput and whose `models` hold every measurement."""
+    from ds41rt_b200.utils import stack_bench as sb
+    if fabric.world != 1:
+        raise SystemExit("--stack runs on one GPU")
+    names = args.stack.split(",")
+    sampler = ClockSampler(fabric.device.index or 0)
+    sampler.start()
+    rep = sb.run(names, fabric.device, args.steps, max(args.warmup, 3), args.prompt, args.chunk, args.layers, args.prompt)
+    clocks = sampler.stop()
+    first = next(iter(rep["models"].values()))
+    print(json.dumps({"metric": f"prefill tok/s ({names[0]}, {first['layers']} layers, prompt of {args.prompt} tokens)",
+                      "value": first["prefill"]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+                      "warmup": max(args.warmup, 3), "higher_is_better": True, "vs_baseline": None, "data": "synthetic",
+                      "dtype": "bf16 (fp32 streams, norms, scores and states)", "clocks": clocks, "impl": "ours", **rep}))
+    return 0
+
+
 PRESETS = {
     2: dict(no_spec=True, prompt=4096, steps=512),
     3: dict(mode="prefill", prompts=8, prompt=8192, chunk=8192, router_std=1.0, steps=2),
@@ -430,6 +450,8 @@ def main():
                     help="prefill: the decoder layers run over the last 128 prompt tokens only (the reference's prompt "
                          "scheme); default is every layer over every token")
     ap.add_argument("--ced-boundary", type=int, default=0, help="first decoder layer for --ced on a truncated stack")
+    ap.add_argument("--stack", default="", help="layer-stack presets (comma-separated, e.g. genesun-1b,genesun-7b): prompt "
+                    "and decode throughput beside ds41 models of equal size; --prompt, --chunk (default 2048), --layers")
     ap.add_argument("--breakdown", action="store_true", help="prefill: per-kernel device time of one prompt (stderr)")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -437,6 +459,8 @@ def main():
     defaults = dict(steps=64, prompt=4096, prompts=1, expert_dtype="mxfp8", prefill_chunk=32, no_spec=False,
                     mode="decode", chunk=1024, concurrency=1, kv_dtype="bf16", router_std=None, mask=False)
     defaults.update(PRESETS.get(args.config, {}))
+    if args.stack:
+        defaults.update(steps=32, chunk=2048)
     for key, val in defaults.items():
         if getattr(args, key) is None:
             setattr(args, key, val)
@@ -459,6 +483,8 @@ def main():
                   file=sys.stderr)
         return 2
     dev = fabric.device
+    if args.stack:
+        return stack_bench(args, fabric)
     if args.model == "flash":
         n_layers = args.layers or LAYERS_FOR_GPUS.get(world, LAYERS_FULL)
         cfg = ModelConfig.flash(n_layers)

@@ -33,6 +33,47 @@ __device__ __forceinline__ T* cache_row(T* pool, const int* page_table, int max_
   return pool + (1ll * id * page_tokens + (pos - pg * page_tokens)) * row_len;
 }
 
+// RMS norm of `n` columns of a projection row into `out` (columns up to the next multiple of four are written as zeros).
+// The row stays in registers while it is short (kHeld pieces per thread).
+template <typename T>
+__device__ __forceinline__ void norm_row(const ds41_proj& p, int r, int n, const float* w, float eps, T* out, float* red) {
+  constexpr int kHeld = 2;
+  float4 held[kHeld], wh[kHeld];
+  float q = 0.f;
+  int c = 0;
+  for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x, ++c) {
+    float4 v = proj_at4(p, r, i);
+    if (i + 1 >= n) v.y = 0.f;
+    if (i + 2 >= n) v.z = 0.f;
+    if (i + 3 >= n) v.w = 0.f;
+#pragma unroll
+    for (int k = 0; k < kHeld; ++k)
+      if (c == k) {
+        held[k] = v;
+        wh[k] = load4(w + i, n - i);
+      }
+    q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  const float s = 1.0f / sqrtf(block_sum(q, red) / n + eps);
+  c = 0;
+  for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x, ++c) {
+    float4 v, g;
+    if (c < kHeld) {
+#pragma unroll
+      for (int k = 0; k < kHeld; ++k)
+        if (c == k) {
+          v = held[k];
+          g = wh[k];
+        }
+    } else {
+      v = proj_at4(p, r, i);
+      g = load4(w + i, n - i);
+    }
+    store4(out + i, make_float4(v.x * s * g.x, i + 1 < n ? v.y * s * g.y : 0.f, i + 2 < n ? v.z * s * g.z : 0.f,
+                                i + 3 < n ? v.w * s * g.w : 0.f));
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_post_kernel(ds41_latent_post_args p) {
   __shared__ float red[33];
@@ -40,56 +81,56 @@ __global__ void __launch_bounds__(256) latent_post_kernel(ds41_latent_post_args 
   pdl_launch_dependents();
   pdl_wait();
   if (blockIdx.y == 0) {
-    float q = 0.f;
-    for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
-      const float v = proj_at(p.dq, r, i);
-      q += v * v;
-    }
-    const float s = 1.0f / sqrtf(block_sum(q, red) / p.q_rank + p.eps);
-    T* out = static_cast<T*>(p.cq) + 1ll * r * p.ld_cq;
-    for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) out[i] = from_f32<T>(proj_at(p.dq, r, i) * s * p.dq_norm[i]);
+    norm_row(p.dq, r, p.q_rank, p.dq_norm, p.eps, static_cast<T*>(p.cq) + 1ll * r * p.ld_cq, red);
     return;
   }
   const int slot = p.row_slot[r], pos = p.row_pos[r];
   if (slot < 0) return;
   T* row = cache_row(static_cast<T*>(p.pool), p.page_table, p.max_pages, p.page_tokens, p.row_len, slot, pos);
   if (row == nullptr) return;
-  float q = 0.f;
-  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) {
-    const float v = proj_at(p.kv, r, i);
-    q += v * v;
-  }
-  const float s = 1.0f / sqrtf(block_sum(q, red) / p.kv_rank + p.eps);
-  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) row[i] = from_f32<T>(proj_at(p.kv, r, i) * s * p.kv_norm[i]);
   for (int i = threadIdx.x; i < p.rot_dim / 2; i += blockDim.x) {
     float a, b;
     rotate_pair(proj_at(p.kr, r, 2 * i), proj_at(p.kr, r, 2 * i + 1), pos, p.freq[i], p.magnitude, a, b);
     row[p.kv_pad + 2 * i] = from_f32<T>(a);
     row[p.kv_pad + 2 * i + 1] = from_f32<T>(b);
   }
+  norm_row(p.kv, r, p.kv_rank, p.kv_norm, p.eps, row, red);
 }
 
-// In place when q is the projection itself (q.data == out): then only the rotated parts change.
+// In place when q is the projection itself (q.data == out): then only the rotated parts change.  A block's heads share the
+// sines and cosines of its row.
+constexpr int kMaxTurns = 256;         // pairs whose sine and cosine are kept per block
 template <typename T>
 __global__ void __launch_bounds__(256) latent_query_kernel(ds41_proj q, const int* row_pos, const float* freq,
                                                            float magnitude, int heads, int dim_pad, int rot_pad,
                                                            int rot_dim, T* out, int ld_out, int in_place) {
+  __shared__ float2 turn[kMaxTurns];
   const int r = blockIdx.y;
   pdl_launch_dependents();
   pdl_wait();
+  const int pos = row_pos[r];
+  for (int i = threadIdx.x; i < rot_dim / 2; i += blockDim.x) {
+    float s, c;
+    sincosf(static_cast<float>(pos) * freq[i], &s, &c);
+    turn[i] = make_float2(c * magnitude, s * magnitude);
+  }
+  __syncthreads();
   const int hs = dim_pad + rot_pad;
   const int half = in_place ? rot_pad / 2 : hs / 2;
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= heads * half) return;
-  const int h = i / half, j = 2 * (i - h * half) + (in_place ? dim_pad : 0), c = h * hs + j;
-  float a = proj_at(q, r, c), b = proj_at(q, r, c + 1);
-  const int t = j - dim_pad;
-  if (t >= 0 && t < rot_dim) {
-    const float u = a, v = b;
-    rotate_pair(u, v, row_pos[r], freq[t / 2], magnitude, a, b);
+  const int first = in_place ? dim_pad : 0;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < heads * half; i += gridDim.x * blockDim.x) {
+    const int h = i / half, j = 2 * (i - h * half) + first, c = h * hs + j;
+    float a = proj_at(q, r, c), b = proj_at(q, r, c + 1);
+    const int t = j - dim_pad;
+    if (t >= 0 && t < rot_dim) {
+      const float2 cs = turn[t / 2];
+      const float u = a, v = b;
+      a = u * cs.x - v * cs.y;
+      b = v * cs.x + u * cs.y;
+    }
+    out[1ll * r * ld_out + c] = from_f32<T>(a);
+    out[1ll * r * ld_out + c + 1] = from_f32<T>(b);
   }
-  out[1ll * r * ld_out + c] = from_f32<T>(a);
-  out[1ll * r * ld_out + c + 1] = from_f32<T>(b);
 }
 
 template <typename T>
@@ -421,28 +462,43 @@ static int attend_mma_heads(const ds41_latent_attend_args& a) {
   return fits(1) ? 16 : 0;
 }
 
+// one block per (head, row): the splits' weights first, then every thread sums four columns over the splits
+constexpr int kMaxSplits = 256;
 template <typename T>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* part_o, const float* part_ml, const float* sink,
                                                            int n_splits, int heads, int kv_pad, T* out, int ld_out) {
+  __shared__ float wt[kMaxSplits];
+  __shared__ float red[33];
   const int h = blockIdx.x, r = blockIdx.y;
   pdl_launch_dependents();
   pdl_wait();
   const long long cell0 = 1ll * r * n_splits * heads + h;
-  float m = sink != nullptr ? sink[h] : -INFINITY;
+  const float sk = sink != nullptr ? sink[h] : -INFINITY;
+  float m = sk;
   for (int s = 0; s < n_splits; ++s) m = fmaxf(m, part_ml[2 * (cell0 + 1ll * s * heads)]);
-  float den = sink != nullptr ? expf(sink[h] - m) : 0.f;
-  for (int s = 0; s < n_splits; ++s) {
-    const float* ml = part_ml + 2 * (cell0 + 1ll * s * heads);
-    if (ml[1] > 0.f) den += ml[1] * expf(ml[0] - m);
+  float den = 0.f;
+  for (int s = threadIdx.x; s < n_splits; s += blockDim.x) {
+    const float2 ml = *reinterpret_cast<const float2*>(part_ml + 2 * (cell0 + 1ll * s * heads));
+    const float e = ml.y > 0.f ? expf(ml.x - m) : 0.f;
+    wt[s] = e;
+    den += e * ml.y;
   }
+  den = block_sum(den, red) + (sink != nullptr ? expf(sk - m) : 0.f);
   const float inv = den > 0.f ? 1.0f / den : 0.f;
-  for (int i = threadIdx.x; i < kv_pad; i += blockDim.x) {
-    float a = 0.f;
+  for (int i = 4 * threadIdx.x; i < kv_pad; i += 4 * blockDim.x) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < n_splits; ++s) {
-      const long long c = cell0 + 1ll * s * heads;
-      if (part_ml[2 * c + 1] > 0.f) a += part_o[c * kv_pad + i] * expf(part_ml[2 * c] - m);
+      const float e = wt[s];
+      if (e > 0.f) {
+        const float4 o = *reinterpret_cast<const float4*>(part_o + (cell0 + 1ll * s * heads) * kv_pad + i);
+        a.x += e * o.x;
+        a.y += e * o.y;
+        a.z += e * o.z;
+        a.w += e * o.w;
+      }
     }
-    out[1ll * r * ld_out + h * kv_pad + i] = from_f32<T>(a * inv);
+    store4(out + 1ll * r * ld_out + h * kv_pad + i, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
   }
 }
 
@@ -455,6 +511,9 @@ extern "C" int ds41_latent_post(const ds41_latent_post_args* a, void* stream) {
       a->ld_cq < a->q_rank)
     return cudaErrorInvalidValue;
   const bool kv = a->pool != nullptr;       // a layer that reads another layer's rows writes none
+  if (!proj_vec4(a->dq) || (a->ld_cq & 3) || a->ld_cq < (a->q_rank + 3) / 4 * 4 ||
+      (kv && (!proj_vec4(a->kv) || (a->row_len & 3) || a->kv_pad < (a->kv_rank + 3) / 4 * 4)))
+    return cudaErrorInvalidValue;
   if (kv && (!proj_ok(a->kv) || !proj_ok(a->kr) || a->kv_norm == nullptr || a->freq == nullptr || a->kv_rank <= 0 ||
              a->kv_pad < a->kv_rank || a->row_len < a->kv_pad + a->rot_dim || (a->rot_dim & 1) || a->page_tokens <= 0 ||
              a->max_pages <= 0 || a->page_table == nullptr || a->row_pos == nullptr || a->row_slot == nullptr))
@@ -469,14 +528,16 @@ extern "C" int ds41_latent_query(const ds41_proj* q, const int* row_pos, const f
                                  int heads, int dim_pad, int rot_pad, int rot_dim, void* out, int ld_out, int f32,
                                  void* stream) {
   if (q == nullptr || !proj_ok(*q) || row_pos == nullptr || freq == nullptr || rows <= 0 || rows > 65535 || heads <= 0 ||
-      dim_pad < 0 || (dim_pad & 1) || (rot_pad & 1) || (rot_dim & 1) || rot_dim > rot_pad || out == nullptr ||
+      dim_pad < 0 || (dim_pad & 1) || (rot_pad & 1) || (rot_dim & 1) || rot_dim > rot_pad || rot_dim > 2 * kMaxTurns || out == nullptr ||
       ld_out < heads * (dim_pad + rot_pad))
     return cudaErrorInvalidValue;
   const int in_place = q->data == out ? 1 : 0;
   if (in_place && ((f32 != 0) == (q->bf16 != 0) || q->splits != 1 || q->col != 0 || q->ld != ld_out)) return cudaErrorInvalidValue;
   if (in_place && rot_pad == 0) return cudaSuccess;
   const int half = in_place ? rot_pad / 2 : (dim_pad + rot_pad) / 2;
-  const dim3 grid((heads * half + 255) / 256, rows);
+  int across = (heads * half + 255) / 256;
+  if (rows > 64 && across > 4) across = 4;          // long passes: fewer blocks per row, each turns more heads
+  const dim3 grid(across, rows);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32)
     return launch_pdl(latent_query_kernel<float>, grid, dim3(256), 0, st, *q, row_pos, freq, magnitude, heads, dim_pad,
@@ -522,7 +583,7 @@ extern "C" int ds41_latent_attend(const ds41_latent_attend_args* a, void* stream
 
 extern "C" int ds41_latent_merge(const float* part_o, const float* part_ml, const float* sink, int n_splits, int rows,
                                  int heads, int kv_pad, void* out, int ld_out, int f32, void* stream) {
-  if (part_o == nullptr || part_ml == nullptr || n_splits <= 0 || rows <= 0 || rows > 65535 || heads <= 0 ||
+  if (part_o == nullptr || part_ml == nullptr || n_splits <= 0 || n_splits > kMaxSplits || (kv_pad & 3) || rows <= 0 || rows > 65535 || heads <= 0 ||
       kv_pad <= 0 || out == nullptr || ld_out < heads * kv_pad)
     return cudaErrorInvalidValue;
   const dim3 grid(heads, rows);

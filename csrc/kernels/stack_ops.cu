@@ -15,66 +15,72 @@ namespace ds41 {
 
 namespace cg = cooperative_groups;
 
-// (mean, sum of squared deviations, count) of the part of a row that one CTA holds, merged over the CTAs of a cluster
+// (mean, sum of squared deviations, count) of a set of values
 struct Moments {
   float mean, m2, n;
 };
-
-template <int CL>
-__device__ __forceinline__ Moments merge_moments(Moments own, float* slot) {
-  if constexpr (CL == 1) {
-    return own;
-  } else {
-    cg::cluster_group cluster = cg::this_cluster();
-    if (threadIdx.x == 0) {
-      slot[0] = own.mean;
-      slot[1] = own.m2;
-      slot[2] = own.n;
-    }
-    cluster.sync();
-    Moments t{0.f, 0.f, 0.f};
+__device__ __forceinline__ Moments merge(Moments a, Moments b) {
+  const float n = a.n + b.n;
+  if (n == 0.f) return a;
+  const float d = b.mean - a.mean, f = b.n / n;
+  return {a.mean + d * f, a.m2 + b.m2 + d * d * (a.n * f), n};
+}
+__device__ __forceinline__ Moments merge_lanes(Moments v) {          // result in lane 0, then in every lane
 #pragma unroll
-    for (int c = 0; c < CL; ++c) {        // the same order in every CTA: all of them get the same numbers
-      const float* s = cluster.map_shared_rank(slot, c);
-      const float mean = s[0], m2 = s[1], n = s[2];
-      if (n == 0.f) continue;
-      const float total = t.n + n, d = mean - t.mean;
-      t.mean += d * (n / total);
-      t.m2 += m2 + d * d * (t.n * n / total);
-      t.n = total;
-    }
-    return t;
-  }
+  for (int o = 16; o; o >>= 1)
+    v = merge(v, {__shfl_down_sync(0xffffffffu, v.mean, o), __shfl_down_sync(0xffffffffu, v.m2, o),
+                  __shfl_down_sync(0xffffffffu, v.n, o)});
+  return {__shfl_sync(0xffffffffu, v.mean, 0), __shfl_sync(0xffffffffu, v.m2, 0), __shfl_sync(0xffffffffu, v.n, 0)};
 }
 
 // Subtrahend and factor of a row's norm - layer norm (subtract the mean) or RMS norm (mean of squares) - from the pieces of
 // four columns that the threads hold; `n` columns of the row are in this CTA, piece i covers columns 4 (tid + i blockDim).
+// Deviations are taken from each thread's own mean and merged pairwise, over the warp, the CTA and the cluster, in an order
+// that is the same in every thread.  `slot` holds 3 x 32 floats; at most 32 warps (4 per CTA of a cluster of 8).
 template <int CL, int NI>
-__device__ __forceinline__ float2 row_norm(const float4 (&v)[NI], int n, int W, int kind, float eps, float* red, float* slot) {
-  float mean = 0.f;
-  if (kind == 0) {
-    float s = 0.f;                       // columns beyond the row hold zeros
+__device__ __forceinline__ float2 row_norm(const float4 (&v)[NI], int n, int W, int kind, float eps, float* slot) {
+  float cnt = 0.f, s = 0.f;              // columns beyond the row hold zeros
 #pragma unroll
-    for (int i = 0; i < NI; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
-    mean = n > 0 ? block_sum(s, red) / n : 0.f;
+  for (int i = 0; i < NI; ++i) {
+    const int live = n - 4 * static_cast<int>(threadIdx.x + i * blockDim.x);
+    cnt += static_cast<float>(max(0, min(4, live)));
+    s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
   }
+  const float mean = kind == 0 && cnt > 0.f ? s / cnt : 0.f;         // an RMS norm merges with zero means
   float q = 0.f;
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
-    const int live = n - 4 * (threadIdx.x + i * blockDim.x);
+    const int live = n - 4 * static_cast<int>(threadIdx.x + i * blockDim.x);
     const float a = v[i].x - mean, b = v[i].y - mean, c = v[i].z - mean, d = v[i].w - mean;
     q += (live > 0 ? a * a : 0.f) + (live > 1 ? b * b : 0.f) + (live > 2 ? c * c : 0.f) + (live > 3 ? d * d : 0.f);
   }
-  q = block_sum(q, red);
-  // the means of squares add up: an RMS norm goes through the same exchange with zero means
-  const Moments t = merge_moments<CL>({mean, q, static_cast<float>(n)}, slot);
+  Moments t = merge_lanes({mean, q, cnt});
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  if (lane == 0) {
+    slot[warp] = t.mean;
+    slot[32 + warp] = t.m2;
+    slot[64 + warp] = t.n;
+  }
+  t = {0.f, 0.f, 0.f};
+  if constexpr (CL == 1) {
+    __syncthreads();
+    if (lane < n_warps) t = {slot[lane], slot[32 + lane], slot[64 + lane]};
+  } else {
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    if (lane < CL * n_warps) {
+      const float* far = cluster.map_shared_rank(slot, lane / n_warps);
+      const int w = lane % n_warps;
+      t = {far[w], far[32 + w], far[64 + w]};
+    }
+  }
+  t = merge_lanes(t);
   return make_float2(t.mean, 1.0f / sqrtf(t.m2 / W + eps));
 }
 
 template <typename T, int CL, int NI>
-__global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_kernel(ds41_resid_args p) {
-  __shared__ float red[33];
-  __shared__ float slots[2][3];
+__global__ void __launch_bounds__(CL == 8 ? 128 : (NI <= 4 ? 256 : 512)) resid_step_kernel(ds41_resid_args p) {
+  __shared__ float slots[2][96];
   const int per = ((p.W + CL - 1) / CL + 3) / 4 * 4;
   const int part = CL > 1 ? blockIdx.x % CL : 0;
   const int r = CL > 1 ? blockIdx.x / CL : blockIdx.x;
@@ -102,6 +108,32 @@ __global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_ke
     for (int i = 0; i < NI; ++i)
       if (live[i] > 0) x[i] = *reinterpret_cast<const float4*>(in + at[i]);
   }
+  // Few rows (clusters): what does not depend on the sublayer is loaded first - the weighted sum of the older kept streams,
+  // the norm weight - since the launch is a chain of latencies.  Many rows: the registers are worth more.
+  constexpr bool kEarly = CL > 1;
+  float4 older[NI], w_next[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    older[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (kEarly) w_next[i] = p.next_w != nullptr && live[i] > 0 ? load4(p.next_w + c0 + at[i], live[i]) : older[i];
+  }
+  auto add_older = [&]() {
+    const float* k0 = p.kept + r * p.ldx + c0;
+#pragma unroll 4
+    for (int j = 0; j < p.n_mix - 1; ++j) {
+      const float c = p.mix[j];
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+        if (live[i] > 0) {
+          const float4 k = *reinterpret_cast<const float4*>(k0 + j * p.kept_stride + at[i]);
+          older[i].x += c * k.x;
+          older[i].y += c * k.y;
+          older[i].z += c * k.z;
+          older[i].w += c * k.w;
+        }
+    }
+  };
+  if (kEarly && p.mix != nullptr) add_older();
   auto clip = [&](float4& v, int i) {         // columns beyond the row hold zeros
     if (live[i] < 4) v.w = 0.f;
     if (live[i] < 3) v.z = 0.f;
@@ -125,7 +157,7 @@ __global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_ke
       }
     }
     float2 s = make_float2(0.f, 1.f);
-    if (p.post_w != nullptr) s = row_norm<CL, NI>(y, n, p.W, p.norm_kind, p.eps, red, slots[0]);
+    if (p.post_w != nullptr) s = row_norm<CL, NI>(y, n, p.W, p.norm_kind, p.eps, slots[0]);
 #pragma unroll
     for (int i = 0; i < NI; ++i)
       if (live[i] > 0) {
@@ -145,31 +177,14 @@ __global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_ke
       if (live[i] > 0) store4(o + at[i], x[i]);
   }
   if (p.mix != nullptr) {
-    // weighted sum of the kept streams; the newest one is the row this block holds
-    const float* k0 = p.kept + r * p.ldx + c0;
-    const float last = p.mix[p.n_mix - 1];
+    if (!kEarly) add_older();
+    const float last = p.mix[p.n_mix - 1];    // the newest kept stream is the row this block holds
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      x[i].x *= last;
-      x[i].y *= last;
-      x[i].z *= last;
-      x[i].w *= last;
+      x[i] = make_float4(older[i].x + last * x[i].x, older[i].y + last * x[i].y, older[i].z + last * x[i].z,
+                         older[i].w + last * x[i].w);
+      clip(x[i], i);
     }
-#pragma unroll 4
-    for (int j = 0; j < p.n_mix - 1; ++j) {
-      const float c = p.mix[j];
-#pragma unroll
-      for (int i = 0; i < NI; ++i)
-        if (live[i] > 0) {
-          const float4 k = *reinterpret_cast<const float4*>(k0 + j * p.kept_stride + at[i]);
-          x[i].x += c * k.x;
-          x[i].y += c * k.y;
-          x[i].z += c * k.z;
-          x[i].w += c * k.w;
-        }
-    }
-#pragma unroll
-    for (int i = 0; i < NI; ++i) clip(x[i], i);
     if (p.x_avg != nullptr) {
       float* o = p.x_avg + r * p.ldx + c0;
 #pragma unroll
@@ -178,12 +193,12 @@ __global__ void __launch_bounds__(CL == 1 && NI <= 4 ? 256 : 1024) resid_step_ke
     }
   }
   if (p.next_w != nullptr) {
-    const float2 s = row_norm<CL, NI>(x, n, p.W, p.norm_kind, p.eps, red, slots[1]);
+    const float2 s = row_norm<CL, NI>(x, n, p.W, p.norm_kind, p.eps, slots[1]);
     T* h = static_cast<T*>(p.h) + 1ll * r * p.ldh + c0;
 #pragma unroll
     for (int i = 0; i < NI; ++i)
       if (live[i] > 0) {
-        const float4 w = load4(p.next_w + c0 + at[i], live[i]);
+        const float4 w = kEarly ? w_next[i] : load4(p.next_w + c0 + at[i], live[i]);
         store4(h + at[i], make_float4((x[i].x - s.x) * s.y * w.x, (x[i].y - s.x) * s.y * w.y, (x[i].z - s.x) * s.y * w.z,
                                       (x[i].w - s.x) * s.y * w.w));
       }
@@ -232,30 +247,87 @@ __global__ void __launch_bounds__(512) polynorm_kernel(ds41_proj z, const float*
 
 template <typename T>
 __global__ void __launch_bounds__(256) gate_mul_kernel(ds41_proj y, ds41_proj gate, int n, T* out, int ld_out) {
-  const int r = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
+  const int r = blockIdx.y, i = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
   pdl_launch_dependents();
   pdl_wait();
-  if (i < n) out[1ll * r * ld_out + i] = from_f32<T>(proj_at(y, r, i) * sigmoid_f32(proj_at(gate, r, i)));
+  if (i >= n) return;
+  const float4 v = proj_at4(y, r, i), g = proj_at4(gate, r, i);
+  store4(out + 1ll * r * ld_out + i, make_float4(v.x * sigmoid_f32(g.x), v.y * sigmoid_f32(g.y), v.z * sigmoid_f32(g.z),
+                                                 v.w * sigmoid_f32(g.w)));
 }
 
-// one warp per (row, head); columns [width, stride) of a head are padding and are written as zeros
+// one block per (row, head); columns [width, stride) of a head are padding and are written as zeros
 template <typename T>
-__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, int ld_o, ds41_proj gate, const float* w,
-                                                             int rows, int heads, int width, int stride, float eps,
-                                                             T* out, int ld_out) {
-  const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+__global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* o, int ld_o, ds41_proj gate, const float* w,
+                                                             int width, int stride, float eps, T* out, int ld_out) {
+  __shared__ float red[4];
+  const int h = blockIdx.x, r = blockIdx.y;
   pdl_launch_dependents();
   pdl_wait();
-  if (item >= rows * heads) return;
+  const float* src = o + 1ll * r * ld_o + h * stride;
+  T* dst = out + 1ll * r * ld_out + h * stride;
+  float q = 0.f;
+  float4 v0 = make_float4(0.f, 0.f, 0.f, 0.f), g0 = v0, w0 = v0;       // the thread's first piece stays in registers
+  for (int i = 4 * threadIdx.x; i < stride; i += 4 * blockDim.x) {
+    const float4 v = load4(src + i, width - i);
+    if (i < 4 * static_cast<int>(blockDim.x)) {
+      v0 = v;
+      g0 = proj_at4(gate, r, h * stride + i);
+      w0 = load4(w + h * stride + i, width - i);
+    }
+    q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  q = warp_sum(q);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = q;
+  __syncthreads();
+  q = 0.f;
+  for (int i = 0; i < static_cast<int>(blockDim.x >> 5); ++i) q += red[i];
+  const float s = 1.0f / sqrtf(q / width + eps);
+  for (int i = 4 * threadIdx.x; i < stride; i += 4 * blockDim.x) {
+    const bool first = i < 4 * static_cast<int>(blockDim.x);
+    const float4 v = first ? v0 : load4(src + i, width - i), ww = first ? w0 : load4(w + h * stride + i, width - i);
+    const float4 g = first ? g0 : proj_at4(gate, r, h * stride + i);
+    store4(dst + i, make_float4(i < width ? v.x * s * ww.x * sigmoid_f32(g.x) : 0.f,
+                                i + 1 < width ? v.y * s * ww.y * sigmoid_f32(g.y) : 0.f,
+                                i + 2 < width ? v.z * s * ww.z * sigmoid_f32(g.z) : 0.f,
+                                i + 3 < width ? v.w * s * ww.w * sigmoid_f32(g.w) : 0.f));
+  }
+}
+
+// many (row, head) pairs of at most 512 columns: one warp each
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_gate_warp_kernel(const float* o, int ld_o, ds41_proj gate, const float* w,
+                                                                  int items, int heads, int width, int stride, float eps,
+                                                                  T* out, int ld_out) {
+  const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  if (item >= items) return;
   const int r = item / heads, h = item - r * heads;
   const float* src = o + 1ll * r * ld_o + h * stride;
-  float q = 0.f;
-  for (int i = lane; i < width; i += 32) q += src[i] * src[i];
-  const float s = 1.0f / sqrtf(warp_sum(q) / width + eps);
   T* dst = out + 1ll * r * ld_out + h * stride;
-  for (int i = lane; i < stride; i += 32) {
-    const int c = h * stride + i;
-    dst[i] = i < width ? from_f32<T>(src[i] * s * w[c] * sigmoid_f32(proj_at(gate, r, c))) : from_f32<T>(0.f);
+  float4 v[4], g[4];
+  float q = 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    v[k] = g[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < stride) {
+      v[k] = load4(src + i, width - i);
+      g[k] = proj_at4(gate, r, h * stride + i);
+    }
+    q += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+  }
+  const float s = 1.0f / sqrtf(warp_sum(q) / width + eps);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    if (i >= stride) break;
+    const float4 ww = load4(w + h * stride + i, width - i);
+    store4(dst + i, make_float4(i < width ? v[k].x * s * ww.x * sigmoid_f32(g[k].x) : 0.f,
+                                i + 1 < width ? v[k].y * s * ww.y * sigmoid_f32(g[k].y) : 0.f,
+                                i + 2 < width ? v[k].z * s * ww.z * sigmoid_f32(g[k].z) : 0.f,
+                                i + 3 < width ? v[k].w * s * ww.w * sigmoid_f32(g[k].w) : 0.f));
   }
 }
 
@@ -279,10 +351,11 @@ template <typename T, int CL>
 static cudaError_t launch_resid(const ds41_resid_args& a, cudaStream_t st) {
   const int pieces = ((a.W + CL - 1) / CL + 3) / 4;
   const auto width = [&](int ni) { return ((pieces + ni - 1) / ni + 31) / 32 * 32; };
-  if (width(1) <= 256) return launch_resid_ni<T, CL, 1>(a, width(1), st);
-  if (width(2) <= 256) return launch_resid_ni<T, CL, 2>(a, width(2), st);
-  if (width(4) <= 256) return launch_resid_ni<T, CL, 4>(a, width(4), st);
-  if (width(8) <= 1024) return launch_resid_ni<T, CL, 8>(a, width(8), st);
+  constexpr int kMost = CL == 8 ? 128 : 256;        // the moments of a cluster's warps fit one warp
+  if (width(1) <= kMost) return launch_resid_ni<T, CL, 1>(a, width(1), st);
+  if (width(2) <= kMost) return launch_resid_ni<T, CL, 2>(a, width(2), st);
+  if (width(4) <= kMost) return launch_resid_ni<T, CL, 4>(a, width(4), st);
+  if (width(8) <= (CL == 8 ? 128 : 512)) return launch_resid_ni<T, CL, 8>(a, width(8), st);
   return cudaErrorInvalidValue;
 }
 
@@ -304,7 +377,7 @@ extern "C" int ds41_resid_step(const ds41_resid_args* a, void* stream) {
     return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // few rows: a cluster of eight CTAs shares a row, so that its loads do not queue on one SM
-  const bool wide = a->rows <= 32 && a->W >= 1024;
+  const bool wide = (a->rows <= 32 && a->W >= 1024) || a->W > 16384;
   if (a->f32) return wide ? launch_resid<float, 8>(*a, st) : launch_resid<float, 1>(*a, st);
   return wide ? launch_resid<__nv_bfloat16, 8>(*a, st) : launch_resid<__nv_bfloat16, 1>(*a, st);
 }
@@ -338,9 +411,9 @@ extern "C" int ds41_polynorm(const ds41_proj* z, const float* coef, int rows, in
 extern "C" int ds41_gate_mul(const ds41_proj* y, const ds41_proj* gate, int rows, int n, void* out, int ld_out, int f32,
                              void* stream) {
   if (y == nullptr || gate == nullptr || !proj_ok(*y) || !proj_ok(*gate) || out == nullptr || rows <= 0 || n <= 0 ||
-      ld_out < n || rows > 65535)
+      ld_out < n || rows > 65535 || (n & 3) || (ld_out & 3) || !proj_vec4(*y) || !proj_vec4(*gate))
     return cudaErrorInvalidValue;
-  const dim3 grid((n + 255) / 256, rows);
+  const dim3 grid((n + 1023) / 1024, rows);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (f32) return launch_pdl(gate_mul_kernel<float>, grid, dim3(256), 0, st, *y, *gate, n, static_cast<float*>(out), ld_out);
   return launch_pdl(gate_mul_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, *y, *gate, n,
@@ -350,15 +423,24 @@ extern "C" int ds41_gate_mul(const ds41_proj* y, const ds41_proj* gate, int rows
 extern "C" int ds41_head_norm_gate(const float* o, int ld_o, const ds41_proj* gate, const float* w, int rows, int heads,
                                    int width, int stride, float eps, void* out, int ld_out, int f32, void* stream) {
   if (o == nullptr || gate == nullptr || !proj_ok(*gate) || w == nullptr || out == nullptr || rows <= 0 || heads <= 0 ||
-      width <= 0 || stride < width || ld_o < heads * stride || ld_out < heads * stride)
+      width <= 0 || stride < width || (stride & 3) || ld_o < heads * stride || (ld_o & 3) || ld_out < heads * stride ||
+      (ld_out & 3) || !proj_vec4(*gate) || rows > 65535)
     return cudaErrorInvalidValue;
-  const dim3 grid((rows * heads + 7) / 8);
+  const dim3 grid(heads, rows), block(stride >= 512 ? 128 : (stride + 127) / 128 * 32);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (stride <= 512 && rows * heads >= 1024) {
+    const dim3 warps((rows * heads + 7) / 8);
+    if (f32)
+      return launch_pdl(head_norm_gate_warp_kernel<float>, warps, dim3(256), 0, st, o, ld_o, *gate, w, rows * heads, heads,
+                        width, stride, eps, static_cast<float*>(out), ld_out);
+    return launch_pdl(head_norm_gate_warp_kernel<__nv_bfloat16>, warps, dim3(256), 0, st, o, ld_o, *gate, w, rows * heads,
+                      heads, width, stride, eps, static_cast<__nv_bfloat16*>(out), ld_out);
+  }
   if (f32)
-    return launch_pdl(head_norm_gate_kernel<float>, grid, dim3(256), 0, st, o, ld_o, *gate, w, rows, heads, width, stride,
-                      eps, static_cast<float*>(out), ld_out);
-  return launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, ld_o, *gate, w, rows, heads, width,
-                    stride, eps, static_cast<__nv_bfloat16*>(out), ld_out);
+    return launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, st, o, ld_o, *gate, w, width, stride, eps,
+                      static_cast<float*>(out), ld_out);
+  return launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, st, o, ld_o, *gate, w, width, stride, eps,
+                    static_cast<__nv_bfloat16*>(out), ld_out);
 }
 
 extern "C" int ds41_gather_rows(const void* src, int ld, const int* index, int n_src, int rows, int W, void* dst, int f32,

@@ -304,7 +304,7 @@ def _ok(err):
 
 
 @pytest.mark.parametrize("rows,W,kind", [(3, 52, 0), (4, 90, 0), (33, 1032, 0), (5, 1032, 1), (3, 1501, 0), (2, 4096, 0),
-                                         (40, 4096, 0), (40, 9000, 1)])
+                                         (40, 4096, 0), (40, 9000, 1), (2, 20001, 0)])
 def test_residual_step(rows, W, kind):
     lib, S, k = _stack()
     g = gen(W)
@@ -359,20 +359,25 @@ def test_polynorm_and_gates(ff):
                         lib.stream()))
     torch.testing.assert_close(out[:, :ff].cpu().double(), polynorm(z.double().sum(0), coef.double(), 1e-5), rtol=3e-5,
                                atol=3e-5)
-    Z, out = z.cuda(), torch.zeros(4, ff).cuda()
-    _ok(k.ds41_gate_mul(C.byref(S.Proj(Z[0], ff).args()), C.byref(S.Proj(Z[1], ff).args()), 4, ff, lib.ptr(out), ff, 1,
+    n, out = ff // 4 * 4, torch.zeros(4, ld).cuda()
+    _ok(k.ds41_gate_mul(C.byref(S.Proj(Z[0], ld).args()), C.byref(S.Proj(Z[1], ld).args()), 4, n, lib.ptr(out), ld, 1,
                         lib.stream()))
-    torch.testing.assert_close(out.cpu(), z[0] * torch.sigmoid(z[1]), rtol=1e-5, atol=1e-6)
-    # heads padded from 5 to 8 columns; the padding comes out as zeros
-    o, gt, w = torch.randn(3, 16, generator=g), torch.randn(3, 16, generator=g), torch.randn(16, generator=g)
-    res = torch.full((3, 16), 9.0).cuda()
-    O, GT, Wn = o.cuda(), gt.cuda(), w.cuda()
-    _ok(k.ds41_head_norm_gate(lib.ptr(O), 16, C.byref(S.Proj(GT, 16).args()), lib.ptr(Wn), 3, 2, 5, 8, C.c_float(1e-6),
-                              lib.ptr(res), 16, 1, lib.stream()))
-    v = lambda t: t.view(-1, 2, 8)[..., :5]
-    want = torch.zeros(3, 2, 8)
-    want[..., :5] = rms_unit(v(o), 1e-6) * v(w) * torch.sigmoid(v(gt))
-    torch.testing.assert_close(res.cpu(), want.view(3, 16), rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(out[:, :n].cpu(), (z[0] * torch.sigmoid(z[1]))[:, :n], rtol=1e-5, atol=1e-6)
+
+
+@pytest.mark.parametrize("rows,heads,width,stride", [(3, 2, 5, 8), (4, 3, 130, 144), (2, 2, 700, 704), (300, 4, 500, 512)])
+def test_head_norm_with_padded_heads(rows, heads, width, stride):
+    """The padding counts for nothing and comes out as zeros."""
+    lib, S, k = _stack()
+    g = gen(rows)
+    o, gt, w = (torch.randn(*s, heads * stride, generator=g) for s in ((rows,), (rows,), ()))
+    O, GT, Wn, res = o.cuda(), gt.cuda(), w.cuda(), torch.full((rows, heads * stride), 9.0).cuda()
+    _ok(k.ds41_head_norm_gate(lib.ptr(O), heads * stride, C.byref(S.Proj(GT, heads * stride).args()), lib.ptr(Wn), rows, heads,
+                              width, stride, C.c_float(1e-6), lib.ptr(res), heads * stride, 1, lib.stream()))
+    v = lambda t: t.view(-1, heads, stride)[..., :width].double()
+    want = torch.zeros(rows, heads, stride, dtype=torch.float64)
+    want[..., :width] = rms_unit(v(o), 1e-6) * v(w) * torch.sigmoid(v(gt))
+    torch.testing.assert_close(res.cpu().double().view(rows, heads, stride), want, rtol=1e-5, atol=1e-5)
 
 
 @pytest.mark.parametrize("M,N,K", [(1, 7, 3), (70, 65, 130), (200, 10, 33)])
