@@ -551,7 +551,8 @@ def cmd_serve(args) -> int:
                             host_cache_bytes=int(args.host_cache_gb * (1 << 30)) if world == 1 else 0,
                             engram=_engram_pipeline(args, cfg, eng, engram_layers, tk), vision=tower)
     srv = ApiServer(backend, tk, host=args.host, port=args.port, queue_depth=args.queue_depth, waiters=args.waiters,
-                    max_context=args.max_context, vision_cfg=vision_cfg).start()
+                    max_context=args.max_context, vision_cfg=vision_cfg,
+                    **({} if fam.name == "ds41" else {"model_id": cfg.name})).start()
     print(json.dumps({"listening": f"http://{args.host}:{srv.port}", "model": cfg.name, "ranks": world,
                       "setup_s": round(time.time() - t0, 1), "kv_pool": plan.as_dict() | {"pages": n_pages},
                       "settings": {k: v for k, v in getattr(args, "_origin", {}).items() if v != "default"}}), flush=True)

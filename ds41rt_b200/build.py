@@ -87,6 +87,10 @@ def _kernel_recipe(verbose: bool = False):
     return sorted((CSRC / "kernels").glob("*.cu")), [nvcc] + flags
 
 
+# what a process that only runs layer-stack models needs of csrc/kernels
+STACK_KERNELS = ("gemm_f32", "gemm_tc", "latent_attn", "latent_prefill", "mlstm", "sampler", "sampler_rows", "stack_ops", "tma")
+
+
 def _core_recipe():
     cxx = shutil.which("g++") or "g++"
     return sorted((CSRC / "core").glob("*.cc")), [cxx] + CXX_FLAGS
@@ -95,6 +99,13 @@ def _core_recipe():
 def build_kernels(verbose: bool = False) -> Path:
     sources, cmd = _kernel_recipe(verbose)
     return _build_lib("libds41_kernels.so", sources, cmd,
+                      [cmd[0], "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"], verbose)
+
+
+def build_stack_kernels(verbose: bool = False) -> Path:
+    """The kernels of layer-stack models alone (objects are shared with the full library)."""
+    sources, cmd = _kernel_recipe(verbose)
+    return _build_lib("libds41_stack.so", [s for s in sources if s.stem in STACK_KERNELS], cmd,
                       [cmd[0], "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"], verbose)
 
 

@@ -385,7 +385,7 @@ class StackEngine(RowsEngine):
         self.rank, self.world = 0, 1
         self.max_rows = R = max_rows
         self.n_layers = cfg.n_layers
-        self.k = lib.kernels()
+        self.k = lib.kernels("stack")
         self.f32 = 1 if weights.dtype == "f32" else 0
         dev, dt = self.device, DTYPES[weights.dtype]
         self.cache = StackCache(cfg, slots, max_ctx, dev, dt, page_tokens, n_pages)

@@ -61,7 +61,7 @@ def gemm_raw(A, B, out, M, N, K, *, lda, ldb, ldo, kind=0, out_mode=0, k_splits=
     if signal is not None:          # (zeroed counter word, epoch word, device array of flag addresses, number of flags)
         a.sig_counter, a.sig_epoch, a.sig_flags, a.sig_world = (lib.ptr(signal[0]), lib.ptr(signal[1]),
                                                                 lib.ptr(signal[2]), signal[3])
-    lib.check(lib.kernels().ds41_gemm_tc(C.byref(a), lib.stream()), "ds41_gemm_tc")
+    lib.check(lib.kernels("any").ds41_gemm_tc(C.byref(a), lib.stream()), "ds41_gemm_tc")
 
 
 def matmul_nt(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, out_dtype=torch.bfloat16,

@@ -15,6 +15,7 @@ import torch
 
 _LIBDIR = Path(__file__).resolve().parent.parent / "_lib"
 _kernels = None
+_kernels_scope = ""
 _core = None
 
 
@@ -101,13 +102,17 @@ def _load(name: str, builder: str):
     return C.CDLL(str(path), mode=C.RTLD_GLOBAL)
 
 
-def kernels():
-    global _kernels
-    if _kernels is None:
-        lib = _load("libds41_kernels.so", "build_kernels")
+def kernels(scope: str = "all"):
+    """The kernel library.  `scope` names what the caller needs: "all", "stack" (the kernels of layer-stack models, enough
+    for a process that runs nothing else - a fresh checkout then compiles only those), or "any" (whatever is loaded)."""
+    global _kernels, _kernels_scope
+    if _kernels is None or (scope == "all" and _kernels_scope == "stack"):
+        small = scope == "stack" and not (_LIBDIR / "libds41_kernels.so").exists()
+        lib = _load("libds41_stack.so", "build_stack_kernels") if small else _load("libds41_kernels.so", "build_kernels")
         for fn in dir_functions():
-            getattr(lib, fn).restype = C.c_int
-        _kernels = lib
+            if not small or hasattr(lib, fn):
+                getattr(lib, fn).restype = C.c_int
+        _kernels, _kernels_scope = lib, "stack" if small else "all"
     return _kernels
 
 

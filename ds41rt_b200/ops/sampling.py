@@ -51,7 +51,7 @@ def sample_rows(logits: torch.Tensor, params: torch.Tensor, masks: Optional[torc
     words = (vocab + 31) // 32
     if masks is not None:
         assert masks.dim() == 2 and masks.shape[1] == words and masks.is_contiguous()
-    lib.check(lib.kernels().ds41_sample_rows(lib.ptr(logits), C.c_longlong(logits.stride(0)), rows, vocab, lib.ptr(masks),
+    lib.check(lib.kernels("any").ds41_sample_rows(lib.ptr(logits), C.c_longlong(logits.stride(0)), rows, vocab, lib.ptr(masks),
                                              words, lib.ptr(params), lib.ptr(tokens), lib.ptr(status), lib.stream()),
               "sample_rows")
     return tokens, status

@@ -67,7 +67,7 @@ class MlstmArgs(C.Structure):
 
 def mlstm_chunk_work(rows: int, heads: int) -> int:
     """Bytes of workspace of the chunked recurrence."""
-    fn = lib.kernels().ds41_mlstm_chunk_work
+    fn = lib.kernels("stack").ds41_mlstm_chunk_work
     fn.restype = C.c_longlong
     return fn(rows, heads)
 
@@ -198,5 +198,5 @@ def per_head(x: torch.Tensor, ldx: int, head_stride: int, rows: int, heads: int,
 
 def gemm_f32(a, b, out, M, N, K, lda, ldb, ldo, batch=1, sa=0, sb=0, so=0):
     ll = C.c_longlong
-    lib.check(lib.kernels().ds41_gemm_f32(lib.ptr(a), lib.ptr(b), lib.ptr(out), M, N, K, ll(lda), ll(ldb), ll(ldo), batch,
+    lib.check(lib.kernels("stack").ds41_gemm_f32(lib.ptr(a), lib.ptr(b), lib.ptr(out), M, N, K, ll(lda), ll(ldb), ll(ldo), batch,
                                           ll(sa), ll(sb), ll(so), lib.stream()), "ds41_gemm_f32")
