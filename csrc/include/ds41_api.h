@@ -551,7 +551,7 @@ typedef struct ds41_mlstm_args {
 int ds41_mlstm_step(const ds41_mlstm_args* args, void* stream);
 // Long pass of one request (row 0's slot; adjacent rows), dim_pad <= 512; q, k, v are bf16 with 16-byte aligned rows.
 int ds41_mlstm_chunk(const ds41_mlstm_args* args, void* stream);
-long long ds41_mlstm_chunk_work(int rows, int heads);
+long long ds41_mlstm_chunk_work(int rows, int heads, int dim_pad, int vdim_pad);
 
 int ds41_gemm_f32(const float* A, const float* B, float* out, int M, int N, int K, long long lda, long long ldb,
                   long long ldo, int batch, long long a_batch_stride, long long b_batch_stride,

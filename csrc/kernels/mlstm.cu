@@ -8,7 +8,8 @@
 //
 //  mlstm_step : one block walks the adjacent rows of a request token by token (decode rows, 32-bit passes), the state in
 //               registers, or in shared memory where it is too large for them
-//  mlstm_chunk: one request's rows, 64 at a time, on the tensor cores.  With F the running sum of f inside a chunk and m0
+//  mlstm_chunk: one request's rows, 64 at a time, on the tensor cores, in three launches: the gates of every chunk; the
+//               states from chunk to chunk; the outputs of all chunks side by side.  With F the running sum of f inside a chunk and m0
 //               the maximum before it, m_t = F_t + max(m0, max_{s<=t}(i_s - F_s)) is the same maximum the walk would find, and
 //                 S'^T q_t = exp(F_t + m0 - m_t) S^T q_t + sum_{s<=t} exp(F_t - F_s + i_s - m_t) (k_s . q_t) v_s
 //               fp32 factors of a product (state, decayed scores, decayed values) enter as bf16 high and low parts.
@@ -296,36 +297,45 @@ __global__ void __launch_bounds__(1024) mlstm_gates_kernel(ds41_mlstm_args p) {
   }
 }
 
+// Layout of the workspace, in bytes from its start.
+struct ChunkWork {
+  long long gates, n, state, total;
+};
+__host__ __device__ inline int chunk_tiles(int dim_pad) {        // NTD of the kernels that take this key width
+  return dim_pad <= 64 ? 2 : dim_pad <= 128 ? 4 : dim_pad <= 192 ? 6 : dim_pad <= 256 ? 8 : dim_pad <= 384 ? 12 : 16;
+}
+__host__ __device__ inline ChunkWork chunk_work(int rows, int heads, int dim_pad, int vdim_pad) {
+  const long long chunks = (rows + kChunk - 1) / kChunk, per = chunks * heads;
+  const long long D = chunk_tiles(dim_pad) * 32, nb = (vdim_pad + kStateCols - 1) / kStateCols;
+  ChunkWork w;
+  w.gates = 0;
+  w.n = per * kGateFloats * 4;
+  w.state = w.n + per * D * 4;
+  w.total = w.state + per * nb * D * kStateCols * 4;
+  return w;
+}
+
+// ---- states: walks the chunks of one head and 32 value columns and leaves the state before every chunk in the workspace
 template <int NTD>
-struct ChunkSmem {
+struct StateSmem {
   static constexpr int D = NTD * 32;
-  static constexpr int kStride = D + 8;                            // bf16 per row of a q / k tile
-  static constexpr int kTile = kChunk * kStride * 2;               // bytes
-  static constexpr int kStage = 2 * kTile + kChunk * kVStride * 2 + kGateFloats * 4;
-  static constexpr int kFixed = 2 * kChunk * kPStride * 2 + 2 * kChunk * kVStride * 2 + 8 * kStride * 2 +
-                                4 * kChunk * kRedStride * 4 + D * 4 + 4 * kChunk * 4;
-  static constexpr int kStages = 2 * kStage + kFixed <= 226 * 1024 ? 2 : 1;
+  static constexpr int kStride = D + 8;                            // bf16 per row of a key tile
+  static constexpr int kStage = kChunk * kStride * 2 + kChunk * kVStride * 2 + (kChunk + 4) * 4;
+  static constexpr int kFixed = 2 * kChunk * kVStride * 2 + D * 4;
+  static constexpr int kStages = 4 * kStage + kFixed <= 224 * 1024 ? 4 : 2;
   static constexpr int kBytes = kStages * kStage + kFixed;
 };
 
-// 256 threads.  In the products over the value columns warp w owns columns 16 (w & 1) .. +16 and the (w >> 1)-th quarter of
-// the key dimension, whose slice of the transposed state it keeps in registers; in Q K^T it owns 16 rows x 32 keys.
+// 256 threads; warp w owns value columns 16 (w & 1) .. +16 and the (w >> 1)-th quarter of the key dimension, whose slice of
+// the transposed state it keeps in registers.
 template <int NTD>
-__global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
-  using Sm = ChunkSmem<NTD>;
-  constexpr int D = Sm::D, DQ = D / 4;
-  extern __shared__ __align__(16) uint8_t mc_smem[];
-  uint8_t* fixed = mc_smem + Sm::kStages * Sm::kStage;
-  __nv_bfloat16* p_hi = reinterpret_cast<__nv_bfloat16*>(fixed);
-  __nv_bfloat16* p_lo = p_hi + kChunk * kPStride;
-  __nv_bfloat16* w_hi = p_lo + kChunk * kPStride;
+__global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
+  using Sm = StateSmem<NTD>;
+  constexpr int D = Sm::D, DQ = D / 4, S = Sm::kStages;
+  extern __shared__ __align__(16) uint8_t ms_raw[];
+  __nv_bfloat16* w_hi = reinterpret_cast<__nv_bfloat16*>(ms_raw + S * Sm::kStage);
   __nv_bfloat16* w_lo = w_hi + kChunk * kVStride;
-  __nv_bfloat16* n_rows = w_lo + kChunk * kVStride;                    // [8][D + 8]: n as high and low parts, zero rows
-  float* red = reinterpret_cast<float*>(n_rows + 8 * Sm::kStride);     // [4][64][33]
-  float* nv = red + 4 * kChunk * kRedStride;                           // [D]
-  float* nq = nv + D;                  // n . q_t before the chunk
-  float* rs = nq + kChunk;             // [2][64] sums of the decayed scores
-  float* inv = rs + 2 * kChunk;        // 1 / denominator
+  float* nv = reinterpret_cast<float*>(w_lo + kChunk * kVStride);      // [D]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int vb = blockIdx.x, h = blockIdx.y;
   const int nt = warp & 1, dq = warp >> 1, g = lane >> 2, q2 = 2 * (lane & 3);
@@ -337,45 +347,41 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
   const int nb = gridDim.x, col0 = vb * kStateCols;
   const long long head = 1ll * slot * p.heads + h;
   float* gS = p.state_s + head * p.dim_pad * p.vdim_pad;
-  float* gn = p.state_n + (head * nb + vb) * p.dim_pad;
+  float* gn = p.state_n + head * nb * p.dim_pad;
+  const ChunkWork wk = chunk_work(p.rows, p.heads, p.dim_pad, p.vdim_pad);
+  uint8_t* work = reinterpret_cast<uint8_t*>(p.work);
 
-  const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(p.q.data) + p.q.col + h * p.dim_pad;
   const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad;
   const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(p.v.data) + p.v.col + h * p.vdim_pad + col0;
   const int n_chunks = (p.rows + kChunk - 1) / kChunk;
   const uint4 zero = make_uint4(0, 0, 0, 0);
-  auto load = [&](int c, int stage) {
-    __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(mc_smem + stage * Sm::kStage);
-    __nv_bfloat16* sk = sq + kChunk * Sm::kStride;
-    __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
-    const int live = p.rows - c * kChunk;
-    constexpr int kPer = D / 8;                       // 16-byte pieces of a row
-    constexpr int kRows = kPer <= 256 ? 256 / kPer : 1;
-    if (kPer * kRows == 256 || tid < kPer * kRows) {
-      const int d = (tid % kPer) * 8;
-      const __nv_bfloat16* q = gq + (1ll * c * kChunk + tid / kPer) * p.q.ld + d;
-      const __nv_bfloat16* k = gk + (1ll * c * kChunk + tid / kPer) * p.k.ld + d;
-      for (int t = tid / kPer; t < kChunk; t += kRows, q += 1ll * kRows * p.q.ld, k += 1ll * kRows * p.k.ld) {
-        if (t < live && d < p.dim_pad) {
-          cp_async_16(sq + t * Sm::kStride + d, q);
-          cp_async_16(sk + t * Sm::kStride + d, k);
-        } else {
-          *reinterpret_cast<uint4*>(sq + t * Sm::kStride + d) = zero;
-          *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
+  auto load = [&](int c) {
+    if (c < n_chunks) {
+      __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(ms_raw + (c % S) * Sm::kStage);
+      __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
+      const int live = p.rows - c * kChunk;
+      constexpr int kPer = D / 8, kRows = 256 / kPer;                  // 16-byte pieces of a row, rows per sweep
+      if (kPer * kRows == 256 || tid < kPer * kRows) {
+        const int d = (tid % kPer) * 8;
+        const __nv_bfloat16* k = gk + (1ll * c * kChunk + tid / kPer) * p.k.ld + d;
+        for (int t = tid / kPer; t < kChunk; t += kRows, k += 1ll * kRows * p.k.ld) {
+          if (t < live && d < p.dim_pad) cp_async_16(sk + t * Sm::kStride + d, k);
+          else *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
         }
       }
-    }
-    {
       const int t = tid >> 2, d = (tid & 3) * 8;
       if (t < live && col0 + d < p.vdim_pad) cp_async_16(sv + t * kVStride + d, gv + (1ll * c * kChunk + t) * p.v.ld + d);
       else *reinterpret_cast<uint4*>(sv + t * kVStride + d) = zero;
+      // the weights of the keys and the scalars
+      const float* gates = p.work + (1ll * c * p.heads + h) * kGateFloats;
+      float* sg = reinterpret_cast<float*>(sv + kChunk * kVStride);
+      if (tid < kChunk / 4) cp_async_16(sg + 4 * tid, gates + 2 * kChunk + 4 * tid);
+      else if (tid == kChunk / 4) cp_async_16(sg + kChunk, gates + 5 * kChunk);
     }
-    if (tid < kGateFloats / 4)
-      cp_async_16(reinterpret_cast<float*>(sv + kChunk * kVStride) + 4 * tid,
-                  p.work + (1ll * c * p.heads + h) * kGateFloats + 4 * tid);
-    cp_async_commit();
+    cp_async_commit();                 // one group per call, so that the waits count calls
   };
-  load(0, 0);
+#pragma unroll
+  for (int i = 0; i < S - 1; ++i) load(i);
   // transposed state: tile j holds columns d = dq DQ + 8 j + q2 + {0, 1} of rows nt 16 + g and + 8
   float st[NTD][4];
 #pragma unroll
@@ -385,88 +391,20 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       const int d = dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
       st[j][e] = !fresh && d < p.dim_pad && c < p.vdim_pad ? gS[1ll * d * p.vdim_pad + c] : 0.f;
     }
-  for (int i = tid; i < 8 * Sm::kStride; i += 256) n_rows[i] = __float2bfloat16_rn(0.f);
-  __syncthreads();
-  for (int d = tid; d < D; d += 256) {
-    const float x = !fresh && d < p.dim_pad ? gn[d] : 0.f;
-    const __nv_bfloat16 hi = __float2bfloat16_rn(x);
-    nv[d] = x;
-    n_rows[d] = hi;
-    n_rows[Sm::kStride + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
-  }
+  if (vb == 0)
+    for (int d = tid; d < D; d += 256) nv[d] = !fresh && d < p.dim_pad ? gn[d] : 0.f;
   float m_end = 0.f;
   for (int c = 0; c < n_chunks; ++c) {
-    const int stage = Sm::kStages == 2 ? (c & 1) : 0;
-    if (Sm::kStages == 2 && c + 1 < n_chunks) {
-      load(c + 1, stage ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    const __nv_bfloat16* sq = reinterpret_cast<const __nv_bfloat16*>(mc_smem + stage * Sm::kStage);
-    const __nv_bfloat16* sk = sq + kChunk * Sm::kStride;
+    cp_async_wait<S - 2>();
+    __syncthreads();                   // chunk c is here; every warp is done with chunk c - 1
+    load(c + S - 1);
+    const __nv_bfloat16* sk = reinterpret_cast<const __nv_bfloat16*>(ms_raw + (c % S) * Sm::kStage);
     const __nv_bfloat16* sv = sk + kChunk * Sm::kStride;
-    const float* gates = reinterpret_cast<const float*>(sv + kChunk * kVStride);
-    __syncthreads();
-
-    // ---- decayed scores, 16 rows x 32 keys per warp; the warps of the first keys also take n . q_t
-    {
-      const int tm = warp >> 1, sh = warp & 1;
-      float acc[4][4] = {}, na[4] = {};
-      const __nv_bfloat16* arow = sq + (tm * 16 + (lane & 15)) * Sm::kStride + (lane >> 4) * 8;
-      const __nv_bfloat16* brow = sk + (sh * 32 + (lane & 7) + (lane >> 4) * 8) * Sm::kStride + ((lane >> 3) & 1) * 8;
-      const __nv_bfloat16* nrow = n_rows + (lane & 7) * Sm::kStride + (lane >> 3) * 8;
-      if (sh * 32 <= tm * 16 + 15) {
-#pragma unroll 4
-        for (int k = 0; k < D; k += 16) {
-          uint32_t a[4], b[8];
-          ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
-          ldmatrix_x4(b[0], b[1], b[2], b[3], brow + k);
-          ldmatrix_x4(b[4], b[5], b[6], b[7], brow + 16 * Sm::kStride + k);
-#pragma unroll
-          for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[j], a, b[2 * j], b[2 * j + 1]);
-        }
-      }
-      if (sh == 0) {
-#pragma unroll 2
-        for (int k = 0; k < D; k += 32) {
-          uint32_t a[4], b[4];
-          ldmatrix_x4(b[0], b[1], b[2], b[3], nrow + k);
-          ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
-          mma_bf16_16816(na, a, b[0], b[1]);
-          ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k + 16);
-          mma_bf16_16816(na, a, b[2], b[3]);
-        }
-        if ((lane & 3) == 0) {
-          nq[tm * 16 + g] = na[0] + na[1];
-          nq[tm * 16 + g + 8] = na[2] + na[3];
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int t = tm * 16 + g + 8 * u;
-        const float e = gates[t];
-        float sum = 0.f;
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const int s = sh * 32 + 8 * j + q2;
-          const float2 as = *reinterpret_cast<const float2*>(gates + kChunk + s);
-          const float x = s <= t ? acc[j][2 * u] * p.q_scale * ex2_approx(e + as.x) : 0.f;
-          const float y = s + 1 <= t ? acc[j][2 * u + 1] * p.q_scale * ex2_approx(e + as.y) : 0.f;
-          sum += x + y;
-          const uint32_t hi = pack_bf16(x, y);
-          *reinterpret_cast<uint32_t*>(p_hi + t * kPStride + s) = hi;
-          *reinterpret_cast<uint32_t*>(p_lo + t * kPStride + s) = pack_bf16_rest(x, y, hi);
-        }
-        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-        if ((lane & 3) == 0) rs[sh * kChunk + t] = sum;
-      }
-    }
+    const float* sg = reinterpret_cast<const float*>(sv + kChunk * kVStride);
     // ---- decayed values
     {
       const int s = tid >> 2, d = (tid & 3) * 8;
-      const float w = gates[2 * kChunk + s];
+      const float w = sg[s];
       const uint4 v4 = *reinterpret_cast<const uint4*>(sv + s * kVStride + d);
       const uint32_t v[4] = {v4.x, v4.y, v4.z, v4.w};
       uint32_t hi[4], lo[4];
@@ -479,12 +417,10 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       *reinterpret_cast<uint4*>(w_hi + s * kVStride + d) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
       *reinterpret_cast<uint4*>(w_lo + s * kVStride + d) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
-    __syncthreads();
-
-    // ---- output, transposed: 16 value columns x 64 rows per warp, this warp's quarter of d and of the keys
+    // ---- the state before this chunk, as the output kernel's left operand wants it: high and low parts per fragment
     {
-      float o[8][4] = {};
-      const __nv_bfloat16* brow = sq + ((lane & 7) + (lane >> 4) * 8) * Sm::kStride + dq * DQ + ((lane >> 3) & 1) * 8;
+      const long long cell = (1ll * c * p.heads + h) * nb + vb;
+      uint4* dst = reinterpret_cast<uint4*>(work + wk.state) + (cell * 8 + warp) * NTD * 32 + lane;
 #pragma unroll
       for (int k = 0; k < NTD / 2; ++k) {
         uint32_t hi[4], lo[4];
@@ -494,72 +430,39 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
           hi[e] = pack_bf16(x, y);
           lo[e] = pack_bf16_rest(x, y, hi[e]);
         }
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          uint32_t b[4];
-          ldmatrix_x4(b[0], b[1], b[2], b[3], brow + 16 * j * Sm::kStride + 16 * k);
-          mma_bf16_16816(o[2 * j], hi, b[0], b[1]);
-          mma_bf16_16816(o[2 * j + 1], hi, b[2], b[3]);
-          mma_bf16_16816(o[2 * j], lo, b[0], b[1]);
-          mma_bf16_16816(o[2 * j + 1], lo, b[2], b[3]);
-        }
+        dst[(2 * k) * 32] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        dst[(2 * k + 1) * 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float2 f = *reinterpret_cast<const float2*>(gates + 3 * kChunk + 8 * j + q2);
-        o[j][0] *= f.x;
-        o[j][1] *= f.y;
-        o[j][2] *= f.x;
-        o[j][3] *= f.y;
+      if (vb == 0) {
+        float* gw = reinterpret_cast<float*>(work + wk.n) + (1ll * c * p.heads + h) * D;
+        for (int d = tid; d < D; d += 256) gw[d] = nv[d];
       }
-      uint32_t a[4];
-      ldmatrix_x4_trans(a[0], a[1], a[2], a[3],
-                        sv + (dq * 16 + (lane & 7) + (lane >> 4) * 8) * kVStride + nt * 16 + ((lane >> 3) & 1) * 8);
-      const int prow = ((lane & 7) + (lane >> 4) * 8) * kPStride + dq * 16 + ((lane >> 3) & 1) * 8;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        uint32_t b[4];
-        ldmatrix_x4(b[0], b[1], b[2], b[3], p_hi + prow + 16 * j * kPStride);
-        mma_bf16_16816(o[2 * j], a, b[0], b[1]);
-        mma_bf16_16816(o[2 * j + 1], a, b[2], b[3]);
-        ldmatrix_x4(b[0], b[1], b[2], b[3], p_lo + prow + 16 * j * kPStride);
-        mma_bf16_16816(o[2 * j], a, b[0], b[1]);
-        mma_bf16_16816(o[2 * j + 1], a, b[2], b[3]);
-      }
-      float* dst = red + dq * kChunk * kRedStride + nt * 16 + g;
-#pragma unroll
-      for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) dst[(8 * j + q2 + (e & 1)) * kRedStride + (e >> 1) * 8] = o[j][e];
     }
-    if (tid < kChunk)
-      inv[tid] = 1.0f / (fmaxf(fabsf(gates[3 * kChunk + tid] * nq[tid] + rs[tid] + rs[kChunk + tid]), gates[4 * kChunk + tid]) +
-                         p.den_eps);
-    // ---- state after the chunk
-    {
-      const float keep = gates[5 * kChunk];
-      m_end = gates[5 * kChunk + 1];
+    __syncthreads();
+    const float keep = sg[kChunk];
+    m_end = sg[kChunk + 1];
 #pragma unroll
-      for (int j = 0; j < NTD; ++j)
+    for (int j = 0; j < NTD; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[j][e] *= keep;
-      const int arow = ((lane & 7) + (lane >> 4) * 8) * kVStride + nt * 16 + ((lane >> 3) & 1) * 8;
-      const __nv_bfloat16* brow = sk + (lane & 15) * Sm::kStride + dq * DQ + (lane >> 4) * 8;
+      for (int e = 0; e < 4; ++e) st[j][e] *= keep;
+    const int arow = ((lane & 7) + (lane >> 4) * 8) * kVStride + nt * 16 + ((lane >> 3) & 1) * 8;
+    const __nv_bfloat16* brow = sk + (lane & 15) * Sm::kStride + dq * DQ + (lane >> 4) * 8;
 #pragma unroll
-      for (int k = 0; k < kChunk; k += 16) {
-        uint32_t hi[4], lo[4];
-        ldmatrix_x4_trans(hi[0], hi[1], hi[2], hi[3], w_hi + arow + k * kVStride);
-        ldmatrix_x4_trans(lo[0], lo[1], lo[2], lo[3], w_lo + arow + k * kVStride);
+    for (int k = 0; k < kChunk; k += 16) {
+      uint32_t hi[4], lo[4];
+      ldmatrix_x4_trans(hi[0], hi[1], hi[2], hi[3], w_hi + arow + k * kVStride);
+      ldmatrix_x4_trans(lo[0], lo[1], lo[2], lo[3], w_lo + arow + k * kVStride);
 #pragma unroll
-        for (int j = 0; j < NTD / 2; ++j) {
-          uint32_t b[4];
-          ldmatrix_x4_trans(b[0], b[1], b[2], b[3], brow + k * Sm::kStride + 16 * j);
-          mma_bf16_16816(st[2 * j], hi, b[0], b[1]);
-          mma_bf16_16816(st[2 * j + 1], hi, b[2], b[3]);
-          mma_bf16_16816(st[2 * j], lo, b[0], b[1]);
-          mma_bf16_16816(st[2 * j + 1], lo, b[2], b[3]);
-        }
+      for (int j = 0; j < NTD / 2; ++j) {
+        uint32_t b[4];
+        ldmatrix_x4_trans(b[0], b[1], b[2], b[3], brow + k * Sm::kStride + 16 * j);
+        mma_bf16_16816(st[2 * j], hi, b[0], b[1]);
+        mma_bf16_16816(st[2 * j + 1], hi, b[2], b[3]);
+        mma_bf16_16816(st[2 * j], lo, b[0], b[1]);
+        mma_bf16_16816(st[2 * j + 1], lo, b[2], b[3]);
       }
+    }
+    if (vb == 0) {
       // n: one row of weights (high parts in row 0, low parts in row 1 of the left operand) times the keys; the two warps
       // of a quarter take half of its columns each
       uint32_t wf[4][2];
@@ -567,7 +470,7 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
       for (int k = 0; k < 4; ++k)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float2 w = *reinterpret_cast<const float2*>(gates + 2 * kChunk + 16 * k + 8 * e + q2);
+          const float2 w = *reinterpret_cast<const float2*>(sg + 16 * k + 8 * e + q2);
           const uint32_t hi = pack_bf16(w.x, w.y);
           wf[k][e] = g == 0 ? hi : (g == 1 ? pack_bf16_rest(w.x, w.y, hi) : 0u);
         }
@@ -591,59 +494,254 @@ __global__ void __launch_bounds__(256) mlstm_chunk_kernel(ds41_mlstm_args p) {
           const int d = dq * DQ + 16 * j + q2;
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
-            const int at = d + 8 * u;
-            const float n0 = nv[at] * keep + (u == 0 ? x[0] : y[0]), n1 = nv[at + 1] * keep + (u == 0 ? x[1] : y[1]);
-            nv[at] = n0;
-            nv[at + 1] = n1;
-            const uint32_t hi = pack_bf16(n0, n1);
-            *reinterpret_cast<uint32_t*>(n_rows + at) = hi;
-            *reinterpret_cast<uint32_t*>(n_rows + Sm::kStride + at) = pack_bf16_rest(n0, n1, hi);
+            nv[d + 8 * u] = nv[d + 8 * u] * keep + (u == 0 ? x[0] : y[0]);
+            nv[d + 8 * u + 1] = nv[d + 8 * u + 1] * keep + (u == 0 ? x[1] : y[1]);
           }
         }
       }
     }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < NTD; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
+      if (d < p.dim_pad && c < p.vdim_pad) gS[1ll * d * p.vdim_pad + c] = st[j][e];
+    }
+  if (vb == 0)                         // every column block's copy of n
+    for (int b = 0; b < nb; ++b)
+      for (int d = tid; d < p.dim_pad; d += 256) gn[1ll * b * p.dim_pad + d] = nv[d];
+  if (tid == 0) p.state_m[head * nb + vb] = m_end;
+}
+
+// ---- outputs: every (chunk, head, pair of value blocks) on its own, from the state before the chunk
+constexpr int kOutCols = 2 * kStateCols;
+constexpr int kOStride = kOutCols + 8;        // bf16 per row of the value tile
+
+template <int NTD>
+struct OutSmem {
+  static constexpr int D = NTD * 32;
+  static constexpr int kStride = D + 8;
+  static constexpr int kTile = kChunk * kStride * 2;
+  static constexpr int kRed = 4 * kChunk * kRedStride * 4;             // takes the key tile's place once it has been used
+  static constexpr int kKeys = kTile > kRed ? kTile : kRed;
+  static constexpr int kBytes = kTile + kKeys + kChunk * kOStride * 2 + kGateFloats * 4 + 2 * kChunk * kPStride * 2 +
+                                8 * kStride * 2 + 4 * kChunk * 4;
+};
+
+// 256 threads.  Q K^T: warp w owns 16 rows x 32 keys; outputs: as in the state kernel, one 32-column block after the other.
+template <int NTD>
+__global__ void __launch_bounds__(256) mlstm_output_kernel(ds41_mlstm_args p) {
+  using Sm = OutSmem<NTD>;
+  constexpr int D = Sm::D, DQ = D / 4;
+  extern __shared__ __align__(16) uint8_t mo_raw[];
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(mo_raw);
+  __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(mo_raw + Sm::kTile);
+  float* red = reinterpret_cast<float*>(sk);                           // [4][64][33]
+  __nv_bfloat16* sv = reinterpret_cast<__nv_bfloat16*>(mo_raw + Sm::kTile + Sm::kKeys);
+  float* gates = reinterpret_cast<float*>(sv + kChunk * kOStride);
+  __nv_bfloat16* p_hi = reinterpret_cast<__nv_bfloat16*>(gates + kGateFloats);
+  __nv_bfloat16* p_lo = p_hi + kChunk * kPStride;
+  __nv_bfloat16* n_rows = p_lo + kChunk * kPStride;                    // [8][D + 8]: n as high and low parts, zero rows
+  float* nq = reinterpret_cast<float*>(n_rows + 8 * Sm::kStride);      // n . q_t before the chunk
+  float* rs = nq + kChunk;             // [2][64] sums of the decayed scores
+  float* inv = rs + 2 * kChunk;        // 1 / denominator
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int pair = blockIdx.x, h = blockIdx.y, c = blockIdx.z;
+  const int nt = warp & 1, dq = warp >> 1, g = lane >> 2, q2 = 2 * (lane & 3);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slot = p.row_slot[0];
+  if (slot < 0 || slot >= p.slots) return;
+  const int nb = (p.vdim_pad + kStateCols - 1) / kStateCols, col0 = pair * kOutCols, live = p.rows - c * kChunk;
+  const ChunkWork wk = chunk_work(p.rows, p.heads, p.dim_pad, p.vdim_pad);
+  const uint8_t* work = reinterpret_cast<const uint8_t*>(p.work);
+  const long long cell = 1ll * c * p.heads + h;
+  {
+    const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(p.q.data) + p.q.col + h * p.dim_pad;
+    const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad;
+    const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(p.v.data) + p.v.col + h * p.vdim_pad + col0;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    constexpr int kPer = D / 8, kRows = 256 / kPer;
+    if (kPer * kRows == 256 || tid < kPer * kRows) {
+      const int d = (tid % kPer) * 8;
+      const __nv_bfloat16* q = gq + (1ll * c * kChunk + tid / kPer) * p.q.ld + d;
+      const __nv_bfloat16* k = gk + (1ll * c * kChunk + tid / kPer) * p.k.ld + d;
+      for (int t = tid / kPer; t < kChunk; t += kRows, q += 1ll * kRows * p.q.ld, k += 1ll * kRows * p.k.ld) {
+        if (t < live && d < p.dim_pad) {
+          cp_async_16(sq + t * Sm::kStride + d, q);
+          cp_async_16(sk + t * Sm::kStride + d, k);
+        } else {
+          *reinterpret_cast<uint4*>(sq + t * Sm::kStride + d) = zero;
+          *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
+        }
+      }
+    }
+#pragma unroll
+    for (int i = tid; i < kChunk * kOutCols / 8; i += 256) {
+      const int t = i >> 3, d = (i & 7) * 8;
+      if (t < live && col0 + d < p.vdim_pad) cp_async_16(sv + t * kOStride + d, gv + (1ll * c * kChunk + t) * p.v.ld + d);
+      else *reinterpret_cast<uint4*>(sv + t * kOStride + d) = zero;
+    }
+    if (tid < kGateFloats / 4) cp_async_16(gates + 4 * tid, p.work + cell * kGateFloats + 4 * tid);
+    cp_async_commit();
+    const float* gw = reinterpret_cast<const float*>(work + wk.n) + cell * D;
+    for (int d = tid; d < D; d += 256) {
+      const float x = gw[d];
+      const __nv_bfloat16 hi = __float2bfloat16_rn(x);
+      n_rows[d] = hi;
+      n_rows[Sm::kStride + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
+    }
+    for (int i = tid; i < 6 * Sm::kStride; i += 256) n_rows[2 * Sm::kStride + i] = __float2bfloat16_rn(0.f);
+    cp_async_wait<0>();
+  }
+  __syncthreads();
+  // ---- decayed scores, 16 rows x 32 keys per warp; one warp per row tile also takes n . q_t
+  {
+    const int tm = warp >> 1, sh = warp & 1;
+    float acc[4][4] = {}, na[4] = {};
+    const __nv_bfloat16* arow = sq + (tm * 16 + (lane & 15)) * Sm::kStride + (lane >> 4) * 8;
+    const __nv_bfloat16* brow = sk + (sh * 32 + (lane & 7) + (lane >> 4) * 8) * Sm::kStride + ((lane >> 3) & 1) * 8;
+    const __nv_bfloat16* nrow = n_rows + (lane & 7) * Sm::kStride + (lane >> 3) * 8;
+    if (sh * 32 <= tm * 16 + 15) {
+#pragma unroll 4
+      for (int k = 0; k < D; k += 16) {
+        uint32_t a[4], b[8];
+        ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
+        ldmatrix_x4(b[0], b[1], b[2], b[3], brow + k);
+        ldmatrix_x4(b[4], b[5], b[6], b[7], brow + 16 * Sm::kStride + k);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[j], a, b[2 * j], b[2 * j + 1]);
+      }
+    }
+    if ((sh == 1) == (tm < 2)) {        // of the first row tiles the warps that have no visible keys
+#pragma unroll 2
+      for (int k = 0; k < D; k += 32) {
+        uint32_t a[4], b[4];
+        ldmatrix_x4(b[0], b[1], b[2], b[3], nrow + k);
+        ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k);
+        mma_bf16_16816(na, a, b[0], b[1]);
+        ldmatrix_x4(a[0], a[1], a[2], a[3], arow + k + 16);
+        mma_bf16_16816(na, a, b[2], b[3]);
+      }
+      if ((lane & 3) == 0) {
+        nq[tm * 16 + g] = na[0] + na[1];
+        nq[tm * 16 + g + 8] = na[2] + na[3];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = tm * 16 + g + 8 * u;
+      const float e = gates[t];
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int s = sh * 32 + 8 * j + q2;
+        const float2 as = *reinterpret_cast<const float2*>(gates + kChunk + s);
+        const float x = s <= t ? acc[j][2 * u] * p.q_scale * ex2_approx(e + as.x) : 0.f;
+        const float y = s + 1 <= t ? acc[j][2 * u + 1] * p.q_scale * ex2_approx(e + as.y) : 0.f;
+        sum += x + y;
+        const uint32_t hi = pack_bf16(x, y);
+        *reinterpret_cast<uint32_t*>(p_hi + t * kPStride + s) = hi;
+        *reinterpret_cast<uint32_t*>(p_lo + t * kPStride + s) = pack_bf16_rest(x, y, hi);
+      }
+      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      if ((lane & 3) == 0) rs[sh * kChunk + t] = sum;
+    }
+  }
+  __syncthreads();
+  if (tid < kChunk)
+    inv[tid] = 1.0f / (fmaxf(fabsf(gates[3 * kChunk + tid] * nq[tid] + rs[tid] + rs[kChunk + tid]), gates[4 * kChunk + tid]) +
+                       p.den_eps);
+  // ---- outputs, transposed: 16 value columns x 64 rows per warp, this warp's quarter of d and of the keys
+#pragma unroll 1
+  for (int half = 0; half < 2; ++half) {
+    const int vb = 2 * pair + half;
+    if (vb >= nb) break;
+    const uint4* frag = reinterpret_cast<const uint4*>(work + wk.state) + ((cell * nb + vb) * 8 + warp) * NTD * 32 + lane;
+    float o[8][4] = {};
+    const __nv_bfloat16* brow = sq + ((lane & 7) + (lane >> 4) * 8) * Sm::kStride + dq * DQ + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int k = 0; k < NTD / 2; ++k) {
+      const uint4 fh = frag[(2 * k) * 32], fl = frag[(2 * k + 1) * 32];
+      const uint32_t hi[4] = {fh.x, fh.y, fh.z, fh.w}, lo[4] = {fl.x, fl.y, fl.z, fl.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        uint32_t b[4];
+        ldmatrix_x4(b[0], b[1], b[2], b[3], brow + 16 * j * Sm::kStride + 16 * k);
+        mma_bf16_16816(o[2 * j], hi, b[0], b[1]);
+        mma_bf16_16816(o[2 * j + 1], hi, b[2], b[3]);
+        mma_bf16_16816(o[2 * j], lo, b[0], b[1]);
+        mma_bf16_16816(o[2 * j + 1], lo, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float2 f = *reinterpret_cast<const float2*>(gates + 3 * kChunk + 8 * j + q2);
+      o[j][0] *= f.x;
+      o[j][1] *= f.y;
+      o[j][2] *= f.x;
+      o[j][3] *= f.y;
+    }
+    uint32_t a[4];
+    ldmatrix_x4_trans(a[0], a[1], a[2], a[3], sv + (dq * 16 + (lane & 7) + (lane >> 4) * 8) * kOStride +
+                                                  half * kStateCols + nt * 16 + ((lane >> 3) & 1) * 8);
+    const int prow = ((lane & 7) + (lane >> 4) * 8) * kPStride + dq * 16 + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      uint32_t b[4];
+      ldmatrix_x4(b[0], b[1], b[2], b[3], p_hi + prow + 16 * j * kPStride);
+      mma_bf16_16816(o[2 * j], a, b[0], b[1]);
+      mma_bf16_16816(o[2 * j + 1], a, b[2], b[3]);
+      ldmatrix_x4(b[0], b[1], b[2], b[3], p_lo + prow + 16 * j * kPStride);
+      mma_bf16_16816(o[2 * j], a, b[0], b[1]);
+      mma_bf16_16816(o[2 * j + 1], a, b[2], b[3]);
+    }
+    float* part = red + dq * kChunk * kRedStride + nt * 16 + g;
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) part[(8 * j + q2 + (e & 1)) * kRedStride + (e >> 1) * 8] = o[j][e];
     __syncthreads();
-    if (col0 + lane < p.vdim_pad) {
-      const int t0 = warp * 8, live = min(8, p.rows - c * kChunk - t0);
-      float* dst = p.out + (1ll * c * kChunk + t0) * p.ld_out + h * p.vdim_pad + col0 + lane;
+    const int col = vb * kStateCols + lane;
+    if (col < p.vdim_pad) {
+      const int t0 = warp * 8;
+      float* dst = p.out + (1ll * c * kChunk + t0) * p.ld_out + h * p.vdim_pad + col;
       const float* src = red + t0 * kRedStride + lane;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         float x = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) x += src[(w * kChunk + i) * kRedStride];
-        if (i < live) dst[1ll * i * p.ld_out] = x * inv[t0 + i];
+        if (t0 + i < live) dst[1ll * i * p.ld_out] = x * inv[t0 + i];
       }
     }
     __syncthreads();
-    if (Sm::kStages == 1 && c + 1 < n_chunks) load(c + 1, 0);
   }
-#pragma unroll
-  for (int j = 0; j < NTD; ++j)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = dq * DQ + 8 * j + q2 + (e & 1), cc = col0 + nt * 16 + g + (e >> 1) * 8;
-      if (d < p.dim_pad && cc < p.vdim_pad) gS[1ll * d * p.vdim_pad + cc] = st[j][e];
-    }
-  for (int d = tid; d < p.dim_pad; d += 256) gn[d] = nv[d];
-  if (tid == 0) p.state_m[head * nb + vb] = m_end;
 }
 
 template <int NTD>
 static int launch_chunk(const ds41_mlstm_args& a, cudaStream_t st) {
   static bool ready = false;
+  cudaError_t e = cudaSuccess;
   if (!ready) {
-    const cudaError_t e = cudaFuncSetAttribute(mlstm_chunk_kernel<NTD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               ChunkSmem<NTD>::kBytes);
+    e = cudaFuncSetAttribute(mlstm_state_kernel<NTD>, cudaFuncAttributeMaxDynamicSharedMemorySize, StateSmem<NTD>::kBytes);
+    if (e != cudaSuccess) return e;
+    e = cudaFuncSetAttribute(mlstm_output_kernel<NTD>, cudaFuncAttributeMaxDynamicSharedMemorySize, OutSmem<NTD>::kBytes);
     if (e != cudaSuccess) return e;
     ready = true;
   }
-  const size_t gate_smem = 3ull * ((a.rows + kChunk - 1) / kChunk) * sizeof(float);
+  const int n_chunks = (a.rows + kChunk - 1) / kChunk, nb = (a.vdim_pad + kStateCols - 1) / kStateCols;
+  const size_t gate_smem = 3ull * n_chunks * sizeof(float);
   if (gate_smem > 48 * 1024) return cudaErrorInvalidValue;
-  const cudaError_t e = launch_pdl(mlstm_gates_kernel, dim3(a.heads), dim3(1024), gate_smem, st, a);
+  e = launch_pdl(mlstm_gates_kernel, dim3(a.heads), dim3(1024), gate_smem, st, a);
   if (e != cudaSuccess) return e;
-  const dim3 grid((a.vdim_pad + kStateCols - 1) / kStateCols, a.heads);
-  return launch_pdl(mlstm_chunk_kernel<NTD>, grid, dim3(256), ChunkSmem<NTD>::kBytes, st, a);
+  e = launch_pdl(mlstm_state_kernel<NTD>, dim3(nb, a.heads), dim3(256), StateSmem<NTD>::kBytes, st, a);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(mlstm_output_kernel<NTD>, dim3((nb + 1) / 2, a.heads, n_chunks), dim3(256), OutSmem<NTD>::kBytes, st, a);
 }
 
 }  // namespace ds41
@@ -688,15 +786,17 @@ extern "C" int ds41_mlstm_chunk(const ds41_mlstm_args* a, void* stream) {
     if (!x->bf16 || (x->ld & 7) || (x->col & 7) || (reinterpret_cast<uintptr_t>(x->data) & 15)) return cudaErrorInvalidValue;
   if ((a->dim_pad & 15) || (a->vdim_pad & 15) || a->work == nullptr || (reinterpret_cast<uintptr_t>(a->work) & 15)) return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (a->dim_pad <= 64) return launch_chunk<2>(*a, st);
-  if (a->dim_pad <= 128) return launch_chunk<4>(*a, st);
-  if (a->dim_pad <= 192) return launch_chunk<6>(*a, st);
-  if (a->dim_pad <= 256) return launch_chunk<8>(*a, st);
-  if (a->dim_pad <= 384) return launch_chunk<12>(*a, st);
-  if (a->dim_pad <= 512) return launch_chunk<16>(*a, st);
-  return cudaErrorInvalidValue;
+  if (a->dim_pad > 512) return cudaErrorInvalidValue;
+  switch (chunk_tiles(a->dim_pad)) {
+    case 2: return launch_chunk<2>(*a, st);
+    case 4: return launch_chunk<4>(*a, st);
+    case 6: return launch_chunk<6>(*a, st);
+    case 8: return launch_chunk<8>(*a, st);
+    case 12: return launch_chunk<12>(*a, st);
+    default: return launch_chunk<16>(*a, st);
+  }
 }
 
-extern "C" long long ds41_mlstm_chunk_work(int rows, int heads) {
-  return rows <= 0 || heads <= 0 ? 0 : 4ll * kGateFloats * heads * ((rows + kChunk - 1) / kChunk);
+extern "C" long long ds41_mlstm_chunk_work(int rows, int heads, int dim_pad, int vdim_pad) {
+  return rows <= 0 || heads <= 0 || dim_pad <= 0 || vdim_pad <= 0 ? 0 : chunk_work(rows, heads, dim_pad, vdim_pad).total;
 }

@@ -431,8 +431,10 @@ class StackEngine(RowsEngine):
         wide = max(S.ceil_to(n, 8) for lw in weights.layers for m in (lw.mixer, lw.mlp) if m is not None
                    for n, _ in m.matrices()["a"])
         self.wide = z((R * wide if R >= self.long_rows and not self.f32 else 8,), BF16)
-        heads_rec = max([lw.mixer.spec.heads for lw in weights.layers if isinstance(lw.mixer, MLSTM)], default=0)
-        self.recurrence_work = z((S.mlstm_chunk_work(R, heads_rec) // 4 + 4,), F32)
+        long_rec = [lw.mixer for lw in weights.layers if isinstance(lw.mixer, MLSTM) and lw.mixer.chunked] \
+            if R >= self.long_rows else []
+        self.recurrence_work = z((max([S.mlstm_chunk_work(R, m.spec.heads, m.dp, m.vp) for m in long_rec], default=0) // 4 + 4,),
+                                 F32)
         self._keys = [z((8,), BF16) for _ in range(3)]
         self.act = z((R * max(act, heads),), dt)
         self.o_heads = z((R * heads,), F32)

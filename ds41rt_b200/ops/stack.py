@@ -65,11 +65,11 @@ class MlstmArgs(C.Structure):
                 ("heads", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int), ("slots", C.c_int), ("ld_out", C.c_int)]
 
 
-def mlstm_chunk_work(rows: int, heads: int) -> int:
-    """Bytes of workspace of the chunked recurrence."""
+def mlstm_chunk_work(rows: int, heads: int, dim_pad: int, vdim_pad: int) -> int:
+    """Bytes of workspace of the chunked recurrence (mostly the state before every chunk)."""
     fn = lib.kernels("stack").ds41_mlstm_chunk_work
     fn.restype = C.c_longlong
-    return fn(rows, heads)
+    return fn(rows, heads, dim_pad, vdim_pad)
 
 
 STATE_COLS = 32       # value columns per state block of the mLSTM kernels (kStateCols)

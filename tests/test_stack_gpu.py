@@ -572,7 +572,7 @@ class Recurrence:
         x = torch.cat([q, kk, v], 1).to(dtype).cuda()
         gates = torch.cat([self.i, self.f], 1).float().cuda()
         bi, bf = self.bi.float().cuda(), self.bf.float().cuda()
-        work = torch.zeros(S.mlstm_chunk_work(self.T, self.H) // 4).cuda()
+        work = torch.zeros(S.mlstm_chunk_work(self.T, self.H, dp, vp) // 4).cuda()
         outs, at, n_call = [], 0, 0
         while at < self.T:
             n = min(sizes[min(n_call, len(sizes) - 1)], self.T - at)
