@@ -316,28 +316,31 @@ __host__ __device__ inline ChunkWork chunk_work(int rows, int heads, int dim_pad
 }
 
 // ---- states: walks the chunks of one head and 32 value columns and leaves the state before every chunk in the workspace
+// The key dimension is shared by kSplit CTAs, whose warps take slices of a quarter each.
 template <int NTD>
 struct StateSmem {
-  static constexpr int D = NTD * 32;
+  static constexpr int kSplit = NTD % 4 == 0 ? 2 : 1;
+  static constexpr int D = NTD * 32 / kSplit;                      // key columns of this CTA
+  static constexpr int NT = NTD / kSplit;                          // state tiles of 8 key columns per warp
   static constexpr int kStride = D + 8;                            // bf16 per row of a key tile
   static constexpr int kStage = kChunk * kStride * 2 + kChunk * kVStride * 2 + (kChunk + 4) * 4;
   static constexpr int kFixed = 2 * kChunk * kVStride * 2 + D * 4;
-  static constexpr int kStages = 4 * kStage + kFixed <= 224 * 1024 ? 4 : 2;
+  static constexpr int kStages = 2 * (4 * kStage + kFixed) <= 224 * 1024 ? 4 : 3;      // two CTAs per SM where they fit
   static constexpr int kBytes = kStages * kStage + kFixed;
 };
 
-// 256 threads; warp w owns value columns 16 (w & 1) .. +16 and the (w >> 1)-th quarter of the key dimension, whose slice of
-// the transposed state it keeps in registers.
+// 256 threads; warp w owns value columns 16 (w & 1) .. +16 and the (w >> 1)-th quarter of this CTA's key columns, whose slice
+// of the transposed state it keeps in registers.
 template <int NTD>
 __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
   using Sm = StateSmem<NTD>;
-  constexpr int D = Sm::D, DQ = D / 4, S = Sm::kStages;
+  constexpr int D = Sm::D, DQ = D / 4, S = Sm::kStages, NT = Sm::NT;
   extern __shared__ __align__(16) uint8_t ms_raw[];
   __nv_bfloat16* w_hi = reinterpret_cast<__nv_bfloat16*>(ms_raw + S * Sm::kStage);
   __nv_bfloat16* w_lo = w_hi + kChunk * kVStride;
   float* nv = reinterpret_cast<float*>(w_lo + kChunk * kVStride);      // [D]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int vb = blockIdx.x, h = blockIdx.y;
+  const int vb = blockIdx.x, h = blockIdx.y, d_base = blockIdx.z * D;
   const int nt = warp & 1, dq = warp >> 1, g = lane >> 2, q2 = 2 * (lane & 3);
   pdl_launch_dependents();
   pdl_wait();
@@ -351,7 +354,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
   const ChunkWork wk = chunk_work(p.rows, p.heads, p.dim_pad, p.vdim_pad);
   uint8_t* work = reinterpret_cast<uint8_t*>(p.work);
 
-  const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad;
+  const __nv_bfloat16* gk = static_cast<const __nv_bfloat16*>(p.k.data) + p.k.col + h * p.dim_pad + d_base;
   const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(p.v.data) + p.v.col + h * p.vdim_pad + col0;
   const int n_chunks = (p.rows + kChunk - 1) / kChunk;
   const uint4 zero = make_uint4(0, 0, 0, 0);
@@ -365,7 +368,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
         const int d = (tid % kPer) * 8;
         const __nv_bfloat16* k = gk + (1ll * c * kChunk + tid / kPer) * p.k.ld + d;
         for (int t = tid / kPer; t < kChunk; t += kRows, k += 1ll * kRows * p.k.ld) {
-          if (t < live && d < p.dim_pad) cp_async_16(sk + t * Sm::kStride + d, k);
+          if (t < live && d_base + d < p.dim_pad) cp_async_16(sk + t * Sm::kStride + d, k);
           else *reinterpret_cast<uint4*>(sk + t * Sm::kStride + d) = zero;
         }
       }
@@ -382,17 +385,17 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
   };
 #pragma unroll
   for (int i = 0; i < S - 1; ++i) load(i);
-  // transposed state: tile j holds columns d = dq DQ + 8 j + q2 + {0, 1} of rows nt 16 + g and + 8
-  float st[NTD][4];
+  // transposed state: tile j holds columns d = d_base + dq DQ + 8 j + q2 + {0, 1} of rows nt 16 + g and + 8
+  float st[NT][4];
 #pragma unroll
-  for (int j = 0; j < NTD; ++j)
+  for (int j = 0; j < NT; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
+      const int d = d_base + dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
       st[j][e] = !fresh && d < p.dim_pad && c < p.vdim_pad ? gS[1ll * d * p.vdim_pad + c] : 0.f;
     }
   if (vb == 0)
-    for (int d = tid; d < D; d += 256) nv[d] = !fresh && d < p.dim_pad ? gn[d] : 0.f;
+    for (int d = tid; d < D; d += 256) nv[d] = !fresh && d_base + d < p.dim_pad ? gn[d_base + d] : 0.f;
   float m_end = 0.f;
   for (int c = 0; c < n_chunks; ++c) {
     cp_async_wait<S - 2>();
@@ -420,9 +423,11 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
     // ---- the state before this chunk, as the output kernel's left operand wants it: high and low parts per fragment
     {
       const long long cell = (1ll * c * p.heads + h) * nb + vb;
-      uint4* dst = reinterpret_cast<uint4*>(work + wk.state) + (cell * 8 + warp) * NTD * 32 + lane;
+      // the output kernel's warp and its first fragment that these columns belong to
+      const int slice = blockIdx.z * 4 + dq, quarter = slice / Sm::kSplit, first = slice % Sm::kSplit * (NT / 2);
+      uint4* dst = reinterpret_cast<uint4*>(work + wk.state) + (cell * 8 + quarter * 2 + nt) * NTD * 32 + first * 64 + lane;
 #pragma unroll
-      for (int k = 0; k < NTD / 2; ++k) {
+      for (int k = 0; k < NT / 2; ++k) {
         uint32_t hi[4], lo[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
@@ -434,7 +439,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
         dst[(2 * k + 1) * 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
       if (vb == 0) {
-        float* gw = reinterpret_cast<float*>(work + wk.n) + (1ll * c * p.heads + h) * D;
+        float* gw = reinterpret_cast<float*>(work + wk.n) + (1ll * c * p.heads + h) * NTD * 32 + d_base;
         for (int d = tid; d < D; d += 256) gw[d] = nv[d];
       }
     }
@@ -442,7 +447,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
     const float keep = sg[kChunk];
     m_end = sg[kChunk + 1];
 #pragma unroll
-    for (int j = 0; j < NTD; ++j)
+    for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) st[j][e] *= keep;
     const int arow = ((lane & 7) + (lane >> 4) * 8) * kVStride + nt * 16 + ((lane >> 3) & 1) * 8;
@@ -453,7 +458,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
       ldmatrix_x4_trans(hi[0], hi[1], hi[2], hi[3], w_hi + arow + k * kVStride);
       ldmatrix_x4_trans(lo[0], lo[1], lo[2], lo[3], w_lo + arow + k * kVStride);
 #pragma unroll
-      for (int j = 0; j < NTD / 2; ++j) {
+      for (int j = 0; j < NT / 2; ++j) {
         uint32_t b[4];
         ldmatrix_x4_trans(b[0], b[1], b[2], b[3], brow + k * Sm::kStride + 16 * j);
         mma_bf16_16816(st[2 * j], hi, b[0], b[1]);
@@ -475,7 +480,7 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
           wf[k][e] = g == 0 ? hi : (g == 1 ? pack_bf16_rest(w.x, w.y, hi) : 0u);
         }
 #pragma unroll
-      for (int j = nt; j < NTD / 2; j += 2) {
+      for (int j = nt; j < NT / 2; j += 2) {
         float x[4] = {}, y[4] = {};
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
@@ -504,16 +509,17 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(ds41_mlstm_args p) {
   cp_async_wait<0>();
   __syncthreads();
 #pragma unroll
-  for (int j = 0; j < NTD; ++j)
+  for (int j = 0; j < NT; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
+      const int d = d_base + dq * DQ + 8 * j + q2 + (e & 1), c = col0 + nt * 16 + g + (e >> 1) * 8;
       if (d < p.dim_pad && c < p.vdim_pad) gS[1ll * d * p.vdim_pad + c] = st[j][e];
     }
   if (vb == 0)                         // every column block's copy of n
     for (int b = 0; b < nb; ++b)
-      for (int d = tid; d < p.dim_pad; d += 256) gn[1ll * b * p.dim_pad + d] = nv[d];
-  if (tid == 0) p.state_m[head * nb + vb] = m_end;
+      for (int d = tid; d < D; d += 256)
+        if (d_base + d < p.dim_pad) gn[1ll * b * p.dim_pad + d_base + d] = nv[d];
+  if (tid == 0 && blockIdx.z == 0) p.state_m[head * nb + vb] = m_end;
 }
 
 // ---- outputs: every (chunk, head, pair of value blocks) on its own, from the state before the chunk
@@ -533,7 +539,7 @@ struct OutSmem {
 
 // 256 threads.  Q K^T: warp w owns 16 rows x 32 keys; outputs: as in the state kernel, one 32-column block after the other.
 template <int NTD>
-__global__ void __launch_bounds__(256) mlstm_output_kernel(ds41_mlstm_args p) {
+__global__ void __launch_bounds__(256, NTD <= 8 ? 2 : 1) mlstm_output_kernel(ds41_mlstm_args p) {
   using Sm = OutSmem<NTD>;
   constexpr int D = Sm::D, DQ = D / 4;
   extern __shared__ __align__(16) uint8_t mo_raw[];
@@ -595,8 +601,16 @@ __global__ void __launch_bounds__(256) mlstm_output_kernel(ds41_mlstm_args p) {
       n_rows[Sm::kStride + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
     }
     for (int i = tid; i < 6 * Sm::kStride; i += 256) n_rows[2 * Sm::kStride + i] = __float2bfloat16_rn(0.f);
-    cp_async_wait<0>();
   }
+  // the state fragments of the first value block travel while the scores are computed
+  constexpr bool kAhead = NTD <= 8;
+  constexpr int kFrags = kAhead ? NTD : 2;
+  const uint4* frag = reinterpret_cast<const uint4*>(work + wk.state) + ((cell * nb + 2 * pair) * 8 + warp) * NTD * 32 + lane;
+  uint4 ahead[kFrags];
+  if (kAhead)
+#pragma unroll
+    for (int k = 0; k < kFrags; ++k) ahead[k] = __ldcg(frag + k * 32);
+  cp_async_wait<0>();
   __syncthreads();
   // ---- decayed scores, 16 rows x 32 keys per warp; one warp per row tile also takes n . q_t
   {
@@ -661,12 +675,12 @@ __global__ void __launch_bounds__(256) mlstm_output_kernel(ds41_mlstm_args p) {
   for (int half = 0; half < 2; ++half) {
     const int vb = 2 * pair + half;
     if (vb >= nb) break;
-    const uint4* frag = reinterpret_cast<const uint4*>(work + wk.state) + ((cell * nb + vb) * 8 + warp) * NTD * 32 + lane;
     float o[8][4] = {};
     const __nv_bfloat16* brow = sq + ((lane & 7) + (lane >> 4) * 8) * Sm::kStride + dq * DQ + ((lane >> 3) & 1) * 8;
 #pragma unroll
     for (int k = 0; k < NTD / 2; ++k) {
-      const uint4 fh = frag[(2 * k) * 32], fl = frag[(2 * k + 1) * 32];
+      const uint4 fh = kAhead ? ahead[(2 * k) % kFrags] : __ldcg(frag + (2 * k) * 32);
+      const uint4 fl = kAhead ? ahead[(2 * k + 1) % kFrags] : __ldcg(frag + (2 * k + 1) * 32);
       const uint32_t hi[4] = {fh.x, fh.y, fh.z, fh.w}, lo[4] = {fl.x, fl.y, fl.z, fl.w};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -678,6 +692,10 @@ __global__ void __launch_bounds__(256) mlstm_output_kernel(ds41_mlstm_args p) {
         mma_bf16_16816(o[2 * j + 1], lo, b[2], b[3]);
       }
     }
+    frag += 8 * NTD * 32;               // the next value block's
+    if (kAhead && half == 0 && vb + 1 < nb)
+#pragma unroll
+      for (int k = 0; k < kFrags; ++k) ahead[k] = __ldcg(frag + k * 32);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float2 f = *reinterpret_cast<const float2*>(gates + 3 * kChunk + 8 * j + q2);
@@ -739,7 +757,7 @@ static int launch_chunk(const ds41_mlstm_args& a, cudaStream_t st) {
   if (gate_smem > 48 * 1024) return cudaErrorInvalidValue;
   e = launch_pdl(mlstm_gates_kernel, dim3(a.heads), dim3(1024), gate_smem, st, a);
   if (e != cudaSuccess) return e;
-  e = launch_pdl(mlstm_state_kernel<NTD>, dim3(nb, a.heads), dim3(256), StateSmem<NTD>::kBytes, st, a);
+  e = launch_pdl(mlstm_state_kernel<NTD>, dim3(nb, a.heads, StateSmem<NTD>::kSplit), dim3(256), StateSmem<NTD>::kBytes, st, a);
   if (e != cudaSuccess) return e;
   return launch_pdl(mlstm_output_kernel<NTD>, dim3((nb + 1) / 2, a.heads, n_chunks), dim3(256), OutSmem<NTD>::kBytes, st, a);
 }
