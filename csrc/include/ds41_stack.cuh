@@ -37,6 +37,27 @@ __device__ __forceinline__ float4 proj_at4(const ds41_proj& a, long long row, in
   }
   return s;
 }
+// Two neighbouring elements at an even column (even row lengths and planes).
+__device__ __forceinline__ float2 proj_at2(const ds41_proj& a, long long row, int col) {
+  const long long i = row * a.ld + a.col + col;
+  if (a.bf16) {
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(a.data) + i);
+    return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
+  }
+  const float* p = static_cast<const float*>(a.data) + i;
+  float2 s = *reinterpret_cast<const float2*>(p);
+#pragma unroll 4
+  for (int k = 1; k < a.splits; ++k) {
+    const float2 t = *reinterpret_cast<const float2*>(p + k * a.plane);
+    s.x += t.x;
+    s.y += t.y;
+  }
+  return s;
+}
+__device__ __forceinline__ void store2(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float x, float y) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y);
+}
 inline bool proj_ok(const ds41_proj& p) {
   return p.data != nullptr && p.ld > 0 && p.splits >= 1 && p.col >= 0 && (p.splits == 1 || (p.plane > 0 && !p.bf16));
 }

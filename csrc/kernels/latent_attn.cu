@@ -97,6 +97,58 @@ __global__ void __launch_bounds__(256) latent_post_kernel(ds41_latent_post_args 
   norm_row(p.kv, r, p.kv_rank, p.kv_norm, p.eps, row, red);
 }
 
+// Long passes: one warp per row and part, the row in registers (up to 2048 columns).
+constexpr int kWarpPieces = 16;
+template <typename T>
+__device__ __forceinline__ void norm_row_warp(const ds41_proj& p, int r, int n, const float* w, float eps, T* out) {
+  const int lane = threadIdx.x & 31;
+  float4 v[kWarpPieces];
+  float q = 0.f;
+#pragma unroll
+  for (int k = 0; k < kWarpPieces; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      v[k] = proj_at4(p, r, i);
+      if (i + 1 >= n) v[k].y = 0.f;
+      if (i + 2 >= n) v[k].z = 0.f;
+      if (i + 3 >= n) v[k].w = 0.f;
+      q += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+  }
+  const float s = 1.0f / sqrtf(warp_sum(q) / n + eps);
+#pragma unroll
+  for (int k = 0; k < kWarpPieces; ++k) {
+    const int i = 4 * (lane + 32 * k);
+    if (i >= n) break;
+    const float4 g = load4(w + i, n - i);
+    store4(out + i, make_float4(v[k].x * s * g.x, v[k].y * s * g.y, v[k].z * s * g.z, v[k].w * s * g.w));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_post_warp_kernel(ds41_latent_post_args p) {
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  if (r >= p.rows) return;
+  if (blockIdx.y == 0) {
+    norm_row_warp(p.dq, r, p.q_rank, p.dq_norm, p.eps, static_cast<T*>(p.cq) + 1ll * r * p.ld_cq);
+    return;
+  }
+  const int slot = p.row_slot[r], pos = p.row_pos[r];
+  if (slot < 0) return;
+  T* row = cache_row(static_cast<T*>(p.pool), p.page_table, p.max_pages, p.page_tokens, p.row_len, slot, pos);
+  if (row == nullptr) return;
+  for (int i = lane; i < p.rot_dim / 2; i += 32) {
+    float a, b;
+    rotate_pair(proj_at(p.kr, r, 2 * i), proj_at(p.kr, r, 2 * i + 1), pos, p.freq[i], p.magnitude, a, b);
+    row[p.kv_pad + 2 * i] = from_f32<T>(a);
+    row[p.kv_pad + 2 * i + 1] = from_f32<T>(b);
+  }
+  norm_row_warp(p.kv, r, p.kv_rank, p.kv_norm, p.eps, row);
+}
+
 // In place when q is the projection itself (q.data == out): then only the rotated parts change.  A block's heads share the
 // sines and cosines of its row.
 constexpr int kMaxTurns = 256;         // pairs whose sine and cosine are kept per block
@@ -120,7 +172,8 @@ __global__ void __launch_bounds__(256) latent_query_kernel(ds41_proj q, const in
   const int first = in_place ? dim_pad : 0;
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < heads * half; i += gridDim.x * blockDim.x) {
     const int h = i / half, j = 2 * (i - h * half) + first, c = h * hs + j;
-    float a = proj_at(q, r, c), b = proj_at(q, r, c + 1);
+    const float2 ab = proj_at2(q, r, c);
+    float a = ab.x, b = ab.y;
     const int t = j - dim_pad;
     if (t >= 0 && t < rot_dim) {
       const float2 cs = turn[t / 2];
@@ -128,8 +181,7 @@ __global__ void __launch_bounds__(256) latent_query_kernel(ds41_proj q, const in
       a = u * cs.x - v * cs.y;
       b = v * cs.x + u * cs.y;
     }
-    out[1ll * r * ld_out + c] = from_f32<T>(a);
-    out[1ll * r * ld_out + c + 1] = from_f32<T>(b);
+    store2(out + 1ll * r * ld_out + c, a, b);
   }
 }
 
@@ -520,6 +572,11 @@ extern "C" int ds41_latent_post(const ds41_latent_post_args* a, void* stream) {
     return cudaErrorInvalidValue;
   const dim3 grid(a->rows, kv ? 2 : 1);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a->rows >= 256 && a->q_rank <= 128 * kWarpPieces && (!kv || a->kv_rank <= 128 * kWarpPieces)) {
+    const dim3 warps((a->rows + 7) / 8, kv ? 2 : 1);
+    return a->f32 ? launch_pdl(latent_post_warp_kernel<float>, warps, dim3(256), 0, st, *a)
+                  : launch_pdl(latent_post_warp_kernel<__nv_bfloat16>, warps, dim3(256), 0, st, *a);
+  }
   return a->f32 ? launch_pdl(latent_post_kernel<float>, grid, dim3(256), 0, st, *a)
                 : launch_pdl(latent_post_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, *a);
 }
@@ -531,6 +588,7 @@ extern "C" int ds41_latent_query(const ds41_proj* q, const int* row_pos, const f
       dim_pad < 0 || (dim_pad & 1) || (rot_pad & 1) || (rot_dim & 1) || rot_dim > rot_pad || rot_dim > 2 * kMaxTurns || out == nullptr ||
       ld_out < heads * (dim_pad + rot_pad))
     return cudaErrorInvalidValue;
+  if ((q->ld & 1) || (q->col & 1) || (q->plane & 1) || (ld_out & 1)) return cudaErrorInvalidValue;
   const int in_place = q->data == out ? 1 : 0;
   if (in_place && ((f32 != 0) == (q->bf16 != 0) || q->splits != 1 || q->col != 0 || q->ld != ld_out)) return cudaErrorInvalidValue;
   if (in_place && rot_pad == 0) return cudaSuccess;

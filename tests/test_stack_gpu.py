@@ -547,6 +547,37 @@ def test_cache_rows_and_queries_are_normed_and_turned():
     torch.testing.assert_close(out.cpu().double().view(rows, 2, 20), want, rtol=1e-4, atol=1e-4)
 
 
+@pytest.mark.parametrize("rows", [5, 300])
+def test_latent_norms_of_odd_widths(rows):
+    """Both forms of the kernel (one block or one warp per row), widths that end inside a vector."""
+    lib, S, k = _stack()
+    g, Q, K, R = gen(rows), 1030, 523, 6
+    x = torch.randn(2, rows, 1032 + 528 + 8, generator=g)
+    nq, nk = torch.rand(Q, generator=g) + 0.5, torch.rand(K, generator=g) + 0.5
+    X, NQ, NK, freq = x.cuda(), nq.cuda(), nk.cuda(), torch.tensor([1.0, 0.3, 0.01]).cuda()
+    n_pages = -(-rows // 64)
+    cq, pool = torch.zeros(rows, 1032).cuda(), torch.zeros(n_pages * 64, 528 + 16).cuda()
+    pos, slot = torch.arange(rows, dtype=torch.int32).cuda(), torch.zeros(rows, dtype=torch.int32).cuda()
+    table = torch.arange(n_pages - 1, -1, -1, dtype=torch.int32).view(1, -1).contiguous().cuda()
+    pin = S.Proj(X, x.shape[2], 2, rows * x.shape[2])
+    a = S.LatentPostArgs()
+    a.dq, a.kv, a.kr = pin.args(), pin.at(1032).args(), pin.at(1560).args()
+    a.dq_norm, a.kv_norm, a.freq, a.cq, a.pool = (lib.ptr(t) for t in (NQ, NK, freq, cq, pool))
+    a.page_table, a.row_pos, a.row_slot, a.magnitude, a.eps = lib.ptr(table), lib.ptr(pos), lib.ptr(slot), 1.0, 1e-5
+    a.rows, a.q_rank, a.ld_cq, a.kv_rank, a.kv_pad, a.rot_dim, a.row_len = rows, Q, 1032, K, 528, R, 544
+    a.max_pages, a.page_tokens, a.f32 = n_pages, 64, 1
+    _ok(k.ds41_latent_post(C.byref(a), lib.stream()))
+    d = x.double().sum(0)
+    got = pool.cpu().double().view(n_pages, 64, 544).flip(0).reshape(-1, 544)[:rows]
+    torch.testing.assert_close(cq[:, :Q].cpu().double(), rms_unit(d[:, :Q], 1e-5) * nq, rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(got[:, :K], rms_unit(d[:, 1032:1032 + K], 1e-5) * nk, rtol=1e-5, atol=1e-5)
+    ang = torch.arange(rows).double()[:, None] * freq.cpu().double()
+    u, v = d[:, 1560:1566:2], d[:, 1561:1566:2]
+    want = torch.stack([u * ang.cos() - v * ang.sin(), v * ang.cos() + u * ang.sin()], -1).flatten(1)
+    torch.testing.assert_close(got[:, 528:534], want, rtol=1e-4, atol=1e-4)
+    assert not got[:, 534:].any() and not got[:, K:528].any()
+
+
 class Recurrence:
     def __init__(self, T, heads, dim, vdim, cap=6.0, seed=0, dtype=F32):
         g = gen(seed)
