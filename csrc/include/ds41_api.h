@@ -14,7 +14,8 @@ extern "C" {
 //   kind      0 bf16, 1 fp8-e4m3 (unscaled), 2 MX fp8 (UE8M0 per 32 elements; scale atoms sfa/sfb)
 //   out_mode  0 bf16 [m,n] | 1 f32 [m,n] | 2 bf16 [n,m] | 3 f32 [n,m]
 //             4 bf16 [n,m] = silu(min(gate,L)) * clamp(up,-L,L) * row_w[b][n] with gate = A rows [m],
-//               up = A rows [up_row_offset + m]   (fused expert FC1)
+//               up = A rows [up_row_offset + m]   (fused expert FC1); with act_alpha != 0 instead
+//               g * sigmoid(act_alpha g) * (u + act_shift) * row_w, g and u clamped fp32 accumulators
 //             5 f32 [n,m] written only where row_w[b][n] != 0 (expert FC2)
 //   k_splits  > 1 writes fp32 planes [split][batch][rows][ldo] into split_workspace (modes 1 and 3)
 //   batch_map / n_active: grouped execution - logical batch b uses A batch batch_map[b]; only b < *n_active run
@@ -91,6 +92,8 @@ typedef struct ds41_gemm_args {
   unsigned int* sig_epoch;
   unsigned int* const* sig_flags;
   int sig_world;
+  float act_alpha, act_shift;   // mode 4: the other activation (0: silu on bf16-rounded values)
+  float softcap;                // modes 1 and 3 without split K: out = softcap * tanh(acc / softcap) (0: acc)
 } ds41_gemm_args;
 
 int ds41_gemm_tc(const ds41_gemm_args* args, void* stream);
@@ -434,7 +437,7 @@ int ds41_act_quant_nvfp4_rows(const void* x, long long ldx, void* q, long long l
                               long long q_batch_stride, long long sf_batch_stride, const int* n_active, void* stream);
 
 // ---------------------------------------------------------------------------------------------------
-// Layer stacks with one fp32 residual stream (stack_ops.cu, latent_attn.cu, mlstm.cu, gemm_f32.cu).  `f32` selects 32-bit
+// Layer stacks with one fp32 residual stream (stack_ops.cu, latent_attn.cu, group_attn.cu, mlstm.cu, gemm_f32.cu).  `f32` selects 32-bit
 // activations, cache rows and weights; 0 = bf16 (the streams, norms, gates, scores and recurrent states are fp32 in both).
 //
 // A projection as its consumer reads it: columns [col, ...) of `splits` fp32 planes [rows][ld] (split-K partial sums), or
@@ -468,6 +471,12 @@ typedef struct ds41_resid_args {
   int norm_kind;        // 0 layer norm without bias, 1 RMS norm
   float eps;
   int f32;
+  // The result of routed experts: y = sum over k < y_top of the y rows that y_route[r][k] names (negative: none) - row
+  // route * y_rows + r where y_rows > 0 (one plane of y_rows rows per expert), else row r * y_top + k (one per route).
+  const int* y_route;
+  int y_top, y_rows;
+  int raw_h;            // next_w == NULL: h = the stream itself
+  int post_rms;         // the norm of the result is an RMS norm whatever norm_kind says
 } ds41_resid_args;
 int ds41_resid_step(const ds41_resid_args* args, void* stream);
 
@@ -479,6 +488,12 @@ int ds41_gate_mul(const ds41_proj* y, const ds41_proj* gate, int rows, int n, vo
 // heads of `stride` columns, `width` of them live: o / rms(o) * w * sigmoid(gate)
 int ds41_head_norm_gate(const float* o, int ld_o, const ds41_proj* gate, const float* w, int rows, int heads, int width,
                         int stride, float eps, void* out, int ld_out, int f32, void* stream);
+// out[r][j] = gelu_tanh(z[r][j]) * embed[token[r]][col + j], j < n (bf16 table; tokens outside it read as zeros); columns
+// up to ld_out are written as zeros
+int ds41_side_act(const ds41_proj* z, const int* tokens, const void* embed, long long embed_ld, int col, int vocab, int rows,
+                  int n, void* out, int ld_out, int f32, void* stream);
+// x = cap * tanh(x / cap), in place
+int ds41_softcap_rows(float* x, long long n, float cap, void* stream);
 int ds41_gather_rows(const void* src, int ld, const int* index, int n_src, int rows, int W, void* dst, int f32,
                      void* stream);
 
@@ -553,9 +568,75 @@ int ds41_mlstm_step(const ds41_mlstm_args* args, void* stream);
 int ds41_mlstm_chunk(const ds41_mlstm_args* args, void* stream);
 long long ds41_mlstm_chunk_work(int rows, int heads, int dim_pad, int vdim_pad);
 
+// Attention with grouped query heads (group_attn.cu, group_prefill.cu).  A cache row is [keys of all key/value heads | values
+// of all key/value heads], heads padded to dim_pad / vdim_pad; `chunk` > 0 restricts a position to its own chunk of that many
+// positions.  The last taps - 1 inputs of the convolution stay in a ring per slot: position p at p % (taps - 1).
+typedef struct ds41_attn_post_args {
+  ds41_proj u;                    // projected [q | k | v]: heads * dim_pad, kv_heads * dim_pad, kv_heads * vdim_pad columns
+  const float* conv;              // [taps][columns of u], newest last; NULL (taps = 1): no convolution
+  const float* q_norm;            // [heads * dim_pad], zero in the padding; NULL: no norm
+  const float* k_norm;
+  const float* freq;              // [rot_dim / 2] rotation per position
+  const float* state;             // [slots][taps - 1][columns of u]
+  void* q;                        // [rows][ld_q]
+  void* pool;
+  const int* page_table;
+  const int* row_pos;
+  const int* row_slot;
+  long long ld_q;
+  float eps;
+  int rows, heads, kv_heads, dim, dim_pad, vdim_pad, rot_dim, taps, slots, max_pages, page_tokens, f32;
+} ds41_attn_post_args;
+int ds41_attn_post(const ds41_attn_post_args* args, void* stream);
+
+typedef struct ds41_group_attend_args {
+  const void* q;                  // [rows][ld_q]: head h at h * dim_pad
+  const void* pool;
+  const int* page_table;
+  const int* row_pos;
+  const int* row_slot;
+  void* out;                      // [rows][ld_out]: head h at h * vdim_pad
+  int* status;
+  ds41_proj gate;                 // one column per head (absent: no gate): output * sigmoid
+  ds41_proj u;                    // taps > 1: this pass's inputs of the convolution, whose last taps - 1 rows per request
+  float* state;                   //   go into the ring
+  long long ld_q;
+  float scale;
+  int rows, heads, kv_heads, dim_pad, vdim_pad, chunk, taps, slots, n_splits, ld_out, max_pages, page_tokens, f32;
+  int n_pages, pos0;              // long passes: pages of the pool, position of row 0
+} ds41_group_attend_args;
+// Any mix of rows; n_splits <= 8 CTAs share a row's keys.
+int ds41_group_attend(const ds41_group_attend_args* args, void* stream);
+// Long prompt pass of one request (bf16, dim_pad <= 256, vdim_pad <= 128, pages of 32, 64 or 128 tokens): row r stands at
+// position pos0 + r.
+int ds41_group_prefill(const ds41_group_attend_args* args, void* stream);
+
+// Router of a layer stack: logits z (+ bias), the `top` largest (lowest index wins ties), weights = softmax over those.
+// Rows without a slot get ids of -1.  With `active` the launch also plans the experts of a small pass: ascending list of
+// used experts, row_w [max_active][row_w_ld] and slot_of [rows][top] (-1: not routed, or a weight of zero); `ticket` is a
+// zeroed device word, left at zero again.
+typedef struct ds41_route_args {
+  ds41_proj z;
+  const float* bias;
+  const int* row_slot;
+  int* ids;                       // [rows][top]
+  float* weights;                 // [rows][top]
+  int* active;
+  int* n_active;
+  float* row_w;
+  int* slot_of;
+  unsigned int* ticket;
+  int rows, experts, top, max_active, row_w_ld;
+} ds41_route_args;
+int ds41_route_softmax(const ds41_route_args* args, void* stream);
+// 32-bit experts: act[b][r][j] = g sigmoid(alpha g) (u + shift) row_w[b][r], gate / up at columns j and up_col + j of x
+int ds41_gated_act(const float* x, int ld_x, int up_col, const float* row_w, int row_w_ld, const int* n_active, int batch,
+                   int rows, int n, float limit, float alpha, float shift, float* act, int ld_act, void* stream);
+
+// batch_map / n_active (optional): batch b multiplies B batch batch_map[b]; only b < *n_active run
 int ds41_gemm_f32(const float* A, const float* B, float* out, int M, int N, int K, long long lda, long long ldb,
                   long long ldo, int batch, long long a_batch_stride, long long b_batch_stride,
-                  long long out_batch_stride, void* stream);
+                  long long out_batch_stride, const int* batch_map, const int* n_active, void* stream);
 
 #ifdef __cplusplus
 }

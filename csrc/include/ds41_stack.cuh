@@ -1,4 +1,4 @@
-// Shared device helpers of the layer-stack kernels (stack_ops.cu, latent_attn.cu, mlstm.cu).
+// Shared device helpers of the layer-stack kernels (stack_ops.cu, latent_attn.cu, group_attn.cu, mlstm.cu).
 #pragma once
 #include "ds41_api.h"
 #include "ds41_launch.cuh"
@@ -103,6 +103,17 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   }
   __syncthreads();
   return red[32];
+}
+
+// Cache row of position `pos` of a request, or null when its page is not leased.
+template <typename T>
+__device__ __forceinline__ T* cache_row(T* pool, const int* page_table, int max_pages, int page_tokens, int row_len,
+                                        int slot, int pos) {
+  const int pg = pos / page_tokens;
+  if (pg < 0 || pg >= max_pages) return nullptr;
+  const int id = page_table[1ll * slot * max_pages + pg];
+  if (id < 0) return nullptr;
+  return pool + (1ll * id * page_tokens + (pos - pg * page_tokens)) * row_len;
 }
 
 // First row of a run of rows that belong to one request (rows of one request are adjacent and in order).

@@ -58,6 +58,9 @@ struct GemmParams {
   const float* row_w;     // modes 4/5: per (logical batch, n) weight, [batch][row_w_ld]
   int row_w_ld;
   float act_limit;        // mode 4: SwiGLU clamp
+  float act_alpha;        // mode 4: != 0 selects g sigmoid(alpha g) (u + shift) on unrounded values
+  float act_shift;
+  float softcap;          // modes 1 and 3: cap * tanh(acc / cap)
   int static_operand;     // 1: A holds weights, 2: B holds weights (may be fetched before the dependency wait)
   float alpha;            // kind 3: product of the two tensors' global scales, applied to the accumulators
   const float* alpha_batch;   // optional extra factor per A batch (one global scale per expert)
@@ -470,6 +473,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #pragma unroll
           for (int j = 0; j < kChunk; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * alpha);
         }
+        if constexpr (KIND == 0 && !DUAL) {
+          if (p.softcap > 0.f) {
+#pragma unroll
+            for (int j = 0; j < kChunk; ++j) v[j] = __float_as_uint(p.softcap * tanhf(__uint_as_float(v[j]) / p.softcap));
+          }
+        }
         const int n0 = n_base + c;
         const float rw_lane = rw_next;
         const int2 meta_lane = meta_next;
@@ -555,9 +564,16 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             for (int j = 0; j < kChunk; ++j) {
               const float rwj = __shfl_sync(0xffffffffu, rw_lane, j);
               if (m < p.M && n0 + j < n_lim) {
-                const float gte = fminf(bf16_round(__uint_as_float(v[j])), p.act_limit);
-                const float upv = fminf(fmaxf(bf16_round(__uint_as_float(u[j])), -p.act_limit), p.act_limit);
-                const float act = gte / (1.0f + __expf(-gte)) * upv * rwj;
+                float act;
+                if (p.act_alpha == 0.f) {
+                  const float gte = fminf(bf16_round(__uint_as_float(v[j])), p.act_limit);
+                  const float upv = fminf(fmaxf(bf16_round(__uint_as_float(u[j])), -p.act_limit), p.act_limit);
+                  act = gte / (1.0f + __expf(-gte)) * upv * rwj;
+                } else {
+                  const float gte = fminf(__uint_as_float(v[j]), p.act_limit);
+                  const float upv = fminf(fmaxf(__uint_as_float(u[j]), -p.act_limit), p.act_limit) + p.act_shift;
+                  act = gte / (1.0f + __expf(-p.act_alpha * gte)) * upv * rwj;
+                }
                 o[1ll * (n0 + j) * p.ldo] = __float2bfloat16_rn(act);
               }
             }
@@ -829,6 +845,7 @@ extern "C" int ds41_gemm_tc(const ds41_gemm_args* a, void* stream) {
     return cudaErrorInvalidValue;
   if (kind == 2 && bn < 32 && N > bn) return cudaErrorInvalidValue;      // 16-row scale tiles cannot be lane-shifted
   if (k_splits > 1 && out_mode != 1 && out_mode != 3) return cudaErrorInvalidValue;   // partials are fp32
+  if (a->softcap < 0.f || (a->softcap > 0.f && (kind != 0 || k_splits > 1 || (out_mode != 1 && out_mode != 3)))) return cudaErrorInvalidValue;
   if ((out_mode == 4 || out_mode == 5 || out_mode == 8) && a->row_w == nullptr) return cudaErrorInvalidValue;
   if (out_mode == 8 && (bn < 32 || (M & 31) != 0 || k_splits != 1)) return cudaErrorInvalidValue;
   if (out_mode == 7 && (a->scatter_meta == nullptr || a->tile_group == nullptr || (a->ldo & 7) != 0))
@@ -927,6 +944,9 @@ extern "C" int ds41_gemm_tc(const ds41_gemm_args* a, void* stream) {
   p.row_w = a->row_w;
   p.row_w_ld = a->row_w_ld;
   p.act_limit = a->act_limit;
+  p.act_alpha = a->act_alpha;
+  p.act_shift = a->act_shift;
+  p.softcap = a->softcap;
   p.tile_group = a->tile_group; p.tile_row0 = a->tile_row0; p.tile_end = a->tile_end; p.n_tiles_dev = a->n_tiles_dev;
   p.wait_flags = reinterpret_cast<const uint32_t* const*>(a->wait_flags);
   p.wait_epoch = reinterpret_cast<const uint32_t*>(a->wait_epoch);

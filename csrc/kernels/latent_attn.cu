@@ -22,17 +22,6 @@ __device__ __forceinline__ void rotate_pair(float u, float v, int pos, float fre
   rv = v * c + u * s;
 }
 
-// Cache row of position `pos` of a request, or null when its page is not leased.
-template <typename T>
-__device__ __forceinline__ T* cache_row(T* pool, const int* page_table, int max_pages, int page_tokens, int row_len,
-                                        int slot, int pos) {
-  const int pg = pos / page_tokens;
-  if (pg < 0 || pg >= max_pages) return nullptr;
-  const int id = page_table[1ll * slot * max_pages + pg];
-  if (id < 0) return nullptr;
-  return pool + (1ll * id * page_tokens + (pos - pg * page_tokens)) * row_len;
-}
-
 // RMS norm of `n` columns of a projection row into `out` (columns up to the next multiple of four are written as zeros).
 // The row stays in registers while it is short (kHeld pieces per thread).
 template <typename T>

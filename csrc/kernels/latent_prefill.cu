@@ -1,332 +1,67 @@
 // Causal attention of a long prompt pass over expanded keys and values: one request, adjacent rows.
 //
-// Head h's key is [K row: dim values | rotated part shared by all heads], its value a V row.  One CTA owns two tiles of 128
-// query rows of one head and walks the keys 128 at a time; both tiles share every key / value tile.
-//   warps 0-3, 4-7 : softmax of tile 0 / 1 (one thread per query row), output epilogue
-//   warp 8         : TMA producer (Q once, then K and V tiles into stage rings)
-//   warp 9         : tcgen05.mma issue: S = Q K^T into TMEM, O += P V with P read from TMEM where it replaces its S
-// While one tile's warps work on its softmax the tensor core runs the other tile's products.  The running maximum is only
-// raised when it grew by more than 2^8, so the accumulated output is rarely rescaled.  The softmax denominator contains
-// exp(sink) of the head; the output is multiplied by the sigmoid of its gate row before it leaves.
-#include <cuda.h>
-
-#include "ds41_stack.cuh"
-#include "ds41_tma.h"
+// Head h's key is [K row: dim values | rotated part shared by all heads], its value a V row; the two query tiles of a CTA are
+// neighbouring tiles of one head (ds41_prompt_attend.cuh).  The softmax denominator contains exp(sink) of the head; the
+// output is multiplied by the sigmoid of its gate row before it leaves.
+#include "ds41_prompt_attend.cuh"
 
 namespace ds41 {
 
-constexpr int kPreThreads = 320;
-constexpr int kPreTile = 128;                  // query rows per tile, keys per tile
-constexpr int kPreChunk = kPreTile * 128;      // bytes of 128 rows x 64 bf16 columns
+struct LatentForm {
+  CUtensorMap q, kv, rot;
+  const float* sinks;
+  ds41_proj gates;
+  static constexpr bool kLowerBound = false;
 
-struct PrefillParams {
-  int rows, heads, dp, rp, vp, n_keys, pos0;
-  int kd, kr, vc;            // 64-column chunks of the unrotated part, the rotated part and the value
-  int k_stages, v_stages;
-  float scale_log2;          // scale * log2(e)
-  const float* sink;
-  ds41_proj gate;
-  __nv_bfloat16* out;
-  int ld_out;
-  int* status;
-};
-
-__device__ __forceinline__ void drain_barrier(uint64_t* bar, uint32_t parity) {
-  for (int i = 0; i < (1 << 20) && !mbar_test_wait(bar, parity); ++i) {
-  }
-}
-
-__global__ void __launch_bounds__(kPreThreads, 1)
-latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
-                      const __grid_constant__ CUtensorMap tm_rot, const PrefillParams p) {
-  extern __shared__ uint8_t smem_raw[];
-  const uint32_t raw = smem_u32(smem_raw);
-  uint8_t* smem = smem_raw + ((1024u - (raw & 1023u)) & 1023u);
-  const int qk_chunks = p.kd + p.kr;
-  const int q_bytes = qk_chunks * kPreChunk, k_bytes = q_bytes, v_bytes = p.vc * kPreChunk;
-  uint8_t* s_q = smem;                                   // two tiles
-  uint8_t* s_k = s_q + 2 * q_bytes;
-  uint8_t* s_v = s_k + p.k_stages * k_bytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_v + p.v_stages * v_bytes);
-  uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;        // [2]
-  uint64_t* k_empty = bars + 3;
-  uint64_t* v_full = bars + 5;
-  uint64_t* v_empty = bars + 7;
-  uint64_t* s_full = bars + 9;        // [2] per tile: S complete (and every earlier MMA of the issuing thread)
-  uint64_t* p_full = bars + 11;       // [2] per tile: P written, O rescaled
-  uint64_t* o_full = bars + 13;       // [2] per tile
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-
-  const int n_pairs = (p.rows + 2 * kPreTile - 1) / (2 * kPreTile);
-  const int h = blockIdx.x % p.heads;
-  const int pair = n_pairs - 1 - static_cast<int>(blockIdx.x) / p.heads;      // the longest walks first
-  const int q0 = pair * 2 * kPreTile;
-  // key tiles that tile t's rows see
-  int n_t[2];
+  __device__ PromptTiles tiles(const PromptParams& p, int block) const {
+    PromptTiles t;
+    const int n_pairs = (p.rows + 2 * kPreTile - 1) / (2 * kPreTile);
+    const int pair = n_pairs - 1 - block / p.heads;                           // the longest walks first
+    t.key0 = 0;
 #pragma unroll
-  for (int t = 0; t < 2; ++t) {
-    const int first = q0 + t * kPreTile;
-    const int last = min(first + kPreTile, p.rows) - 1;
-    n_t[t] = first < p.rows ? min((p.pos0 + last) / kPreTile + 1, (p.n_keys + kPreTile - 1) / kPreTile) : 0;
-  }
-  const int n = max(n_t[0], n_t[1]);
-
-  pdl_launch_dependents();
-  if (threadIdx.x == 0) {
-    mbar_init(q_full, 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&k_full[i], 1);
-      mbar_init(&k_empty[i], 1);
-      mbar_init(&v_full[i], 1);
-      mbar_init(&v_empty[i], 1);
-      mbar_init(&s_full[i], 1);
-      mbar_init(&p_full[i], kPreTile);
-      mbar_init(&o_full[i], 1);
+      t.head[i] = block % p.heads;
+      t.row0[i] = (2 * pair + i) * kPreTile;
+      const int last = min(t.row0[i] + kPreTile, p.rows) - 1;
+      t.n[i] = t.row0[i] < p.rows ? min((p.pos0 + last) / kPreTile + 1, (p.n_keys + kPreTile - 1) / kPreTile) : 0;
     }
-    mbar_init_fence();
+    return t;
   }
-  if (warp == 9) {
-    tmem_alloc(tmem_slot, 512);
-    tmem_relinquish();
+  __device__ void prefetch() const {
+    tma_prefetch_desc(&q);
+    tma_prefetch_desc(&kv);
   }
-  tc_fence_before();
-  __syncthreads();
-  tc_fence_after();
-  const uint32_t tmem = *tmem_slot;
-  pdl_wait();
-
-  if (warp == 8) {
-    if (lane == 0) {
-      tma_prefetch_desc(&tm_q);
-      tma_prefetch_desc(&tm_kv);
-      const int tiles = n_t[1] > 0 ? 2 : 1;
-      mbar_expect_tx(q_full, tiles * q_bytes);
-      const int qx = h * (p.dp + p.rp);
-      for (int t = 0; t < tiles; ++t) {
-        for (int c = 0; c < p.kd; ++c)
-          tma_load_3d(s_q + t * q_bytes + c * kPreChunk, &tm_q, q_full, qx + 64 * c, q0 + t * kPreTile, 0);
-        for (int c = 0; c < p.kr; ++c)
-          tma_load_3d(s_q + t * q_bytes + (p.kd + c) * kPreChunk, &tm_q, q_full, qx + p.dp + 64 * c, q0 + t * kPreTile, 0);
-      }
-      bool ok = true;
-      const int vx = p.heads * p.dp + h * p.vp;
-      int j = 0;
-      for (; j < n && ok; ++j) {
-        const int ks = j % p.k_stages, vs = j % p.v_stages;
-        ok = mbar_wait(&k_empty[ks], ((j / p.k_stages) & 1) ^ 1, p.status, 400);
-        if (!ok) break;
-        mbar_expect_tx(&k_full[ks], k_bytes);
-        uint8_t* k = s_k + ks * k_bytes;
-        for (int c = 0; c < p.kd; ++c) tma_load_3d(k + c * kPreChunk, &tm_kv, &k_full[ks], h * p.dp + 64 * c, j * kPreTile, 0);
-        for (int c = 0; c < p.kr; ++c)
-          tma_load_3d(k + (p.kd + c) * kPreChunk, &tm_rot, &k_full[ks], 64 * c, j * kPreTile, 0);
-        ok = mbar_wait(&v_empty[vs], ((j / p.v_stages) & 1) ^ 1, p.status, 401);
-        if (!ok) {
-          drain_barrier(&k_full[ks], (j / p.k_stages) & 1);
-          break;
-        }
-        mbar_expect_tx(&v_full[vs], v_bytes);
-        for (int c = 0; c < p.vc; ++c) tma_load_3d(s_v + vs * v_bytes + c * kPreChunk, &tm_kv, &v_full[vs], vx + 64 * c, j * kPreTile, 0);
-      }
-      if (!ok) {
-        // something else gave up: let the copies of the last tiles land before the shared memory goes away
-        drain_barrier(q_full, 0);
-        for (int b = max(0, j - 2); b < j; ++b) {
-          drain_barrier(&k_full[b % p.k_stages], (b / p.k_stages) & 1);
-          drain_barrier(&v_full[b % p.v_stages], (b / p.v_stages) & 1);
-        }
-      }
-    }
-  } else if (warp == 9) {
-    const bool leader = elect_one();
-    const uint32_t idesc_s = umma_idesc(kPreTile, kPreTile, 1u, 1u);
-    const uint32_t idesc_pv = umma_idesc_bmn(kPreTile, p.vp, 1u, 1u);
-    const uint64_t q_desc = umma_desc_sw128(smem_u32(s_q)), k_desc = umma_desc_sw128(smem_u32(s_k));
-    const uint64_t v_desc = umma_desc_sw128_mn(smem_u32(s_v), kPreChunk, 1024);
-    const int kd16 = p.dp / 16, kr16 = p.rp / 16;
-    auto wait = [&](uint64_t* bar, uint32_t parity, int where) {
-      const bool ok = mbar_wait(bar, parity, p.status, where);
-      return __all_sync(0xffffffffu, ok) != 0;
-    };
-    auto issue_s = [&](int t, int stage) {
-      const uint64_t qd = q_desc + static_cast<uint64_t>(t * q_bytes / 16), kd = k_desc + static_cast<uint64_t>(stage * k_bytes / 16);
-      for (int k = 0; k < kd16; ++k) {
-        const uint64_t off = static_cast<uint64_t>((k >> 2) * (kPreChunk / 16) + (k & 3) * 2);
-        umma_bf16_if(leader, tmem + t * 128, qd + off, kd + off, idesc_s, k > 0 ? 1u : 0u);
-      }
-      for (int k = 0; k < kr16; ++k) {
-        const uint64_t off = static_cast<uint64_t>((p.kd + (k >> 2)) * (kPreChunk / 16) + (k & 3) * 2);
-        umma_bf16_if(leader, tmem + t * 128, qd + off, kd + off, idesc_s, kd16 + k > 0 ? 1u : 0u);
-      }
-      tc_commit_if(leader, &s_full[t]);
-    };
-    auto issue_pv = [&](int t, int stage, bool first) {
-      const uint64_t vd = v_desc + static_cast<uint64_t>(stage * v_bytes / 16);
-#pragma unroll
-      for (int k = 0; k < kPreTile / 16; ++k)
-        umma_bf16_ts_if(leader, tmem + 256 + t * 128, tmem + t * 128 + 8 * k, vd + 128 * k, idesc_pv, first && k == 0 ? 0u : 1u);
-    };
-    bool ok = wait(q_full, 0, 410) && wait(&k_full[0], 0, 411);
-    if (ok) {
-      tc_fence_after();
-      issue_s(0, 0);
-      if (n_t[1] > 0) issue_s(1, 0);
-      tc_commit_if(leader, &k_empty[0]);
-    }
-    for (int j = 0; j < n && ok; ++j) {
-      const int vs = j % p.v_stages, ks = (j + 1) % p.k_stages;
-      ok = wait(&v_full[vs], (j / p.v_stages) & 1, 412);
-      if (ok && j + 1 < n) ok = wait(&k_full[ks], ((j + 1) / p.k_stages) & 1, 413);
-      if (!ok) break;
-#pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        if (j < n_t[t]) {
-          if (ok) ok = wait(&p_full[t], j & 1, 414 + t);
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(t, vs, j == 0);
-          if (j == n_t[t] - 1) tc_commit_if(leader, &o_full[t]);
-        }
-        if (t == 1) tc_commit_if(leader, &v_empty[vs]);
-        if (j + 1 < n_t[t]) issue_s(t, ks);
-      }
-      if (ok && j + 1 < n) tc_commit_if(leader, &k_empty[ks]);
-    }
-  } else {
-    const int t = warp >> 2, quad = warp & 3;
-    const int row = q0 + t * kPreTile + quad * 32 + lane;
-    const int pos = p.pos0 + row, warp_pos = p.pos0 + q0 + t * kPreTile + quad * 32;
-    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
-    const uint32_t s_t = tmem + lanes + t * 128, o_t = tmem + lanes + 256 + t * 128;
-    float m = -INFINITY, l = 0.f;
-    bool ok = true;
-    for (int j = 0; j < n_t[t] && ok; ++j) {
-      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[t], j & 1, p.status, 420 + t)) != 0;
-      if (!ok) break;
-      tc_fence_after();
-      const int key0 = j * kPreTile;
-      const bool edge = key0 + kPreTile - 1 > warp_pos;
-      const int seen = pos - key0;                       // columns [0, seen] of this tile are visible
-      float top = -INFINITY;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t v[32];
-        tmem_ld_32x32(s_t + 32 * c, v);
-        tmem_wait_ld();
-        if (edge) {
-#pragma unroll
-          for (int i = 0; i < 32; ++i)
-            if (32 * c + i <= seen) top = fmaxf(top, __uint_as_float(v[i]) * p.scale_log2);
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) top = fmaxf(top, __uint_as_float(v[i]) * p.scale_log2);
-        }
-      }
-      const bool grow = top > m + 8.f || (m == -INFINITY && top > m);
-      if (__any_sync(0xffffffffu, grow)) {
-        const float m_new = grow ? top : m;
-        const float alpha = m == -INFINITY ? 0.f : ex2_approx(m - m_new);
-        l *= alpha;
-        m = m_new;
-        if (j > 0) {
-          const float keep = grow ? alpha : 1.f;
-          for (int c = 0; c < p.vp; c += 16) {
-            uint32_t o[16];
-            tmem_ld_32x16(o_t + c, o);
-            tmem_wait_ld();
-#pragma unroll
-            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * keep);
-            tmem_st_32x16(o_t + c, o);
-          }
-        }
-      }
-      const float neg = m == -INFINITY ? 0.f : -m;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t v[32], w[16];
-        tmem_ld_32x32(s_t + 32 * c, v);
-        tmem_wait_ld();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          float a = ex2_approx(fmaf(__uint_as_float(v[2 * i]), p.scale_log2, neg));
-          float b = ex2_approx(fmaf(__uint_as_float(v[2 * i + 1]), p.scale_log2, neg));
-          if (edge) {
-            a = 32 * c + 2 * i <= seen ? a : 0.f;
-            b = 32 * c + 2 * i + 1 <= seen ? b : 0.f;
-          }
-          l += a + b;
-          const __nv_bfloat162 q = __floats2bfloat162_rn(a, b);
-          w[i] = *reinterpret_cast<const uint32_t*>(&q);
-        }
-        tmem_st_32x16(s_t + 16 * c, w);                  // columns whose S this thread has read
-      }
-      tmem_wait_st();
-      tc_fence_before();
-      mbar_arrive(&p_full[t]);
-    }
-    if (ok && n_t[t] > 0) ok = __all_sync(0xffffffffu, mbar_wait(&o_full[t], 0, p.status, 430 + t)) != 0;
-    if (ok && n_t[t] > 0) {
-      tc_fence_after();
-      const float sink2 = p.sink != nullptr ? p.sink[h] * 1.4426950408889634f : -INFINITY;
-      const float m_fin = fmaxf(m, sink2);
-      const float w_o = m == -INFINITY ? 0.f : ex2_approx(m - m_fin);
-      const float den = l * w_o + (sink2 == -INFINITY ? 0.f : ex2_approx(sink2 - m_fin));
-      const float f = den > 0.f ? w_o / den : 0.f;
-      for (int c = 0; c < p.vp; c += 16) {
-        uint32_t o[16];
-        tmem_ld_32x16(o_t + c, o);
-        tmem_wait_ld();
-        if (row < p.rows) {
-          float g[16];
-          if (p.gate.data != nullptr) {
-            const long long at = 1ll * row * p.gate.ld + p.gate.col + h * p.vp + c;
-            if (p.gate.bf16) {
-              const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(static_cast<const __nv_bfloat16*>(p.gate.data) + at);
-#pragma unroll
-              for (int i = 0; i < 8; ++i) {
-                const float2 x = __bfloat1622float2(gp[i]);
-                g[2 * i] = x.x;
-                g[2 * i + 1] = x.y;
-              }
-            } else {
-              const float4* gp = reinterpret_cast<const float4*>(static_cast<const float*>(p.gate.data) + at);
-#pragma unroll
-              for (int i = 0; i < 4; ++i) {
-                const float4 x = gp[i];
-                g[4 * i] = x.x;
-                g[4 * i + 1] = x.y;
-                g[4 * i + 2] = x.z;
-                g[4 * i + 3] = x.w;
-              }
-            }
-          }
-          uint32_t w[8];
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            float a = __uint_as_float(o[2 * i]) * f, b = __uint_as_float(o[2 * i + 1]) * f;
-            if (p.gate.data != nullptr) {
-              a *= sigmoid_f32(g[2 * i]);
-              b *= sigmoid_f32(g[2 * i + 1]);
-            }
-            const __nv_bfloat162 q = __floats2bfloat162_rn(a, b);
-            w[i] = *reinterpret_cast<const uint32_t*>(&q);
-          }
-          uint4* dst = reinterpret_cast<uint4*>(p.out + 1ll * row * p.ld_out + h * p.vp + c);
-          dst[0] = make_uint4(w[0], w[1], w[2], w[3]);
-          dst[1] = make_uint4(w[4], w[5], w[6], w[7]);
-        }
-      }
-    }
-    tc_fence_before();
+  __device__ void load_q(const PromptParams& p, uint8_t* dst, uint64_t* bar, int h, int row0) const {
+    const int x = h * (p.dp + p.rp);
+    for (int c = 0; c < p.kd; ++c) tma_load_3d(dst + c * kPreChunk, &q, bar, x + 64 * c, row0, 0);
+    for (int c = 0; c < p.kr; ++c) tma_load_3d(dst + (p.kd + c) * kPreChunk, &q, bar, x + p.dp + 64 * c, row0, 0);
   }
-  __syncthreads();
-  if (warp == 9) {
-    tc_fence_after();
-    tmem_dealloc(tmem, 512);
+  __device__ void load_k(const PromptParams& p, uint8_t* dst, uint64_t* bar, int h, int key) const {
+    for (int c = 0; c < p.kd; ++c) tma_load_3d(dst + c * kPreChunk, &kv, bar, h * p.dp + 64 * c, key, 0);
+    for (int c = 0; c < p.kr; ++c) tma_load_3d(dst + (p.kd + c) * kPreChunk, &rot, bar, 64 * c, key, 0);
   }
-}
+  __device__ void load_v(const PromptParams& p, uint8_t* dst, uint64_t* bar, int h, int key) const {
+    const int x = p.heads * p.dp + h * p.vp;
+    for (int c = 0; c < p.vc; ++c) tma_load_3d(dst + c * kPreChunk, &kv, bar, x + 64 * c, key, 0);
+  }
+  __device__ int first_key(int) const { return 0; }
+  __device__ float sink(int h) const { return sinks != nullptr ? sinks[h] * 1.4426950408889634f : -INFINITY; }
+  __device__ void gate(const PromptParams& p, int row, int h, int c, float (&f)[16]) const {
+    if (gates.data == nullptr) {
+#pragma unroll
+      for (int i = 0; i < 16; ++i) f[i] = 1.f;
+      return;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float4 x = proj_at4(gates, row, h * p.vp + c + 4 * i);
+      f[4 * i] = sigmoid_f32(x.x);
+      f[4 * i + 1] = sigmoid_f32(x.y);
+      f[4 * i + 2] = sigmoid_f32(x.z);
+      f[4 * i + 3] = sigmoid_f32(x.w);
+    }
+  }
+};
 
 }  // namespace ds41
 
@@ -341,39 +76,28 @@ extern "C" int ds41_latent_prefill(const ds41_latent_prefill_args* a, void* stre
   if (a->gate.data != nullptr &&
       (a->gate.splits != 1 || (a->gate.ld & 7) || (a->gate.col & 7) || (reinterpret_cast<uintptr_t>(a->gate.data) & 15)))
     return cudaErrorInvalidValue;
-  PrefillParams p{};
+  PromptParams p{};
   p.rows = a->rows; p.heads = a->heads; p.dp = a->dim_pad; p.rp = a->rot_pad; p.vp = a->vdim_pad;
   p.n_keys = a->n_keys; p.pos0 = a->pos0;
-  p.kd = (p.dp + 63) / 64; p.kr = (p.rp + 63) / 64; p.vc = (p.vp + 63) / 64;
   p.scale_log2 = a->scale * 1.4426950408889634f;
-  p.sink = a->sink; p.gate = a->gate; p.out = static_cast<__nv_bfloat16*>(a->out); p.ld_out = a->ld_out;
+  p.out = static_cast<__nv_bfloat16*>(a->out); p.ld_out = a->ld_out;
   p.status = a->status;
-  const int qk = (p.kd + p.kr) * kPreChunk, v = p.vc * kPreChunk;
-  constexpr int kLimit = 226 * 1024 - 1024 - 256;
-  p.k_stages = p.v_stages = 1;
-  if (2 * qk + qk + v > kLimit) return cudaErrorInvalidValue;
-  if (2 * qk + 2 * qk + v <= kLimit) p.k_stages = 2;
-  if (2 * qk + p.k_stages * qk + 2 * v <= kLimit) p.v_stages = 2;
-  const int smem = 2 * qk + p.k_stages * qk + p.v_stages * v + 1024 + 256;
-  CUtensorMap tq, tkv, trot;
+  const int smem = prompt_smem(p);
+  if (smem == 0) return cudaErrorInvalidValue;
+  LatentForm f{};
+  f.sinks = a->sink;
+  f.gates = a->gate;
   const int hs = p.dp + p.rp;
-  cudaError_t e = make_tensor_map_3d(&tq, a->q, TmaDtype::kBF16, 1ull * p.heads * hs, p.rows, 1, a->ld_q * 2, 0, 64, kPreTile, true);
+  cudaError_t e = make_tensor_map_3d(&f.q, a->q, TmaDtype::kBF16, 1ull * p.heads * hs, p.rows, 1, a->ld_q * 2, 0, 64, kPreTile, true);
   if (e != cudaSuccess) return e;
-  e = make_tensor_map_3d(&tkv, a->kv, TmaDtype::kBF16, 1ull * p.heads * (p.dp + p.vp), p.n_keys, 1, a->ld_kv * 2, 0, 64,
+  e = make_tensor_map_3d(&f.kv, a->kv, TmaDtype::kBF16, 1ull * p.heads * (p.dp + p.vp), p.n_keys, 1, a->ld_kv * 2, 0, 64,
                          kPreTile, true);
   if (e != cudaSuccess) return e;
-  trot = tkv;
+  f.rot = f.kv;
   if (p.rp > 0) {
-    e = make_tensor_map_3d(&trot, a->rot, TmaDtype::kBF16, p.rp, p.n_keys, 1, 2ull * p.rp, 0, 64, kPreTile, true);
+    e = make_tensor_map_3d(&f.rot, a->rot, TmaDtype::kBF16, p.rp, p.n_keys, 1, 2ull * p.rp, 0, 64, kPreTile, true);
     if (e != cudaSuccess) return e;
-  }
-  static bool ready = false;
-  if (!ready) {
-    e = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-    if (e != cudaSuccess) return e;
-    ready = true;
   }
   const int pairs = (p.rows + 2 * kPreTile - 1) / (2 * kPreTile);
-  return launch_pdl(latent_prefill_kernel, dim3(p.heads * pairs), dim3(kPreThreads), smem, static_cast<cudaStream_t>(stream),
-                    tq, tkv, trot, p);
+  return launch_prompt_attend(f, p, p.heads * pairs, smem, static_cast<cudaStream_t>(stream));
 }

@@ -11,9 +11,13 @@
 //  moe_combine   : per row, fixed-order sum of its routes' FC2 rows plus the shared expert's split planes ->
 //                  this rank's fp32 partial plane (the cross-rank sum happens in hc_post_mix).
 //                  (reduction-order contract of native/cuda/kernels/v41_route_reduce.cu:13-34)
+//  route_softmax : the router of layer stacks: top-k of logits + bias, softmax over the chosen ones; a small pass is planned
+//                  by the block that finishes last, in the same launch
+//  gated_act     : activation of 32-bit experts
 #include "ds41_api.h"
 #include "ds41_launch.cuh"
 #include "ds41_ptx.cuh"
+#include "ds41_stack.cuh"
 
 namespace ds41 {
 
@@ -156,6 +160,115 @@ __global__ void __launch_bounds__(512) moe_plan_kernel(PlanParams p) {
     p.slot_of[i] = s;
     if (s >= 0) p.row_w[1ll * s * p.row_w_ld + i / p.topk] = p.weights[i];
   }
+}
+
+// one warp per row, lane l holds the logits of experts l, l + 32, ...; lane k keeps the k-th choice
+constexpr int kRouteThreads = 256;
+constexpr int kRouteMax = 512;           // experts
+__global__ void __launch_bounds__(kRouteThreads) route_softmax_kernel(ds41_route_args p) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x * (kRouteThreads / 32) + warp;
+  if (r < p.rows) {
+    constexpr int kMine = kRouteMax / 32;
+    float z[kMine];
+#pragma unroll
+    for (int i = 0; i < kMine; ++i) {
+      const int e = lane + 32 * i;
+      z[i] = e < p.experts ? proj_at(p.z, r, e) + (p.bias != nullptr ? p.bias[e] : 0.f) : -INFINITY;
+    }
+    float my_z = -INFINITY, best = -INFINITY;
+    int my_id = -1;
+    uint32_t taken = 0;                  // bit i: expert lane + 32 i is chosen
+    for (int k = 0; k < p.top; ++k) {
+      float v = -INFINITY;
+      int at = kRouteMax;
+#pragma unroll
+      for (int i = 0; i < kMine; ++i)
+        if (32 * i + lane < p.experts && !(taken >> i & 1u) && (at == kRouteMax || z[i] > v)) {
+          v = z[i];
+          at = lane + 32 * i;
+        }
+#pragma unroll
+      for (int o = 16; o; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ov > v || (ov == v && oi < at) || at == kRouteMax) {
+          v = ov;
+          at = oi;
+        }
+      }
+      if (k == 0) best = v;
+      if (lane == k) {
+        my_z = v;
+        my_id = at < p.experts ? at : -1;
+      }
+      if ((at & 31) == lane && at < kRouteMax) taken |= 1u << (at >> 5);
+    }
+    const float e = lane < p.top && my_id >= 0 ? expf(my_z - best) : 0.f;
+    const float w = e / warp_sum(e);
+    if (lane < p.top) {
+      p.ids[r * p.top + lane] = p.row_slot[r] >= 0 ? my_id : -1;
+      p.weights[r * p.top + lane] = w;
+    }
+  }
+  if (p.active == nullptr) return;
+  // ---- the block that arrives last sees every route and plans the experts
+  __shared__ unsigned int last;
+  __shared__ int used[kRouteMax];
+  __shared__ int slot_of_expert[kRouteMax];
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) last = atomicAdd(p.ticket, 1u) == gridDim.x - 1 ? 1u : 0u;
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  for (int e = tid; e < p.experts; e += kRouteThreads) used[e] = 0;
+  for (int i = tid; i < p.max_active * p.row_w_ld; i += kRouteThreads) p.row_w[i] = 0.f;
+  __syncthreads();
+  const int n = p.rows * p.top;
+  for (int i = tid; i < n; i += kRouteThreads) {
+    const int e = __ldcg(p.ids + i);
+    if (e >= 0 && __ldcg(p.weights + i) > 0.f) used[e] = 1;
+  }
+  __syncthreads();
+  if (warp == 0) {
+    int base = 0;
+    for (int e0 = 0; e0 < p.experts; e0 += 32) {
+      const int e = e0 + lane;
+      const bool u = e < p.experts && used[e] != 0;
+      const uint32_t m = __ballot_sync(0xffffffffu, u);
+      const int slot = base + __popc(m & ((1u << lane) - 1u));
+      if (e < p.experts) slot_of_expert[e] = u && slot < p.max_active ? slot : -1;
+      if (u && slot < p.max_active) p.active[slot] = e;
+      base += __popc(m);
+    }
+    if (lane == 0) {
+      *p.n_active = min(base, p.max_active);
+      *p.ticket = 0u;
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < n; i += kRouteThreads) {
+    const int e = __ldcg(p.ids + i);
+    const float w = __ldcg(p.weights + i);
+    const int s = e >= 0 && w > 0.f ? slot_of_expert[e] : -1;
+    p.slot_of[i] = s;
+    if (s >= 0) p.row_w[1ll * s * p.row_w_ld + i / p.top] = w;
+  }
+}
+
+__global__ void __launch_bounds__(256) gated_act_kernel(const float* x, int ld_x, int up_col, const float* row_w, int row_w_ld,
+                                                        const int* n_active, int rows, int n, float limit, float alpha,
+                                                        float shift, float* act, int ld_act) {
+  const int j = blockIdx.x * 256 + threadIdx.x, r = blockIdx.y, b = blockIdx.z;
+  pdl_launch_dependents();
+  pdl_wait();
+  if (b >= *n_active || j >= n) return;
+  const long long row = 1ll * b * rows + r;
+  const float g = fminf(x[row * ld_x + j], limit), u = fminf(fmaxf(x[row * ld_x + up_col + j], -limit), limit);
+  act[row * ld_act + j] = g / (1.0f + expf(-alpha * g)) * (u + shift) * row_w[1ll * b * row_w_ld + r];
 }
 
 struct CombineParams {
@@ -317,6 +430,28 @@ extern "C" int ds41_moe_plan(const int* ids, const float* weights, const int* ro
   if (rows <= 0 || e1 - e0 > 512 || e1 <= e0 || row_w_ld < rows) return cudaErrorInvalidValue;
   PlanParams p{ids, weights, row_slot, rows, topk, e0, e1, max_active, row_w_ld, active, n_active, row_w, slot_of};
   return launch_pdl(moe_plan_kernel, dim3(1), dim3(512), 0, static_cast<cudaStream_t>(stream), p);
+}
+
+extern "C" int ds41_route_softmax(const ds41_route_args* a, void* stream) {
+  if (a == nullptr || !proj_ok(a->z) || a->row_slot == nullptr || a->ids == nullptr || a->weights == nullptr ||
+      a->rows <= 0 || a->experts <= 0 || a->experts > kRouteMax || a->top <= 0 || a->top > 32 || a->top > a->experts)
+    return cudaErrorInvalidValue;
+  if (a->active != nullptr && (a->n_active == nullptr || a->row_w == nullptr || a->slot_of == nullptr || a->ticket == nullptr ||
+                               a->max_active <= 0 || a->row_w_ld < a->rows))
+    return cudaErrorInvalidValue;
+  constexpr int kWarps = kRouteThreads / 32;
+  return launch_pdl(route_softmax_kernel, dim3((a->rows + kWarps - 1) / kWarps), dim3(kRouteThreads), 0,
+                    static_cast<cudaStream_t>(stream), *a);
+}
+
+extern "C" int ds41_gated_act(const float* x, int ld_x, int up_col, const float* row_w, int row_w_ld, const int* n_active,
+                              int batch, int rows, int n, float limit, float alpha, float shift, float* act, int ld_act,
+                              void* stream) {
+  if (x == nullptr || row_w == nullptr || n_active == nullptr || act == nullptr || batch <= 0 || batch > 65535 || rows <= 0 ||
+      rows > 65535 || n <= 0 || up_col < n || ld_x < up_col + n || ld_act < n || row_w_ld < rows)
+    return cudaErrorInvalidValue;
+  return launch_pdl(gated_act_kernel, dim3((n + 255) / 256, rows, batch), dim3(256), 0, static_cast<cudaStream_t>(stream), x,
+                    ld_x, up_col, row_w, row_w_ld, n_active, rows, n, limit, alpha, shift, act, ld_act);
 }
 
 extern "C" int ds41_moe_combine(const float* fc2, const int* slot_of, const float* shared, int shared_splits,

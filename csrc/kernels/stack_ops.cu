@@ -1,11 +1,14 @@
 // Row-wise steps of a layer stack whose residual stream is one fp32 row per token.
 //
-//  resid_step    : closes a sublayer and opens the next one.  result -> sigmoid gate -> norm -> added to the stream;
+//  resid_step    : closes a sublayer and opens the next one.  result (of routed experts: the sum of the rows that the routes
+//                  name) -> sigmoid gate -> norm -> added to the stream;
 //                  optionally the stream becomes a weighted sum of the kept streams of all layers so far (depth average);
 //                  then the norm that feeds the next sublayer.  With `tokens` the stream starts from the embedding.
 //  polynorm      : activation a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square
 //  gate_mul      : result x sigmoid(gate)
 //  head_norm_gate: per-head RMS norm x weight x sigmoid(gate)
+//  side_act      : gelu_tanh(projection) x a layer's part of the token's second embedding
+//  softcap_rows  : cap tanh(x / cap) in place
 //  gather_rows   : picks rows of an activation matrix by index
 #include <cooperative_groups.h>
 
@@ -78,6 +81,22 @@ __device__ __forceinline__ float2 row_norm(const float4 (&v)[NI], int n, int W, 
   return make_float2(t.mean, 1.0f / sqrtf(t.m2 / W + eps));
 }
 
+// Four columns of the sum of a row's routed results, in route order.
+__device__ __forceinline__ float4 routed_at4(const ds41_resid_args& p, int r, int col) {
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int k = 0; k < p.y_top; ++k) {
+    const int e = p.y_route[r * p.y_top + k];
+    if (e < 0) continue;
+    const float4 v = proj_at4(p.y, p.y_rows > 0 ? 1ll * e * p.y_rows + r : 1ll * r * p.y_top + k, col);
+    s.x += v.x;
+    s.y += v.y;
+    s.z += v.z;
+    s.w += v.w;
+  }
+  return s;
+}
+
 template <typename T, int CL, int NI>
 __global__ void __launch_bounds__(CL == 8 ? 128 : (NI <= 4 ? 256 : 512)) resid_step_kernel(ds41_resid_args p) {
   __shared__ float slots[2][96];
@@ -145,7 +164,7 @@ __global__ void __launch_bounds__(CL == 8 ? 128 : (NI <= 4 ? 256 : 512)) resid_s
     for (int i = 0; i < NI; ++i) {
       y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (live[i] > 0) {
-        y[i] = proj_at4(p.y, r, c0 + at[i]);
+        y[i] = p.y_route != nullptr ? routed_at4(p, r, c0 + at[i]) : proj_at4(p.y, r, c0 + at[i]);
         if (p.gate.data != nullptr) {
           const float4 g = proj_at4(p.gate, r, c0 + at[i]), b = load4(p.gate_bias + c0 + at[i], live[i]);
           y[i].x *= sigmoid_f32(g.x + b.x);
@@ -157,7 +176,7 @@ __global__ void __launch_bounds__(CL == 8 ? 128 : (NI <= 4 ? 256 : 512)) resid_s
       }
     }
     float2 s = make_float2(0.f, 1.f);
-    if (p.post_w != nullptr) s = row_norm<CL, NI>(y, n, p.W, p.norm_kind, p.eps, slots[0]);
+    if (p.post_w != nullptr) s = row_norm<CL, NI>(y, n, p.W, p.post_rms ? 1 : p.norm_kind, p.eps, slots[0]);
 #pragma unroll
     for (int i = 0; i < NI; ++i)
       if (live[i] > 0) {
@@ -202,6 +221,12 @@ __global__ void __launch_bounds__(CL == 8 ? 128 : (NI <= 4 ? 256 : 512)) resid_s
         store4(h + at[i], make_float4((x[i].x - s.x) * s.y * w.x, (x[i].y - s.x) * s.y * w.y, (x[i].z - s.x) * s.y * w.z,
                                       (x[i].w - s.x) * s.y * w.w));
       }
+  }
+  if (p.next_w == nullptr && p.raw_h) {
+    T* h = static_cast<T*>(p.h) + 1ll * r * p.ldh + c0;
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+      if (live[i] > 0) store4(h + at[i], x[i]);
   }
   if constexpr (CL > 1) cg::this_cluster().sync();      // peers may still read this CTA's moments
 }
@@ -331,6 +356,33 @@ __global__ void __launch_bounds__(256) head_norm_gate_warp_kernel(const float* o
   }
 }
 
+// one block per row; columns [n, ld_out) are written as zeros
+template <typename T>
+__global__ void __launch_bounds__(128) side_act_kernel(ds41_proj z, const int* tokens, const __nv_bfloat16* embed,
+                                                       long long embed_ld, int col, int vocab, int n, T* out, int ld_out) {
+  const int r = blockIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tok = tokens[r];
+  const bool known = tok >= 0 && tok < vocab;
+  for (int j = threadIdx.x; j < ld_out; j += blockDim.x) {
+    float v = 0.f;
+    if (j < n) {
+      const float a = proj_at(z, r, j);
+      const float e = known ? __bfloat162float(embed[tok * embed_ld + col + j]) : 0.f;
+      v = 0.5f * a * (1.0f + tanhf(0.7978845608028654f * (a + 0.044715f * a * a * a))) * e;
+    }
+    out[1ll * r * ld_out + j] = from_f32<T>(v);
+  }
+}
+
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+  const long long i = 1ll * blockIdx.x * blockDim.x + threadIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
+  if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) gather_rows_kernel(const T* src, int ld, const int* index, int n_src, int W, T* dst) {
   const int r = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -370,7 +422,8 @@ extern "C" int ds41_resid_step(const ds41_resid_args* a, void* stream) {
   if (a->y.data != nullptr && !proj_ok(a->y)) return cudaErrorInvalidValue;
   if (a->gate.data != nullptr && (!proj_ok(a->gate) || a->gate_bias == nullptr)) return cudaErrorInvalidValue;
   if (a->mix != nullptr && (a->n_mix < 1 || (a->n_mix > 1 && a->kept == nullptr))) return cudaErrorInvalidValue;
-  if (a->next_w != nullptr && (a->h == nullptr || a->ldh < a->W || (a->ldh & 3))) return cudaErrorInvalidValue;
+  if (a->y_route != nullptr && (a->y.data == nullptr || a->y_top <= 0 || a->y_rows < 0)) return cudaErrorInvalidValue;
+  if ((a->next_w != nullptr || a->raw_h) && (a->h == nullptr || a->ldh < a->W || (a->ldh & 3))) return cudaErrorInvalidValue;
   // rows are walked in pieces of four columns
   if ((a->ldx & 3) || (a->kept_stride & 3) || (a->tokens != nullptr && (a->embed_ld & 3)) ||
       (a->y.data != nullptr && !proj_vec4(a->y)) || (a->gate.data != nullptr && !proj_vec4(a->gate)))
@@ -441,6 +494,26 @@ extern "C" int ds41_head_norm_gate(const float* o, int ld_o, const ds41_proj* ga
                       static_cast<float*>(out), ld_out);
   return launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, st, o, ld_o, *gate, w, width, stride, eps,
                     static_cast<__nv_bfloat16*>(out), ld_out);
+}
+
+extern "C" int ds41_side_act(const ds41_proj* z, const int* tokens, const void* embed, long long embed_ld, int col, int vocab,
+                             int rows, int n, void* out, int ld_out, int f32, void* stream) {
+  if (z == nullptr || !proj_ok(*z) || tokens == nullptr || embed == nullptr || out == nullptr || rows <= 0 || n <= 0 ||
+      ld_out < n || col < 0 || embed_ld < col + n || vocab <= 0 || z->ld < z->col + n)
+    return cudaErrorInvalidValue;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const __nv_bfloat16* e = static_cast<const __nv_bfloat16*>(embed);
+  if (f32)
+    return launch_pdl(side_act_kernel<float>, dim3(rows), dim3(128), 0, st, *z, tokens, e, embed_ld, col, vocab, n,
+                      static_cast<float*>(out), ld_out);
+  return launch_pdl(side_act_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, *z, tokens, e, embed_ld, col, vocab, n,
+                    static_cast<__nv_bfloat16*>(out), ld_out);
+}
+
+extern "C" int ds41_softcap_rows(float* x, long long n, float cap, void* stream) {
+  if (x == nullptr || n <= 0 || !(cap > 0.f) || (n + 255) / 256 > 0x7fffffffll) return cudaErrorInvalidValue;
+  return launch_pdl(softcap_kernel, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0,
+                    static_cast<cudaStream_t>(stream), x, n, cap);
 }
 
 extern "C" int ds41_gather_rows(const void* src, int ld, const int* index, int n_src, int rows, int W, void* dst, int f32,

@@ -74,8 +74,7 @@ def cmd_info(args) -> int:
     fam, cfg = _family(args)
     if fam.name != "ds41":
         import math
-        from .models import genesun
-        shapes = genesun.tensor_shapes(cfg)
+        shapes = fam.tensor_shapes(cfg)
         print(json.dumps({"model": cfg.name, "family": fam.name, "layers": cfg.n_layers, "hidden": cfg.hidden,
                           "mixers": [l.mixer.kind for l in cfg.layers], "vocab": cfg.vocab,
                           "checkpoint_tensors": len(shapes), "cache_rows_of_layers": cfg.cache_layers(),
@@ -147,8 +146,7 @@ def cmd_inspect_model(args) -> int:
     if fam.name != "ds41":
         import math
         from .loader.stack import StackCheckpoint
-        from .models import genesun
-        shapes = genesun.tensor_shapes(cfg)
+        shapes = fam.tensor_shapes(cfg)
         rep = {"model": cfg.name, "family": fam.name, "tensors": len(shapes),
                "total_gb": round(2 * sum(math.prod(x) for x in shapes.values()) / 2 ** 30, 3)}
         if args.checkpoint:

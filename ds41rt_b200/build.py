@@ -88,7 +88,8 @@ def _kernel_recipe(verbose: bool = False):
 
 
 # what a process that only runs layer-stack models needs of csrc/kernels
-STACK_KERNELS = ("gemm_f32", "gemm_tc", "latent_attn", "latent_prefill", "mlstm", "sampler", "sampler_rows", "stack_ops", "tma")
+STACK_KERNELS = ("ep", "gemm_f32", "gemm_tc", "group_attn", "group_prefill", "latent_attn", "latent_prefill", "mlstm", "moe", "sampler",
+                 "sampler_rows", "stack_ops", "tma")
 
 
 def _core_recipe():

@@ -24,6 +24,9 @@ class RopeConfig:
     beta_fast: float = 32.0
     beta_slow: float = 1.0
     original_max_position: int = 65536
+    # (low, high): instead of YaRN, frequencies are scaled by their wavelength - kept below original / high, divided by
+    # `factor` above original / low, interpolated between (the Llama 3.1 scheme)
+    bands: Optional[Tuple[float, float]] = None
 
     @property
     def scaled(self) -> bool:
@@ -322,11 +325,24 @@ class ModelConfig:
 
 def rope_inv_freq(rope: RopeConfig, dim: int) -> List[float]:
     """Inverse frequencies for `dim` rotary dims (dim/2 pairs) with YaRN
-    correction when factor > 1 (native/cuda/kernels/v41_attention_ops.cu:328-341)."""
+    correction when factor > 1 (native/cuda/kernels/v41_attention_ops.cu:328-341), or with wavelength bands."""
     half = dim // 2
     base = [rope.theta ** (-2.0 * i / dim) for i in range(half)]
     if not rope.scaled:
         return base
+    if rope.bands is not None:
+        low, high = rope.bands
+
+        def banded(f: float) -> float:
+            turns = rope.original_max_position * f / (2 * math.pi)     # full turns over the original context
+            if turns > high:
+                return f
+            if turns < low:
+                return f / rope.factor
+            s = (turns - low) / (high - low)
+            return (1 - s) * f / rope.factor + s * f
+
+        return [banded(f) for f in base]
 
     def corr_dim(rot: float) -> float:
         return dim * math.log(rope.original_max_position / (rot * 2 * math.pi)) / (2 * math.log(rope.theta))

@@ -11,7 +11,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from ..config import RopeConfig
-from ..stack_config import ConfigError, DenseMLPSpec, LatentAttentionSpec, LayerSpec, MLSTMSpec, StackConfig
+from ..stack_config import ConfigError, DenseMLPSpec, LatentAttentionSpec, LayerSpec, MLSTMSpec, StackConfig, take
 
 ARCHITECTURE = "Genesun"
 
@@ -20,47 +20,37 @@ def matches(doc: dict) -> bool:
     return doc.get("architecture") == ARCHITECTURE
 
 
-def _take(d, keys, where: str, optional=()):
-    """Values of exactly `keys` (and possibly `optional`) of a JSON object."""
-    if not isinstance(d, dict):
-        raise ConfigError(f"{where}: expected an object")
-    unknown, missing = set(d) - set(keys) - set(optional), set(keys) - set(d)
-    if unknown or missing:
-        raise ConfigError(f"{where}: unknown keys {sorted(unknown)}, missing keys {sorted(missing)}")
-    return [d[k] for k in keys] + [d.get(k) for k in optional]
-
-
 def _rope(rot, rot_dim: int, where: str) -> RopeConfig:
-    base, dims, scaling = _take(rot, ("base", "dims"), where, ("scaling",))
+    base, dims, scaling = take(rot, ("base", "dims"), where, ("scaling",))
     if dims != rot_dim or dims % 2:
         raise ConfigError(f"{where}: dims must equal the mixer's rot_dim and be even")
     if scaling is None:
         return RopeConfig(theta=float(base))
-    factor, fast, slow, original = _take(scaling, ("factor", "fast", "slow", "original"), where + ".scaling")
+    factor, fast, slow, original = take(scaling, ("factor", "fast", "slow", "original"), where + ".scaling")
     return RopeConfig(theta=float(base), factor=float(factor), beta_fast=float(fast), beta_slow=float(slow),
                       original_max_position=original)
 
 
 def parse(doc: dict, name: str = "genesun") -> StackConfig:
-    _, layers, norm, vocab, width = _take(doc, ("architecture", "layers", "norm", "vocab", "width"), "config")
-    (eps,) = _take(norm, ("eps",), "norm")
+    _, layers, norm, vocab, width = take(doc, ("architecture", "layers", "norm", "vocab", "width"), "config")
+    (eps,) = take(norm, ("eps",), "norm")
     specs = []
     for l, d in enumerate(layers):
-        kind, mx, mlp = _take(d, ("type", "mixer", "mlp"), f"layers[{l}]")
+        kind, mx, mlp = take(d, ("type", "mixer", "mlp"), f"layers[{l}]")
         where = f"layers[{l}].mixer"
         if kind == "latent_attention":
-            heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, rot, src = _take(
+            heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, rot, src = take(
                 mx, ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "rot"), where, ("kv_from",))
             mixer = LatentAttentionSpec(heads, dim, rot_dim, vdim, q_rank, kv_rank, float(scale),
                                         _rope(rot, rot_dim, where + ".rot"), src)
         elif kind == "mlstm":
-            heads, dim, vdim, cap = _take(mx, ("heads", "dim", "vdim", "gate_cap"), where)
+            heads, dim, vdim, cap = take(mx, ("heads", "dim", "vdim", "gate_cap"), where)
             mixer = MLSTMSpec(heads, dim, vdim, float(cap))
         else:
             raise ConfigError(f"layers[{l}]: unknown type {kind!r}")
         ff = None
         if mlp is not None:
-            mlp_kind, width_ff = _take(mlp, ("kind", "ff"), f"layers[{l}].mlp")
+            mlp_kind, width_ff = take(mlp, ("kind", "ff"), f"layers[{l}].mlp")
             if mlp_kind != "dense":
                 raise ConfigError(f"layers[{l}].mlp: unknown kind {mlp_kind!r}")
             ff = DenseMLPSpec(width_ff)

@@ -7,7 +7,7 @@ import os
 from typing import Dict, List, Optional
 
 from ..config import ModelConfig
-from . import genesun
+from . import belasun, genesun
 
 
 class UnsupportedDtype(ValueError):
@@ -65,20 +65,27 @@ class DS41Family(Family):
         return DS41Engine(cfg, weights, fabric, **kw)
 
 
-class GenesunFamily(Family):
-    """Layer stacks of latent attention and mLSTM (models/genesun.py, models/stack.py)."""
-    name = "genesun"
-    presets = genesun.PRESETS
+class StackFamily(Family):
+    """Layer-stack models (models/stack.py); `module` reads the family's configuration and names its tensors."""
     dtypes = ("bf16", "f32")
 
+    def __init__(self, name: str, module):
+        self.name, self.module, self.presets = name, module, module.PRESETS
+
     def matches(self, doc):
-        return genesun.matches(doc)
+        return self.module.matches(doc)
 
     def config(self, doc, text, name):
-        return genesun.parse(doc, name)
+        return self.module.parse(doc, name)
 
     def preset(self, name, layers=0):
-        return genesun.preset(name, layers or None)
+        return self.module.preset(name, layers or None)
+
+    def tensor_shapes(self, cfg):
+        return self.module.tensor_shapes(cfg)
+
+    def layer_shapes(self, cfg, layer: int):
+        return self.module.layer_shapes(cfg, layer)
 
     def _one_rank(self, world):
         if world != 1:
@@ -87,11 +94,11 @@ class GenesunFamily(Family):
     def load_weights(self, directory, cfg, device, dtype="bf16", rank=0, world=1, expert_dtype=None):
         from ..loader.stack import StackCheckpoint
         self._one_rank(world)
-        return genesun.build_weights(cfg, StackCheckpoint(directory, genesun.tensor_shapes(cfg)).read, device, dtype)
+        return self.module.build_weights(cfg, StackCheckpoint(directory, self.tensor_shapes(cfg)).read, device, dtype)
 
     def random_weights(self, cfg, device, seed=0, dtype="bf16", rank=0, world=1, expert_dtype=None):
         self._one_rank(world)
-        return genesun.random_weights(cfg, device, seed, dtype)
+        return self.module.random_weights(cfg, device, seed, dtype)
 
     def engine(self, cfg, weights, fabric=None, kv_dtype="bf16", **kw):
         from .stack import StackEngine
@@ -100,12 +107,13 @@ class GenesunFamily(Family):
         return StackEngine(cfg, weights, **kw)
 
 
-FAMILIES: Dict[str, Family] = {f.name: f for f in (DS41Family(), GenesunFamily())}
+FAMILIES: Dict[str, Family] = {f.name: f for f in (DS41Family(), StackFamily("genesun", genesun),
+                                                  StackFamily("belasun", belasun))}
 PRESETS: List[str] = [p for f in FAMILIES.values() for p in f.presets]
 
 
 def family_of(cfg) -> Family:
-    return FAMILIES["ds41"] if isinstance(cfg, ModelConfig) else FAMILIES["genesun"]
+    return FAMILIES["ds41"] if isinstance(cfg, ModelConfig) else FAMILIES[cfg.family]
 
 
 def config_from_file(path: str):

@@ -6,8 +6,8 @@ depends on data stays on the device, so a decode pass is captured as a CUDA grap
 (matrix products and activations in bf16 with fp32 accumulation; streams, norms, gates, attention weights and recurrent
 states in fp32); `dtype="f32"` keeps everything in true 32-bit.
 
-`StackCache` holds what a request leaves behind: paged latent rows of the attention layers that produce them (a layer that
-reads another layer's rows has none of its own) and one recurrent state per slot and recurrent layer.
+`StackCache` holds what a request leaves behind: paged rows of the attention layers that produce them (a layer that reads
+another layer's rows has none of its own) and one state per slot for recurrences and for the inputs of short convolutions.
 """
 from __future__ import annotations
 
@@ -21,7 +21,7 @@ from ..config import rope_inv_freq
 from ..ops import lib
 from ..ops import stack as S
 from ..ops.stack import Matrix, Proj, ceil_to
-from ..stack_config import LatentAttentionSpec, MLSTMSpec, StackConfig
+from ..stack_config import GroupedAttentionSpec, LatentAttentionSpec, MLSTMSpec, MoESpec, StackConfig
 from .base import RowsEngine
 from .paged import PagedSlots
 
@@ -50,7 +50,21 @@ def latent_row_len(m: LatentAttentionSpec) -> Tuple[int, int]:
     return kv, kv + ceil_to(m.rot_dim, 16)
 
 
-def mlstm_state_shapes(m: MLSTMSpec) -> Tuple[Tuple[int, ...], ...]:
+def grouped_widths(m: GroupedAttentionSpec) -> Tuple[int, int, int]:
+    """(query columns, key columns, value columns) of all heads, every head padded to 16 values."""
+    d, v = ceil_to(m.dim, 16), ceil_to(m.vdim, 16)
+    return m.heads * d, m.kv_heads * d, m.kv_heads * v
+
+
+def cache_row_len(m) -> int:
+    """Values of one token's cache row."""
+    return latent_row_len(m)[1] if m.kind == "latent_attention" else sum(grouped_widths(m)[1:])
+
+
+def state_shapes(m) -> Tuple[Tuple[int, ...], ...]:
+    """fp32 state of one request: the recurrence's, or the convolution's last inputs (a ring over positions)."""
+    if m.kind == "grouped_attention":
+        return ((m.taps - 1, sum(grouped_widths(m))),)
     d, v = ceil_to(m.dim, 16), ceil_to(m.vdim, 16)
     nb = -(-v // S.STATE_COLS)
     return (m.heads, d, v), (m.heads, nb, d), (m.heads, nb)
@@ -63,11 +77,11 @@ class StackCache(PagedSlots):
         self._init_pages(slots, max_ctx, device, page_tokens, n_pages)
         self.pools: Dict[int, torch.Tensor] = {}
         for l in cfg.cache_layers():
-            row = latent_row_len(cfg.layers[l].mixer)[1]
+            row = cache_row_len(cfg.layers[l].mixer)
             self.pools[l] = torch.zeros(self.n_pages * page_tokens, row, dtype=dtype, device=device)
         self.states: Dict[int, Tuple[torch.Tensor, ...]] = {
             l: tuple(torch.zeros(slots, *shape, dtype=F32, device=device)
-                     for shape in mlstm_state_shapes(cfg.layers[l].mixer)) for l in cfg.state_layers()}
+                     for shape in state_shapes(cfg.layers[l].mixer)) for l in cfg.state_layers()}
 
     def snapshot(self, slot: int, n_tokens: int) -> StackSnapshot:
         """Capture `slot`, whose last pass ended at position n_tokens - 1 (call it between passes, on the stream)."""
@@ -291,7 +305,83 @@ class MLSTM:
         return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
 
 
-MIXERS = {"latent_attention": LatentAttention, "mlstm": MLSTM}
+class GroupedAttention:
+    """Grouped-query attention over cached keys and values, head widths padded to 16 values: projection, then convolution,
+    norm, rotation and cache rows in one launch, then attention with the head gates.  Long prompt passes of one request
+    take the tcgen05 form, everything else a CTA (or a cluster of them) per row and key/value head."""
+
+    def __init__(self, spec: GroupedAttentionSpec, cfg: StackConfig, t: Dict[str, torch.Tensor], gate: Dict[str, torch.Tensor],
+                 device, dtype):
+        self.spec, self.cfg = spec, cfg
+        H, G = spec.heads, spec.kv_heads
+        self.dp, self.vp = ceil_to(spec.dim, 16), ceil_to(spec.vdim, 16)
+        self.cols = sum(grouped_widths(spec))
+
+        def heads(name, suffix=""):
+            n, w, p = {"q": (H, spec.dim, self.dp), "k": (G, spec.dim, self.dp), "v": (G, spec.vdim, self.vp)}[name]
+            return S.pad_heads(t[name + suffix], n, w, p)
+
+        f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
+        parts = [("u", torch.cat([heads(n) for n in "qkv"], 0))]
+        if spec.head_gate:
+            parts += [("g", t["g"])]
+        if gate:
+            parts += [("gate", gate["w"])]
+        self.w_in, self.at = S.stack_rows(parts, device, dtype)
+        self.conv = f32(torch.cat([heads(n, ".conv") for n in "qkv"], 0).t()) if spec.taps else None
+        self.q_norm, self.k_norm = (f32(heads(n, ".norm")) if spec.qk_norm else None for n in "qk")
+        self.freq = torch.tensor(rope_inv_freq(spec.rope, spec.rot_dim) or [0.0], dtype=F32, device=device) \
+            if spec.rot_dim else None
+        self.w_o = Matrix(S.pad_heads(t["o"].t().contiguous(), H, spec.vdim, self.vp).t(), device, dtype)
+        # the tcgen05 form keeps two query tiles, a key tile and a value tile of 128 rows in shared memory
+        self.tiled = dtype == BF16 and self.vp <= 128 and 3 * -(-self.dp // 64) + -(-self.vp // 64) <= 14
+
+    def matrices(self):
+        return {"a": [(self.w_in.n, self.w_in.k)], "b": [(self.w_o.n, self.w_o.k)]}
+
+    def splits(self, e: "StackEngine", rows: int) -> int:
+        """CTAs that share a row's keys: enough to fill the GPU about twice, static per batch size (a captured pass replays
+        while the context grows)."""
+        sp = self.spec
+        span = min(sp.chunk or e.cache.max_ctx, e.cache.max_ctx)
+        blocks = rows * sp.kv_heads * -(-(sp.heads // sp.kv_heads) // 16)
+        return max(1, min(2 * 148 // blocks, 8, -(-span // 64)))
+
+    def run(self, e: "StackEngine", l: int, R: int, src: int) -> Tuple[Proj, Optional[Proj]]:
+        sp, k, c = self.spec, e.k, e.cache
+        long = e.long_keys if self.tiled and c.page_tokens in (32, 64, 128) else 0
+        pin = e.project_wide("gemm_mix_in", R, self.w_in) if long else \
+            e.project("gemm_mix_in", e.h, e.ldh, R, self.w_in, e.planes_a)
+        u = pin.at(self.at["u"])
+        state = c.states[l][0] if sp.taps > 1 else None
+        ldq, ldo = sp.heads * self.dp, sp.heads * self.vp
+        a = S.AttnPostArgs()
+        a.u, a.conv, a.q_norm, a.k_norm, a.freq = u.args(), lib.ptr(self.conv), lib.ptr(self.q_norm), lib.ptr(self.k_norm), \
+            lib.ptr(self.freq)
+        a.state, a.q, a.pool, a.ld_q, a.eps = lib.ptr(state), lib.ptr(e.q), lib.ptr(c.pools[src]), ldq, self.cfg.norm_eps
+        a.page_table, a.row_pos, a.row_slot = lib.ptr(c.page_table), lib.ptr(e.row_pos), lib.ptr(e.row_slot)
+        a.rows, a.heads, a.kv_heads, a.dim, a.dim_pad, a.vdim_pad = R, sp.heads, sp.kv_heads, sp.dim, self.dp, self.vp
+        a.rot_dim, a.taps, a.slots, a.max_pages, a.page_tokens, a.f32 = sp.rot_dim, max(sp.taps, 1), c.slots, c.max_pages, \
+            c.page_tokens, e.f32
+        e._run("attn_post", k.ds41_attn_post, C.byref(a), lib.stream())
+        b = S.GroupAttendArgs()
+        b.q, b.pool, b.out, b.status = lib.ptr(e.q), lib.ptr(c.pools[src]), lib.ptr(e.act), lib.ptr(e.status)
+        b.page_table, b.row_pos, b.row_slot = a.page_table, a.row_pos, a.row_slot
+        b.gate = pin.at(self.at["g"]).args() if sp.head_gate else S.NO_PROJ
+        b.u, b.state, b.ld_q, b.scale = u.args(), lib.ptr(state), ldq, sp.scale
+        b.rows, b.heads, b.kv_heads, b.dim_pad, b.vdim_pad, b.chunk = R, sp.heads, sp.kv_heads, self.dp, self.vp, sp.chunk
+        b.taps, b.slots, b.ld_out, b.max_pages, b.page_tokens, b.f32 = a.taps, c.slots, ldo, c.max_pages, c.page_tokens, e.f32
+        if long:
+            b.n_pages, b.pos0, b.n_splits = c.n_pages, long - R, 1
+            e._run("group_prefill", k.ds41_group_prefill, C.byref(b), lib.stream())
+        else:
+            b.n_splits = self.splits(e, R)
+            e._run("group_attend", k.ds41_group_attend, C.byref(b), lib.stream())
+        y = e.project("gemm_o", e.act, ldo, R, self.w_o, e.planes_b)
+        return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
+
+
+MIXERS = {"latent_attention": LatentAttention, "grouped_attention": GroupedAttention, "mlstm": MLSTM}
 
 
 class DenseMLP:
@@ -316,6 +406,89 @@ class DenseMLP:
         return y, (pin.at(self.at["gate"]) if "gate" in self.at else None)
 
 
+class RoutedExperts:
+    """Mixture of experts.  Passes of up to `moe_rows` rows run every used expert over all rows, planned by the router's
+    launch; longer ones sort the rows by expert (parallel/ep.py).  Either way the routes' results are summed by the residual
+    step that follows.  32-bit passes always take the first form."""
+
+    def __init__(self, spec: MoESpec, cfg: StackConfig, t: Dict[str, torch.Tensor], gate: Dict[str, torch.Tensor],
+                 device, dtype):
+        self.spec, self.cfg = spec, cfg
+        E, W, ff = spec.experts, cfg.hidden, spec.ff
+        self.ld, self.ffp = ceil_to(W, 8), ceil_to(ff, 8)
+        self.w_router, self.at = S.stack_rows([("router", t["router"])] + ([("gate", gate["w"])] if gate else []), device, dtype)
+        self.bias = t["router.b"].to(device=device, dtype=F32).contiguous() if "router.b" in t else None
+        z = lambda *shape: torch.zeros(*shape, dtype=dtype, device=device)
+        self.w13, self.w2 = z(E, 2 * self.ffp, self.ld), z(E, self.ld, self.ffp)
+        for e in range(E):
+            self.w13[e, :ff, :W] = t[f"e{e}.gate"].to(device=device, dtype=dtype)
+            self.w13[e, self.ffp:self.ffp + ff, :W] = t[f"e{e}.up"].to(device=device, dtype=dtype)
+            self.w2[e, :W, :ff] = t[f"e{e}.down"].to(device=device, dtype=dtype)
+
+    def matrices(self):
+        return {"a": [(self.w_router.n, self.w_router.k)]}
+
+    def run(self, e: "StackEngine", R: int) -> Tuple[Proj, Optional[Proj]]:
+        sp, k, E, top = self.spec, e.k, self.spec.experts, self.spec.top
+        z = e.project("gemm_router", e.h, e.ldh, R, self.w_router, e.planes_a, few=True)
+        planned = R <= e.moe_rows
+        a = S.RouteArgs()
+        a.z, a.bias, a.row_slot = z.at(self.at["router"]).args(), lib.ptr(self.bias), lib.ptr(e.row_slot)
+        a.ids, a.weights, a.rows, a.experts, a.top = lib.ptr(e.ids), lib.ptr(e.route_w), R, E, top
+        if planned:
+            a.active, a.n_active, a.row_w, a.slot_of, a.ticket = (lib.ptr(x) for x in (e.active, e.n_active, e.row_w, e.slot_of,
+                                                                                      e.ticket))
+            a.max_active, a.row_w_ld = e.max_active(sp), e.moe_rows
+        e._run("route", k.ds41_route_softmax, C.byref(a), lib.stream())
+        gate = z.at(self.at["gate"]) if "gate" in self.at else None
+        if not planned:
+            ep = e.exchange(self)
+            if e.only is None or "ep_moe" in e.only:
+                e.launches += 4
+            ids, wt = e.ids[:R * top].view(R, top), e.route_w[:R * top].view(R, top)
+            e._run("ep_moe", ep.forward, e.h[:R], ids, wt, None)
+            return S.RoutedProj(ep.comb, self.ld, route=e.ids, top=top), gate
+        I, n = self.ffp, e.max_active(sp)
+        if e.f32:
+            e._run("gemm_fc1", S.gemm_f32, e.h, self.w13, e.moe_up, R, 2 * I, self.ld, e.ldh, self.ld, 2 * I, batch=n, sb=2 * I * self.ld,
+                   so=R * 2 * I, batch_map=e.active, n_active=e.n_active)
+            e._run("gated_act", k.ds41_gated_act, lib.ptr(e.moe_up), 2 * I, I, lib.ptr(e.row_w), e.moe_rows, lib.ptr(e.n_active), n, R,
+                   I, C.c_float(sp.limit), C.c_float(sp.alpha), C.c_float(sp.shift), lib.ptr(e.moe_act), I, lib.stream())
+            e._run("gemm_fc2", S.gemm_f32, e.moe_act, self.w2, e.moe_out, R, self.ld, I, I, I, self.ld, batch=n, sa=R * I,
+                   sb=self.ld * I, so=R * self.ld, batch_map=e.active, n_active=e.n_active)
+        else:
+            act = dict(act_limit=sp.limit, act_alpha=sp.alpha, act_shift=sp.shift)
+            many = dict(batch=n, a_batches=E, batch_map=e.active, n_active=e.n_active, row_w=e.row_w, row_w_ld=e.moe_rows,
+                        bn=S.G.pick_bn(R), status=e.status)
+            e._run("gemm_fc1", S.G.gemm_raw, self.w13, e.h, e.moe_act, I, R, self.ld, lda=self.ld, ldb=e.ldh, ldo=I, out_mode=4,
+                   a_batch_stride=2 * I * self.ld, out_batch_stride=R * I, b_batch_kind=1, up_row_offset=I, **act, **many)
+            e._run("gemm_fc2", S.G.gemm_raw, self.w2, e.moe_act, e.moe_out, self.ld, R, I, lda=I, ldb=I, ldo=self.ld, out_mode=5,
+                   a_batch_stride=self.ld * I, b_batch_stride=R * I, out_batch_stride=R * self.ld, b_batch_kind=2, **many)
+        return S.RoutedProj(e.moe_out, self.ld, route=e.slot_of, top=top, rows=R), gate
+
+
+MLPS = {"dense": DenseMLP, "moe": RoutedExperts}
+
+
+class TokenSide:
+    """What a layer adds from its own part of the tokens' second embedding: norm(proj(gelu(gate x) * part))."""
+
+    def __init__(self, layer: int, cfg: StackConfig, t: Dict[str, torch.Tensor], device, dtype):
+        self.cfg, self.dim, self.col = cfg, cfg.token_side, layer * cfg.token_side
+        self.w_gate, self.w_proj = Matrix(t["gate"], device, dtype), Matrix(t["proj"], device, dtype)
+        self.norm = t["norm"].to(device=device, dtype=F32).contiguous()
+
+    def matrices(self):
+        return {"a": [(self.w_gate.n, self.w_gate.k)], "b": [(self.w_proj.n, self.w_proj.k)]}
+
+    def run(self, e: "StackEngine", R: int) -> Tuple[Proj, Optional[Proj]]:
+        z = e.project("gemm_side_gate", e.h, e.ldh, R, self.w_gate, e.planes_a, few=True)
+        ld, table = self.w_proj.ld, e.w.side_embed
+        e._run("side_act", e.k.ds41_side_act, C.byref(z.args()), lib.ptr(e.in_tokens), lib.ptr(table), C.c_longlong(table.shape[1]),
+               self.col, self.cfg.vocab, R, self.dim, lib.ptr(e.act), ld, e.f32, lib.stream())
+        return e.project("gemm_side_proj", e.act, ld, R, self.w_proj, e.planes_b), None
+
+
 # ---------------------------------------------------------------------------------------------------- weights
 @dataclass
 class StackLayer:
@@ -323,17 +496,21 @@ class StackLayer:
     norm1: torch.Tensor
     norm1b: Optional[torch.Tensor]
     bias1: Optional[torch.Tensor]
-    mlp: Optional[DenseMLP] = None
+    mlp: object = None
     norm2: Optional[torch.Tensor] = None
     norm2b: Optional[torch.Tensor] = None
     bias2: Optional[torch.Tensor] = None
     mix: Optional[torch.Tensor] = None
+    side: Optional[TokenSide] = None
+
+    def parts(self):
+        return [m for m in (self.mixer, self.mlp, self.side) if m is not None]
 
 
 class StackWeights:
     """Kernel-layout weights built from a family's tensors: `get(l)` returns layer l's tensors under canonical names
-    (mixer tensors "mix.*", feed-forward "mlp.*", norms, "rg1" / "rg1.b" / "rg2" / "rg2.b", "dwa"); `top` has "embed",
-    "final.norm" and "head"."""
+    (mixer tensors "mix.*", feed-forward "mlp.*", "side.*", norms, "rg1" / "rg1.b" / "rg2" / "rg2.b", "dwa"); `top` has
+    "embed", "final.norm", "head" (the same tensor as "embed" where they are tied) and "side.embed"."""
 
     def __init__(self, cfg: StackConfig, get, top: Dict[str, torch.Tensor], device, dtype: str = "bf16"):
         self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
@@ -341,7 +518,8 @@ class StackWeights:
         f32 = lambda x: x.to(device=device, dtype=F32).contiguous()
         self.embed = Matrix(top["embed"], device, BF16)
         self.final_norm = f32(top["final.norm"])
-        self.head = Matrix(top["head"], device, dt)
+        self.head = self.embed if top["head"] is top["embed"] and dt == BF16 else Matrix(top["head"], device, dt)
+        self.side_embed = top["side.embed"].to(device=device, dtype=BF16).contiguous() if cfg.token_side else None
         self.layers: List[StackLayer] = []
         for l, spec in enumerate(cfg.layers):
             t = get(l)
@@ -352,10 +530,12 @@ class StackWeights:
             lw = StackLayer(MIXERS[spec.mixer.kind](spec.mixer, cfg, part("mix."), gate("rg1"), device, dt),
                             f32(t["norm1"]), post("norm1b"), bias("rg1.b"))
             if spec.mlp is not None:
-                lw.mlp = DenseMLP(spec.mlp, cfg, part("mlp."), gate("rg2"), device, dt)
+                lw.mlp = MLPS[spec.mlp.kind](spec.mlp, cfg, part("mlp."), gate("rg2"), device, dt)
                 lw.norm2, lw.norm2b, lw.bias2 = f32(t["norm2"]), post("norm2b"), bias("rg2.b")
             if cfg.depth_average:
                 lw.mix = f32(t["dwa"])
+            if cfg.token_side:
+                lw.side = TokenSide(l, cfg, part("side."), device, dt)
             self.layers.append(lw)
 
     def nbytes(self) -> int:
@@ -367,7 +547,7 @@ class StackWeights:
                     if v.untyped_storage().data_ptr() not in seen:
                         seen.add(v.untyped_storage().data_ptr())
                         total += v.untyped_storage().nbytes()
-                elif isinstance(v, (list, Matrix, StackLayer, DenseMLP) + tuple(MIXERS.values())):
+                elif isinstance(v, (list, Matrix, StackLayer, TokenSide) + tuple(MLPS.values()) + tuple(MIXERS.values())):
                     todo.append(v)
         return total
 
@@ -380,7 +560,7 @@ class StackEngine(RowsEngine):
     taps = None
 
     def __init__(self, cfg: StackConfig, weights: StackWeights, *, max_rows: int = 8, slots: int = 1, max_ctx: int = 4096,
-                 page_tokens: int = 64, n_pages: Optional[int] = None):
+                 page_tokens: int = 64, n_pages: Optional[int] = None, moe_rows: int = 32):
         self.cfg, self.w, self.device = cfg, weights, weights.device
         self.rank, self.world = 0, 1
         self.max_rows = R = max_rows
@@ -408,15 +588,18 @@ class StackEngine(RowsEngine):
         self.attn_rows = min(R, 256)
         cells = 1
         for lw in weights.layers:
-            for m in (lw.mixer, lw.mlp):
-                if m is not None:
-                    for b, ms in m.matrices().items():
-                        for n, kk in ms:
-                            need[b] = max(need[b], S.plane_floats(R, n, kk))
+            for m in lw.parts():
+                for b, ms in m.matrices().items():
+                    for n, kk in ms:
+                        need[b] = max(need[b], S.plane_floats(R, n, kk))
             mx = lw.mixer
             heads = max(heads, mx.spec.heads * mx.vp)
-            if lw.mlp is not None:
+            if isinstance(lw.mlp, DenseMLP):
                 act = max(act, lw.mlp.ffp)
+            if lw.side is not None:
+                act = max(act, lw.side.w_proj.ld)
+            if isinstance(mx, GroupedAttention):
+                q = max(q, mx.spec.heads * mx.dp)
             if isinstance(mx, LatentAttention):
                 q = max(q, mx.spec.heads * mx.hs)
                 q_rank = max(q_rank, mx.spec.q_rank)
@@ -428,8 +611,7 @@ class StackEngine(RowsEngine):
         self.long_rows = 64
         self.long_keys = 0            # > 0 during a long pass: positions its last row sees
         self.gathered = None
-        wide = max(S.ceil_to(n, 8) for lw in weights.layers for m in (lw.mixer, lw.mlp) if m is not None
-                   for n, _ in m.matrices()["a"])
+        wide = max(S.ceil_to(n, 8) for lw in weights.layers for m in lw.parts() for n, _ in m.matrices()["a"])
         self.wide = z((R * wide if R >= self.long_rows and not self.f32 else 8,), BF16)
         long_rec = [lw.mixer for lw in weights.layers if isinstance(lw.mixer, MLSTM) and lw.mixer.chunked] \
             if R >= self.long_rows else []
@@ -438,11 +620,12 @@ class StackEngine(RowsEngine):
         self._keys = [z((8,), BF16) for _ in range(3)]
         self.act = z((R * max(act, heads),), dt)
         self.o_heads = z((R * heads,), F32)
+        self.q = z((R * q,), dt)
         if lat:
             self.cq = z((R, ceil_to(q_rank, 8)), dt)
-            self.q = z((R * q,), dt)
             self.q_abs, self.o_lat = z((self.attn_rows * lat,), dt), z((self.attn_rows * lat,), dt)
             self.part_o, self.part_ml = z((cells,), F32), z((cells // 8 + 2,), F32)
+        self._init_experts(R, moe_rows, z, dt)
         # head
         self.head_cap = min(R, 64)
         self.last_head_row = 0
@@ -455,6 +638,40 @@ class StackEngine(RowsEngine):
         self._init_instruments()
         self.on_layer = None      # callable (layer, streams [rows, width]) after every layer of an eager pass
 
+    def _init_experts(self, R: int, moe_rows: int, z, dt):
+        """Routes, plans and buffers of the mixtures of experts: passes of at most `moe_rows` rows (32-bit passes: all) run
+        every used expert over all rows, longer ones sort the rows by expert."""
+        moes = [lw.mlp for lw in self.w.layers if isinstance(lw.mlp, RoutedExperts)]
+        self.moe_rows = Rm = R if self.f32 else min(R, moe_rows)
+        self._exchanges: Dict[tuple, object] = {}
+        top = max([m.spec.top for m in moes], default=1)
+        self.ids, self.route_w, self.slot_of = z((R * top,), I32), z((R * top,), F32), z((R * top,), I32)
+        live = [(self.max_active(m.spec), m) for m in moes] or [(1, None)]
+        most = max(n for n, _ in live)
+        self.active, self.n_active, self.ticket = z((most,), I32), z((1,), I32), z((1,), I32)
+        self.row_w = z((most * Rm,), F32)
+        size = lambda f: max([n * Rm * f(m) for n, m in live if m is not None], default=8)
+        self.moe_act, self.moe_out = z((size(lambda m: m.ffp),), dt), z((size(lambda m: m.ld),), F32)
+        self.moe_up = z((size(lambda m: 2 * m.ffp) if self.f32 else 8,), F32)
+
+    def max_active(self, m: MoESpec) -> int:
+        """Most experts that a planned pass can use."""
+        return min(m.experts, self.moe_rows * m.top)
+
+    def exchange(self, m: RoutedExperts):
+        """The sorted-rows form for experts of this shape, pointed at the layer's weights."""
+        from ..parallel.ep import ExpertParallelMoE
+        from ..parallel.fabric import Fabric
+        sp = m.spec
+        key = (sp.experts, sp.top, m.ffp, sp.limit, sp.alpha, sp.shift)
+        if key not in self._exchanges:
+            ep = ExpertParallelMoE(Fabric.single(self.device), m.w13, m.w2, topk=sp.top, max_tokens=self.max_rows,
+                                   act_limit=sp.limit, act_alpha=sp.alpha, act_shift=sp.shift)
+            ep.status = self.status
+            self._exchanges[key] = ep
+        self._exchanges[key].set_weights(m.w13, m.w2)
+        return self._exchanges[key]
+
     # ------------------------------------------------------------------ helpers
     def attn_splits(self, rows: int, heads: int) -> int:
         """Key splits per row of the absorbed attention: enough blocks to fill the GPU about twice, static per batch
@@ -462,9 +679,11 @@ class StackEngine(RowsEngine):
         want = 2 * 148 // (rows * -(-heads // 32))
         return max(1, min(want, 32, -(-self.cache.max_ctx // 64)))
 
-    def project(self, tag: str, x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor) -> Proj:
+    def project(self, tag: str, x: torch.Tensor, ldx: int, rows: int, m: Matrix, buf: torch.Tensor, few: bool = False) -> Proj:
+        """fp32 result of a projection; `few`: the matrix has few rows, which long passes take as the 128-row operand."""
         out: List[Proj] = []
-        self._run(tag, lambda: out.append(S.project(x, ldx, rows, m, buf, self.status)))
+        fn = S.project_few if few and rows > S.SWAP_ROWS and not self.f32 else S.project
+        self._run(tag, lambda: out.append(fn(x, ldx, rows, m, buf, self.status)))
         return out[0] if out else S.Proj(buf, m.out_ld)
 
     def project_wide(self, tag: str, rows: int, m: Matrix) -> Proj:
@@ -508,7 +727,8 @@ class StackEngine(RowsEngine):
         self.row_slot.copy_(torch.tensor(slots + [-1] * pad, dtype=I32), non_blocking=True)
 
     def _resid(self, R: int, *, y: Optional[Proj] = None, gate: Optional[Proj] = None, bias=None, post=None, x_in=None,
-               x_out=None, layer: Optional[int] = None, next_w=None):
+               x_out=None, layer: Optional[int] = None, next_w=None, post_rms: bool = False):
+        """`next_w`: weight of the norm that opens the next sublayer, None: that sublayer reads the stream itself."""
         a = S.ResidArgs()
         cfg = self.cfg
         a.y, a.gate = (y.args() if y is not None else S.NO_PROJ), (gate.args() if gate is not None else S.NO_PROJ)
@@ -521,6 +741,9 @@ class StackEngine(RowsEngine):
             a.n_mix, a.x_avg = layer + 2, lib.ptr(self.x_avg)
         a.h, a.ldh, a.ldx, a.vocab, a.rows, a.W = lib.ptr(self.h), self.ldh, self.ldx, cfg.vocab, R, cfg.hidden
         a.norm_kind, a.eps, a.f32 = cfg.norm_kind, cfg.norm_eps, self.f32
+        a.raw_h, a.post_rms = int(next_w is None), int(post_rms)
+        if isinstance(y, S.RoutedProj):
+            a.y_route, a.y_top, a.y_rows = lib.ptr(y.route), y.top, y.rows
         self._run("resid_step", self.k.ds41_resid_step, C.byref(a), lib.stream())
 
     # ------------------------------------------------------------------ one pass
@@ -535,16 +758,20 @@ class StackEngine(RowsEngine):
         self._resid(R, x_out=cur, next_w=layers[0].norm1)
         for l, lw in enumerate(layers):
             after = layers[l + 1].norm1 if l + 1 < len(layers) else self.w.final_norm
-            done = self.kept[l + 1] if cfg.depth_average else self.kept[0]
-            mix = l if cfg.depth_average else None
-            y, gate = lw.mixer.run(self, l, R, cfg.source_of(l))
-            if lw.mlp is None:
-                self._resid(R, y=y, gate=gate, bias=lw.bias1, post=lw.norm1b, x_in=cur, x_out=done, layer=mix, next_w=after)
-            else:
-                self._resid(R, y=y, gate=gate, bias=lw.bias1, post=lw.norm1b, x_in=cur, x_out=self.x_mid, next_w=lw.norm2)
-                y, gate = lw.mlp.run(self, R)
-                self._resid(R, y=y, gate=gate, bias=lw.bias2, post=lw.norm2b, x_in=self.x_mid, x_out=done, layer=mix,
-                            next_w=after)
+            # (run, norm of its input, what follows its result) of the layer's sublayers
+            subs = [(lambda: lw.mixer.run(self, l, R, cfg.source_of(l)), lw.norm1, dict(bias=lw.bias1, post=lw.norm1b))]
+            if lw.mlp is not None:
+                subs.append((lambda: lw.mlp.run(self, R), lw.norm2, dict(bias=lw.bias2, post=lw.norm2b)))
+            if lw.side is not None:
+                subs.append((lambda: lw.side.run(self, R), None, dict(post=lw.side.norm, post_rms=True)))
+            for i, (run, _, closing) in enumerate(subs):
+                y, gate = run()
+                if i + 1 < len(subs):
+                    self._resid(R, y=y, gate=gate, x_in=cur, x_out=self.x_mid, next_w=subs[i + 1][1], **closing)
+                    cur = self.x_mid
+                else:
+                    self._resid(R, y=y, gate=gate, x_in=cur, x_out=self.kept[l + 1] if cfg.depth_average else self.kept[0],
+                                layer=l if cfg.depth_average else None, next_w=after, **closing)
             cur = self.x_avg if cfg.depth_average else self.kept[0]
             if self.layer_timer is not None:
                 self.layer_timer.mark()
@@ -559,10 +786,13 @@ class StackEngine(RowsEngine):
         m = self.w.head
         if self.f32:
             self._run("gemm_head", S.gemm_f32, x, m.w, self.logits, rows, m.n, m.k, self.ldh, m.ld, self.cfg.vocab)
+            if self.cfg.logit_softcap:
+                self._run("softcap_rows", self.k.ds41_softcap_rows, lib.ptr(self.logits), C.c_longlong(rows * self.cfg.vocab),
+                          C.c_float(self.cfg.logit_softcap), lib.stream())
         else:
             from ..ops import gemm as G
             self._run("gemm_head", G.gemm_raw, m.w, x, self.logits, m.n, rows, m.k, lda=m.ld, ldb=self.ldh,
-                      ldo=self.cfg.vocab, out_mode=3, status=self.status, static_operand=1)
+                      ldo=self.cfg.vocab, out_mode=3, status=self.status, static_operand=1, softcap=self.cfg.logit_softcap)
 
     def head_rows(self, rows: int, mask: Optional[torch.Tensor] = None):
         """Logits and greedy choice of the pass's rows; a long pass only needs its last row, whose logits land in row 0."""

@@ -38,6 +38,7 @@ class GemmArgs(C.Structure):
         ("scatter_meta", C.c_void_p), ("wait_flags", C.c_void_p), ("wait_epoch", C.c_void_p),
         ("scatter_out", C.c_void_p * 8), ("max_tiles", C.c_int), ("wait_world", C.c_int), ("a_format", C.c_int), ("col_limit", C.c_void_p), ("alpha", C.c_float), ("alpha_batch", C.c_void_p),
         ("sig_counter", C.c_void_p), ("sig_epoch", C.c_void_p), ("sig_flags", C.c_void_p), ("sig_world", C.c_int),
+        ("act_alpha", C.c_float), ("act_shift", C.c_float), ("softcap", C.c_float),
     ]
 
 
@@ -136,7 +137,8 @@ def dir_functions():
         "ds41_resid_step", "ds41_polynorm", "ds41_gate_mul", "ds41_head_norm_gate", "ds41_gather_rows",
         "ds41_latent_post", "ds41_latent_query", "ds41_latent_gather", "ds41_latent_attend", "ds41_latent_merge",
         "ds41_latent_prefill", "ds41_mlstm_chunk",
-        "ds41_mlstm_step", "ds41_gemm_f32",
+        "ds41_mlstm_step", "ds41_gemm_f32", "ds41_side_act", "ds41_softcap_rows", "ds41_attn_post", "ds41_group_attend",
+        "ds41_group_prefill", "ds41_route_softmax", "ds41_gated_act",
     ]
 
 

@@ -1,5 +1,5 @@
-"""Front end of the layer-stack kernels (csrc/kernels/stack_ops.cu, latent_attn.cu, mlstm.cu, gemm_f32.cu) and the projection
-helper that the stack engine's matrix products go through."""
+"""Front end of the layer-stack kernels (csrc/kernels/stack_ops.cu, latent_attn.cu, group_attn.cu, mlstm.cu, moe.cu, gemm_f32.cu)
+and the projection helper that the stack engine's matrix products go through."""
 from __future__ import annotations
 
 import ctypes as C
@@ -30,7 +30,8 @@ class ResidArgs(C.Structure):
                 ("x_out", C.c_void_p), ("mix", C.c_void_p), ("kept", C.c_void_p), ("kept_stride", C.c_longlong),
                 ("x_avg", C.c_void_p), ("next_w", C.c_void_p), ("h", C.c_void_p), ("ldx", C.c_longlong),
                 ("ldh", C.c_int), ("n_mix", C.c_int), ("vocab", C.c_int), ("rows", C.c_int), ("W", C.c_int),
-                ("norm_kind", C.c_int), ("eps", C.c_float), ("f32", C.c_int)]
+                ("norm_kind", C.c_int), ("eps", C.c_float), ("f32", C.c_int), ("y_route", C.c_void_p), ("y_top", C.c_int),
+                ("y_rows", C.c_int), ("raw_h", C.c_int), ("post_rms", C.c_int)]
 
 
 class LatentPostArgs(C.Structure):
@@ -65,6 +66,31 @@ class MlstmArgs(C.Structure):
                 ("heads", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int), ("slots", C.c_int), ("ld_out", C.c_int)]
 
 
+class AttnPostArgs(C.Structure):
+    _fields_ = [("u", ProjArgs), ("conv", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("freq", C.c_void_p),
+                ("state", C.c_void_p), ("q", C.c_void_p), ("pool", C.c_void_p), ("page_table", C.c_void_p),
+                ("row_pos", C.c_void_p), ("row_slot", C.c_void_p), ("ld_q", C.c_longlong), ("eps", C.c_float),
+                ("rows", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int),
+                ("vdim_pad", C.c_int), ("rot_dim", C.c_int), ("taps", C.c_int), ("slots", C.c_int), ("max_pages", C.c_int),
+                ("page_tokens", C.c_int), ("f32", C.c_int)]
+
+
+class GroupAttendArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("pool", C.c_void_p), ("page_table", C.c_void_p), ("row_pos", C.c_void_p),
+                ("row_slot", C.c_void_p), ("out", C.c_void_p), ("status", C.c_void_p), ("gate", ProjArgs), ("u", ProjArgs),
+                ("state", C.c_void_p), ("ld_q", C.c_longlong), ("scale", C.c_float), ("rows", C.c_int), ("heads", C.c_int),
+                ("kv_heads", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int), ("chunk", C.c_int), ("taps", C.c_int),
+                ("slots", C.c_int), ("n_splits", C.c_int), ("ld_out", C.c_int), ("max_pages", C.c_int),
+                ("page_tokens", C.c_int), ("f32", C.c_int), ("n_pages", C.c_int), ("pos0", C.c_int)]
+
+
+class RouteArgs(C.Structure):
+    _fields_ = [("z", ProjArgs), ("bias", C.c_void_p), ("row_slot", C.c_void_p), ("ids", C.c_void_p), ("weights", C.c_void_p),
+                ("active", C.c_void_p), ("n_active", C.c_void_p), ("row_w", C.c_void_p), ("slot_of", C.c_void_p),
+                ("ticket", C.c_void_p), ("rows", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("max_active", C.c_int),
+                ("row_w_ld", C.c_int)]
+
+
 def mlstm_chunk_work(rows: int, heads: int, dim_pad: int, vdim_pad: int) -> int:
     """Bytes of workspace of the chunked recurrence (mostly the state before every chunk)."""
     fn = lib.kernels("stack").ds41_mlstm_chunk_work
@@ -89,6 +115,15 @@ class Proj:
 
     def args(self) -> ProjArgs:
         return ProjArgs(self.data.data_ptr(), self.plane, self.ld, self.splits, 1 if self.data.dtype == BF16 else 0, self.col)
+
+
+@dataclass
+class RoutedProj(Proj):
+    """Rows of routed experts whose sum is a pass row's result: row route[r * top + k] * rows + r, or, with rows = 0, one row
+    per route; negative routes count for nothing."""
+    route: Optional[torch.Tensor] = None
+    top: int = 1
+    rows: int = 0
 
 
 NO_PROJ = ProjArgs(None, 0, 0, 0, 0, 0)
@@ -196,7 +231,8 @@ def per_head(x: torch.Tensor, ldx: int, head_stride: int, rows: int, heads: int,
                a_batch_stride=n * ldw, b_batch_stride=head_stride, out_batch_stride=n, status=status, static_operand=1)
 
 
-def gemm_f32(a, b, out, M, N, K, lda, ldb, ldo, batch=1, sa=0, sb=0, so=0):
+def gemm_f32(a, b, out, M, N, K, lda, ldb, ldo, batch=1, sa=0, sb=0, so=0, batch_map=None, n_active=None):
     ll = C.c_longlong
     lib.check(lib.kernels("stack").ds41_gemm_f32(lib.ptr(a), lib.ptr(b), lib.ptr(out), M, N, K, ll(lda), ll(ldb), ll(ldo), batch,
-                                          ll(sa), ll(sb), ll(so), lib.stream()), "ds41_gemm_f32")
+                                          ll(sa), ll(sb), ll(so), lib.ptr(batch_map), lib.ptr(n_active),
+                                                 lib.stream()), "ds41_gemm_f32")

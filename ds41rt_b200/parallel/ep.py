@@ -35,8 +35,9 @@ class ExpertParallelMoE:
                  act_limit: float = 10.0, capacity: Optional[int] = None, w13_sf: Optional[torch.Tensor] = None,
                  w2_sf: Optional[torch.Tensor] = None, fp4: bool = False, nvfp4=None,
                  w13_gs: Optional[torch.Tensor] = None, w2_gs: Optional[torch.Tensor] = None,
-                 wire: str = "auto", tile_tokens: Optional[int] = None):
-        """w13: [E_local, 2*I, H] (gate rows then up rows), w2: [E_local, H, I]; bf16, or e4m3 with UE8M0 scale atoms,
+                 wire: str = "auto", tile_tokens: Optional[int] = None, act_alpha: float = 0.0, act_shift: float = 0.0):
+        """act_alpha / act_shift: the activation g sigmoid(alpha g) (u + shift) instead of silu(g) u (ops/gemm.py).
+        w13: [E_local, 2*I, H] (gate rows then up rows), w2: [E_local, H, I]; bf16, or e4m3 with UE8M0 scale atoms,
         or (fp4) E2M1 codes two per byte ([.., H/2] / [.., I/2] uint8) with UE8M0 scale atoms, or (nvfp4 = the two
         activation scales) E2M1 codes with E4M3 scale atoms per 16 and one global scale per expert (w13_gs / w2_gs):
         then the received rows and the FC1 output are quantised to NVFP4 too (W4A4).
@@ -56,11 +57,13 @@ class ExpertParallelMoE:
             self.H *= 2
         self.I = two_i // 2
         self.topk, self.max_tokens, self.act_limit = topk, max_tokens, act_limit
+        self.act_alpha, self.act_shift = act_alpha, act_shift
         assert wire in ("auto", "fp8", "bf16")
         self.wire_fp8 = self.mx and wire != "bf16"
         W, dev = fabric.world, fabric.device
-        assert self.H % 128 == 0 and self.I % 128 == 0 and W <= 8
         scaled = self.mx or self.nv is not None
+        unit = 128 if scaled else 8          # scale atoms, or just the copy engine's 16 bytes
+        assert self.H % unit == 0 and self.I % unit == 0 and W <= 8
         # FC1 tile width in tokens.  Gate and up accumulators share tensor memory with the scale columns: the block-scaled
         # FP8 kind still takes 128 tokens with a single accumulator set (half the weight bytes per token from L2, which
         # is what bounds it); NVFP4 carries four times the scale columns and stays at 64
@@ -171,6 +174,7 @@ class ExpertParallelMoE:
         a.tile_group, a.tile_row0 = lib.ptr(self.tile_group[t0:]), lib.ptr(self.tile_row0[t0:])
         a.tile_end, a.n_tiles_dev, a.max_tiles = lib.ptr(self.tile_end[t0:]), lib.ptr(self.n_tiles[table:]), self.max_tiles
         a.row_w, a.act_limit = lib.ptr(self.recv_w), self.act_limit
+        a.act_alpha, a.act_shift = self.act_alpha, self.act_shift
         if wait_phase is not None and self.f.world > 1:
             a.wait_flags, a.wait_epoch, a.wait_world = lib.ptr(self.flag_ptrs[wait_phase]), lib.ptr(self.epoch), self.f.world
         for key, val in kw.items():
@@ -179,7 +183,7 @@ class ExpertParallelMoE:
             a.scatter_meta = lib.ptr(self.recv_meta)
             for r, base in enumerate(self.sym.peer_ptrs):
                 a.scatter_out[r] = base + self.lay["comb"]
-        lib.check(lib.kernels().ds41_gemm_tc(C.byref(a), lib.stream()), "grouped gemm")
+        lib.check(lib.kernels("any").ds41_gemm_tc(C.byref(a), lib.stream()), "grouped gemm")
 
     def _mark(self, name: str) -> None:
         if self.marks is not None:
@@ -201,15 +205,16 @@ class ExpertParallelMoE:
         return acc
 
     # ------------------------------------------------------------------ the fused layer
-    def forward(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, out: torch.Tensor,
+    def forward(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, out: Optional[torch.Tensor],
                 extra: Optional[torch.Tensor] = None) -> None:
         """x [T,H] bf16, ids [T,topk] int32 (global expert ids), weights [T,topk] fp32 -> out [T,H] (bf16 or fp32).
 
+        out = None (one rank): the routes' rows stay in `comb` ([T * topk, H] bf16) for a consumer that sums them itself.
         `extra` ([T,H] fp32, e.g. the shared expert's output) is added before the routed rows, in a fixed order."""
         T = x.shape[0]
         assert T <= self.max_tokens and x.dtype == torch.bfloat16 and x.is_contiguous()
         assert ids.dtype == torch.int32 and weights.dtype == torch.float32
-        k, st, H, I = lib.kernels(), lib.stream, self.H, self.I
+        k, st, H, I = lib.kernels("any"), lib.stream, self.H, self.I
         a = self._ep_args(x, ids, weights, T)
         lib.check(k.ds41_ep_count(C.byref(a), st()), "ep_count")
         lib.check(k.ds41_ep_plan(C.byref(a), st()), "ep_plan")
@@ -258,6 +263,9 @@ class ExpertParallelMoE:
             self._mark("fc1")
             self._grouped(self.w2, self.act, self.comb, H, I, lda=I, ldo=H, out_mode=7, table=1)
             self._mark("fc2")
+        if out is None:
+            assert self.f.world == 1
+            return None
         lib.check(k.ds41_ep_mark(C.byref(a), 3, st()), "ep_mark")
         lib.check(k.ds41_ep_combine(C.byref(a), lib.ptr(self.comb), lib.ptr(extra),
                                     C.c_longlong(extra.stride(0) if extra is not None else 0), lib.ptr(out),

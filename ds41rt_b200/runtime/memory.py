@@ -47,22 +47,22 @@ def kv_row_bytes(cfg: ModelConfig, kv_dtype: str) -> tuple:
 
 
 def stack_page_bytes(cfg: StackConfig, page_tokens: int, elem: int = 2) -> int:
-    from ..models.stack import latent_row_len
-    return sum(page_tokens * latent_row_len(cfg.layers[l].mixer)[1] * elem for l in cfg.cache_layers())
+    from ..models.stack import cache_row_len
+    return sum(page_tokens * cache_row_len(cfg.layers[l].mixer) * elem for l in cfg.cache_layers())
 
 
 def stack_state_bytes(cfg: StackConfig) -> int:
-    """fp32 recurrent state of one request."""
+    """fp32 state of one request besides its cache rows (recurrences, inputs of convolutions)."""
     import math
-    from ..models.stack import mlstm_state_shapes
-    return sum(4 * math.prod(s) for l in cfg.state_layers() for s in mlstm_state_shapes(cfg.layers[l].mixer))
+    from ..models.stack import state_shapes
+    return sum(4 * math.prod(s) for l in cfg.state_layers() for s in state_shapes(cfg.layers[l].mixer))
 
 
 def plan_pool(cfg: ModelConfig, *, n_layers: int, slots: int, max_context: int, free_bytes: int, kv_dtype: str = "bf16",
               page_tokens: int = 64, retained: int = 40, ring_rows: Optional[int] = None,
               reserve_bytes: int = 0) -> PoolPlan:
     if isinstance(cfg, StackConfig):
-        # latent rows of the layers that produce them; recurrent states (one per slot, and per retained snapshot) stand
+        # cache rows of the layers that produce them; states (one per slot, and per retained snapshot) stand
         # where the other models have their window rings
         per_page, state = stack_page_bytes(cfg, page_tokens), stack_state_bytes(cfg)
         ring_bytes = state * (slots + retained)
