@@ -18,7 +18,7 @@ snapshot, 1024 output tokens, paged FP8 KV rows; 5 = speculative C1 decode over 
 vocabulary mask on the target's choices.
 
   python bench.py --gpus N --steps K --warmup W          (N > 1: launched by torch.distributed.run)
-  python bench.py --stack genesun-1b,genesun-7b          (layer-stack models beside ds41 models of equal size; one GPU)
+  python bench.py --stack genesun-1b,belasun-1b          (layer-stack models beside ds41 models of equal size; one GPU)
   python bench.py --impl reference ...                   (prints the reference arm's availability line)
 
 Prints ONE JSON line on rank 0.  `value` is device-timed (CUDA events on the launching stream, barrier and
@@ -450,7 +450,7 @@ def main():
                     help="prefill: the decoder layers run over the last 128 prompt tokens only (the reference's prompt "
                          "scheme); default is every layer over every token")
     ap.add_argument("--ced-boundary", type=int, default=0, help="first decoder layer for --ced on a truncated stack")
-    ap.add_argument("--stack", default="", help="layer-stack presets (comma-separated, e.g. genesun-1b,genesun-7b): prompt "
+    ap.add_argument("--stack", default="", help="layer-stack presets (comma-separated, e.g. genesun-1b,belasun-1b): prompt "
                     "and decode throughput beside ds41 models of equal size; --prompt, --chunk (default 2048), --layers")
     ap.add_argument("--breakdown", action="store_true", help="prefill: per-kernel device time of one prompt (stderr)")
     args = ap.parse_args()

@@ -16,7 +16,7 @@ import torch
 
 from ..config import ModelConfig, RopeConfig
 from ..models import registry
-from ..models.stack import mlstm_state_shapes
+from ..models.stack import state_shapes
 from ..runtime.session import DecodeSession
 from ..stack_config import StackConfig
 
@@ -33,34 +33,41 @@ def peaks() -> dict:
 
 
 def ds41_like(cfg: StackConfig) -> ModelConfig:
-    """A ds41 configuration of the same width, depth and vocabulary whose active weights per token are close to cfg's."""
+    """A ds41 configuration of the same width, depth and vocabulary whose active weights per token are close to cfg's (with
+    as many experts, where cfg has mixtures)."""
     W, L = cfg.hidden, cfg.n_layers
-    attn = [l.mixer for l in cfg.layers if l.mixer.kind == "latent_attention"]
+    attn = [l.mixer for l in cfg.layers if l.mixer.kind != "mlstm"]
+    moe = next((l.mlp for l in cfg.layers if l.mlp is not None and l.mlp.kind == "moe"), None)
     heads = max(m.heads for m in attn)
-    q = max(m.q_rank for m in attn)
+    q = max(getattr(m, "q_rank", W // 4) for m in attn)
     groups = max(1, heads // 4)
     D, o_lora = 512, 1024 if W >= 4096 else 512
     dense = (q + D) * W + q * heads * D + groups * o_lora * (heads // groups) * D + W * groups * o_lora
     left = stack_layer_weights(cfg) / L - dense
-    topk = 3
+    experts, topk = (moe.experts, moe.top) if moe is not None else (4, 3)
     inter = max(128, int(left / (3 * W * (topk + 1))) // 128 * 128)
     c = ModelConfig(name=f"ds41-like-{cfg.name}", vocab=cfg.vocab, hidden=W, n_layers=L, n_heads=heads, head_dim=D, q_lora=q,
                     o_groups=groups, o_lora=o_lora, window=128, source_layers={0: 1}, compress_ratios=[1] * L,
                     index_layers=tuple(range(0, L, 4)), index_topk=512, candidate_layer=-1, candidate_topk_blocks=0,
-                    n_experts=4, topk=topk, inter=inter, rope_long=RopeConfig(), dspark=None, engram=None, vision=None)
+                    n_experts=experts, topk=topk, inter=inter, rope_long=RopeConfig(), dspark=None, engram=None, vision=None)
     c.validate()
     return c
 
 
 def stack_layer_weights(cfg: StackConfig) -> int:
-    """Matrix weights of all layers (read once per decode step)."""
-    from ..models import genesun
-    return sum(s[0] * s[1] for l in range(cfg.n_layers) for s in genesun.layer_shapes(cfg, l).values() if len(s) == 2)
+    """Matrix weights of all layers that one token uses."""
+    fam = registry.family_of(cfg)
+    total = 0
+    for l, spec in enumerate(cfg.layers):
+        unused = spec.mlp.experts - spec.mlp.top if spec.mlp is not None and spec.mlp.kind == "moe" else 0
+        total += sum(s[0] * s[1] for s in fam.layer_shapes(cfg, l).values() if len(s) == 2)
+        total -= unused * 3 * cfg.hidden * (spec.mlp.ff if unused else 0)
+    return total
 
 
-def work(cfg: StackConfig, R: int, n_keys: int, first: int, decode: bool) -> Dict[str, Tuple[float, float]]:
+def work(cfg: StackConfig, R: int, n_keys: int, first: int, decode: bool, active: int = 0) -> Dict[str, Tuple[float, float]]:
     """Kernel class -> (algorithmic bytes, FLOPs) of one pass of R rows (decode: R requests of n_keys positions each; else
-    one request's rows [first, n_keys)), summed over the layers."""
+    one request's rows [first, n_keys)), summed over the layers.  `active`: experts that a planned pass uses."""
     W, out = cfg.hidden, {}
     act = 4 if decode else 2           # projections leave as fp32 planes in decode, as bf16 in long passes
 
@@ -71,10 +78,27 @@ def work(cfg: StackConfig, R: int, n_keys: int, first: int, decode: bool) -> Dic
     def gemm(tag, n, k, out_bytes):
         add(tag, 2.0 * n * k + R * (2.0 * k + out_bytes * n), 2.0 * R * n * k)
 
-    pairs = R * n_keys if decode else sum(range(first + 1, n_keys + 1))
+    def seen(pos, chunk):
+        return pos % chunk + 1 if chunk else pos + 1
+
     for l, spec in enumerate(cfg.layers):
         m = spec.mixer
-        if m.kind == "latent_attention":
+        chunk = getattr(m, "chunk", 0)
+        pairs = R * seen(n_keys - 1, chunk) if decode else sum(seen(p, chunk) for p in range(first, n_keys))
+        if m.kind == "grouped_attention":
+            H, G = m.heads, m.kv_heads
+            cols, row = H * m.dim + G * (m.dim + m.vdim), G * (m.dim + m.vdim)
+            back = max(m.taps - 1, 0)
+            gemm("gemm_mix_in", cols + (H if m.head_gate else 0), W, act)
+            add("attn_post", R * cols * (act + 2.0) + 4.0 * cols * max(m.taps, 1) + (4.0 * R * back * cols if decode else 0))
+            if decode:
+                add("group_attend", pairs * row * 2.0 + R * H * (m.dim + m.vdim) * 2.0 + (8.0 * R * cols if back else 0),
+                    2.0 * pairs * H * (m.dim + m.vdim))
+            else:
+                low = first - first % chunk if chunk else 0
+                add("group_prefill", (n_keys - low) * row * 2.0 + R * H * (m.dim + m.vdim) * 2.0, 2.0 * pairs * H * (m.dim + m.vdim))
+            gemm("gemm_o", W, H * m.vdim, 4)
+        elif m.kind == "latent_attention":
             own = m.kv_from is None
             H, kv = m.heads, m.kv_rank + m.rot_dim
             gemm("gemm_mix_in", m.q_rank + (kv if own else 0) + H * m.vdim + W, W, act)
@@ -108,15 +132,33 @@ def work(cfg: StackConfig, R: int, n_keys: int, first: int, decode: bool) -> Dic
                     R * H * (2.0 * 64 * (D + V) + 4.0 * D * V))
             add("head_norm_gate", R * H * V * (6.0 + act))
             gemm("gemm_o", W, H * V, 4)
-        n_resid = 1
-        if spec.mlp is not None:
-            ff = spec.mlp.ff
-            gemm("gemm_up", ff + W, W, act)
-            add("polynorm", R * ff * (act + 2.0))
-            gemm("gemm_down", W, ff, 4)
-            n_resid = 2
-        # result, gate and stream in, stream and next input out; the depth average reads every kept stream and writes one
-        add("resid_step", R * W * (n_resid * (4.0 + act + 4 + 4 + 2) + 4.0 * (l + 1) + 4))
+        ml = spec.mlp
+        gate = act if cfg.residual_gate else 0
+        # result, gate and stream in, stream and next input out
+        add("resid_step", R * W * (4.0 + gate + 4 + 4 + 2))
+        if ml is not None and ml.kind == "dense":
+            gemm("gemm_up", ml.ff + W, W, act)
+            add("polynorm", R * ml.ff * (act + 2.0))
+            gemm("gemm_down", W, ml.ff, 4)
+            add("resid_step", R * W * (4.0 + gate + 4 + 4 + 2))
+        elif ml is not None:
+            routes = R * ml.top
+            gemm("gemm_router", ml.experts, W, 4)
+            add("route", R * ml.experts * 4.0 + routes * 8.0)
+            if decode and active:
+                add("gemm_fc1", active * 4.0 * ml.ff * W + R * 2.0 * W + routes * 2.0 * ml.ff, routes * 4.0 * ml.ff * W)
+                add("gemm_fc2", active * 2.0 * ml.ff * W + routes * (2.0 * ml.ff + 4.0 * W), routes * 2.0 * ml.ff * W)
+            else:
+                used = min(ml.experts, routes)
+                add("ep_moe", used * 6.0 * ml.ff * W + R * 2.0 * W + routes * 2.0 * (2 * W + 2 * ml.ff), routes * 6.0 * ml.ff * W)
+            add("resid_step", R * W * (ml.top * (4.0 if decode and active else 2.0) + gate + 4 + 4 + 2))
+        if cfg.token_side:
+            gemm("gemm_side_gate", cfg.token_side, W, 4)
+            add("side_act", R * cfg.token_side * 8.0)
+            gemm("gemm_side_proj", W, cfg.token_side, 4)
+            add("resid_step", R * W * (4.0 + 4 + 4 + 2))
+        if cfg.depth_average:          # reads every kept stream and writes the sum
+            add("resid_step", R * W * (4.0 * (l + 1) + 4))
     add("resid_step", R * W * 8.0)
     heads = R if decode else 1
     add("gemm_head", 2.0 * cfg.vocab * W + 4.0 * heads * cfg.vocab, 2.0 * heads * cfg.vocab * W)
@@ -187,7 +229,7 @@ def bench_engine(e, prompt_len: int, chunk: int, batches, steps: int, warmup: in
     for B in batches:
         for s in range(B):
             assert e.cache.ensure(s, context + 4 * (steps + warmup) + 64)
-        rows = ([5] * B, [context] * B, list(range(B)))
+        rows = ([(5 + 37 * s) % e.cfg.vocab for s in range(B)], [context] * B, list(range(B)))
         ses = DecodeSession(e)
         e.set_rows(*rows)
         ses.graph(B, feedback=True)
@@ -197,6 +239,7 @@ def bench_engine(e, prompt_len: int, chunk: int, batches, steps: int, warmup: in
         # a kernel class alone: the same graph with every other launch left out
         e.set_rows(*rows)
         counts = {t: c for t, (c, _) in _classes(e, lambda: e.forward_rows(B)).items()}
+        active = int(e.n_active) if work_of and "gemm_fc1" in counts else 0      # what the last layer's routes left
         acc = {}
         for tag, c in counts.items():
             e.only = {tag}
@@ -208,7 +251,7 @@ def bench_engine(e, prompt_len: int, chunk: int, batches, steps: int, warmup: in
             e.only = None
         rep["decode"].append({"batch": B, "context": context, "ms_per_step": round(ms, 4), "tok_s": round(B / ms * 1e3, 1),
                               "launches": launches,
-                              "kernels": table(acc, work_of(B, context + 1, 0, True) if work_of else None)})
+                              "kernels": table(acc, work_of(B, context + 1, 0, True, active) if work_of else None)})
         e.check_status("decode")
         for s in range(B):
             e.cache.release(s)
@@ -219,7 +262,7 @@ def run(names: List[str], dev, steps: int, warmup: int, prompt: int, chunk: int,
         batches=(1, 8, 32)) -> dict:
     out = {"peaks": peaks(), "models": {}}
     for name in names:
-        fam, cfg = registry.preset(name, layers or {"genesun-1b": 16, "genesun-7b": 8}.get(name, 0))
+        fam, cfg = registry.preset(name, layers or {"1b": 16, "7b": 8}.get(name.split("-")[-1], 0))
         like = ds41_like(cfg)
         max_ctx = max(prompt, context + 4 * (steps + warmup) + 64) // 64 * 64 + 128
         for family, c in ((fam, cfg), (registry.FAMILIES["ds41"], like)):
@@ -233,7 +276,7 @@ def run(names: List[str], dev, steps: int, warmup: int, prompt: int, chunk: int,
                        else ds41_active(c))
             if family is fam:
                 rep["state_mb_per_request"] = round(sum(4 * _prod(s) for l in c.state_layers()
-                                                        for s in mlstm_state_shapes(c.layers[l].mixer)) / 1e6, 2)
+                                                        for s in state_shapes(c.layers[l].mixer)) / 1e6, 2)
             out["models"][c.name] = rep
             del e, w
             torch.cuda.empty_cache()
