@@ -603,9 +603,10 @@ typedef struct ds41_group_attend_args {
   long long ld_q;
   float scale;
   int rows, heads, kv_heads, dim_pad, vdim_pad, chunk, taps, slots, n_splits, ld_out, max_pages, page_tokens, f32;
-  int n_pages, pos0;              // long passes: pages of the pool, position of row 0
+  int n_pages;                    // pages of the pool
+  int pos0;                       // long passes: position of row 0
 } ds41_group_attend_args;
-// Any mix of rows; n_splits <= 8 CTAs share a row's keys.
+// Any mix of rows; n_splits <= 16 CTAs share a row's keys.
 int ds41_group_attend(const ds41_group_attend_args* args, void* stream);
 // Long prompt pass of one request (bf16, dim_pad <= 256, vdim_pad <= 128, pages of 32, 64 or 128 tokens): row r stands at
 // position pos0 + r.

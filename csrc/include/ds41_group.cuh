@@ -8,13 +8,14 @@ namespace ds41 {
 __host__ __device__ __forceinline__ int chunk_start(int pos, int chunk) { return chunk > 0 ? pos - pos % chunk : 0; }
 
 // If row r is one of the last taps - 1 rows of its request in this pass, its share of the convolution's inputs goes into the
-// request's ring.  `part` of `parts` blocks works on the row.
-__device__ __forceinline__ void keep_inputs(const ds41_group_attend_args& p, int r, int slot, int pos, int part, int parts) {
+// request's ring.  `part` of `parts` blocks works on the row, with `threads` threads each.
+__device__ __forceinline__ void keep_inputs(const ds41_group_attend_args& p, int r, int slot, int pos, int part, int parts,
+                                            int thread, int threads) {
   const int back = p.taps - 1;
   if (back <= 0 || (r + back < p.rows && p.row_slot[r + back] == slot)) return;
   const int C = (p.heads + p.kv_heads) * p.dim_pad + p.kv_heads * p.vdim_pad;
   float* ring = p.state + (1ll * slot * back + pos % back) * C;
-  for (int c = 4 * (part * blockDim.x + threadIdx.x); c < C; c += 4 * parts * blockDim.x)
+  for (int c = 4 * (part * threads + thread); c < C; c += 4 * parts * threads)
     *reinterpret_cast<float4*>(ring + c) = proj_at4(p.u, r, c);
 }
 

@@ -77,7 +77,7 @@ __global__ void __launch_bounds__(256) keep_inputs_kernel(ds41_group_attend_args
   pdl_wait();
   const int r = p.rows - 1 - static_cast<int>(blockIdx.y);
   if (r < 0 || p.row_slot[r] < 0) return;
-  keep_inputs(p, r, p.row_slot[r], p.row_pos[r], blockIdx.x, gridDim.x);
+  keep_inputs(p, r, p.row_slot[r], p.row_pos[r], blockIdx.x, gridDim.x, threadIdx.x, blockDim.x);
 }
 
 }  // namespace ds41

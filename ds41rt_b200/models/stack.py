@@ -345,7 +345,8 @@ class GroupedAttention:
         sp = self.spec
         span = min(sp.chunk or e.cache.max_ctx, e.cache.max_ctx)
         blocks = rows * sp.kv_heads * -(-(sp.heads // sp.kv_heads) // 16)
-        return max(1, min(2 * 148 // blocks, 8, -(-span // 64)))
+        n = max(1, min(2 * 148 // blocks, 16, -(-span // 128)))
+        return n if n <= 8 or n == 16 else 8
 
     def run(self, e: "StackEngine", l: int, R: int, src: int) -> Tuple[Proj, Optional[Proj]]:
         sp, k, c = self.spec, e.k, e.cache
@@ -371,8 +372,9 @@ class GroupedAttention:
         b.u, b.state, b.ld_q, b.scale = u.args(), lib.ptr(state), ldq, sp.scale
         b.rows, b.heads, b.kv_heads, b.dim_pad, b.vdim_pad, b.chunk = R, sp.heads, sp.kv_heads, self.dp, self.vp, sp.chunk
         b.taps, b.slots, b.ld_out, b.max_pages, b.page_tokens, b.f32 = a.taps, c.slots, ldo, c.max_pages, c.page_tokens, e.f32
+        b.n_pages = c.n_pages
         if long:
-            b.n_pages, b.pos0, b.n_splits = c.n_pages, long - R, 1
+            b.pos0, b.n_splits = long - R, 1
             e._run("group_prefill", k.ds41_group_prefill, C.byref(b), lib.stream())
         else:
             b.n_splits = self.splits(e, R)

@@ -340,7 +340,7 @@ SHAPES = [(6, 2, 20, 24), (3, 3, 64, 64), (8, 1, 128, 128), (40, 2, 48, 80), (1,
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("splits", [1, 3, 8])
+@pytest.mark.parametrize("splits", [1, 3, 16])
 @pytest.mark.parametrize("shape", SHAPES)
 def test_attention_over_pages_and_chunks(shape, splits, dtype):
     """Rows around chunk borders: the last position of a chunk, the first of the next, the middle; or everything visible."""
@@ -435,6 +435,7 @@ class Post:
             b.gate, b.u, b.ld_q, b.scale = S.NO_PROJ, a.u, H * dp, 1.0
             b.rows, b.heads, b.kv_heads, b.dim_pad, b.vdim_pad, b.chunk, b.taps, b.slots = n, H, G, dp, vp, 0, back + 1, 2
             b.n_splits, b.ld_out, b.max_pages, b.page_tokens, b.f32 = splits, H * vp, a.max_pages, page, a.f32
+            b.n_pages = pages.total
             _ok(k.ds41_group_attend(C.byref(b), lib.stream()))
             torch.cuda.synchronize()
             out_q.append(q.cpu().double())
@@ -603,7 +604,7 @@ def test_bad_arguments_are_refused_on_the_host():
         assert getattr(k, f"ds41_{fn}")(C.byref(args()), lib.stream()) != 0 and getattr(k, f"ds41_{fn}")(None, lib.stream()) != 0
     c = Attention(4, 2, 64, 32, 100, 3, 64, BF16)
     with pytest.raises(AssertionError):
-        c.run("attend", splits=9)
+        c.run("attend", splits=17)
     c.pages.page = 48                                                      # a page size the long-pass form does not take
     with pytest.raises(AssertionError):
         c.run("prefill")
