@@ -169,7 +169,34 @@ __device__ __forceinline__ void post_store(const ds41_attn_post_args& p, const P
   store4(dst + (t.b - off), make_float4(o[4], o[5], o[6], o[7]));
 }
 
-template <int RB, int THREADS>
+// A unit of a projection row as it was loaded: bf16 pairs, or eight floats.
+template <bool PACKED>
+struct RawUnit {
+  uint2 a, b;
+  __device__ __forceinline__ void load(const ds41_proj& u, long long r, const PostUnit& t) {
+    const __nv_bfloat16* row = static_cast<const __nv_bfloat16*>(u.data) + r * u.ld + u.col;
+    a = *reinterpret_cast<const uint2*>(row + t.a);
+    b = *reinterpret_cast<const uint2*>(row + t.b);
+  }
+  __device__ __forceinline__ Eight get() const {
+    const uint32_t q[4] = {a.x, a.y, b.x, b.y};
+    Eight x;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x.v[2 * i] = __uint_as_float(q[i] << 16);
+      x.v[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
+    }
+    return x;
+  }
+};
+template <>
+struct RawUnit<false> {
+  Eight x;
+  __device__ __forceinline__ void load(const ds41_proj& u, long long r, const PostUnit& t) { x = proj_unit(u, r, t); }
+  __device__ __forceinline__ Eight get() const { return x; }
+};
+
+template <int RB, int THREADS, bool PACKED>
 __global__ void __launch_bounds__(THREADS) attn_post_rows_kernel(ds41_attn_post_args p) {
   extern __shared__ float2 pr_turns[];             // [kPostRows][rot_dim / 2]
   __shared__ float red[2][THREADS / 32][RB];       // sums of squares per row of a batch
@@ -196,31 +223,35 @@ __global__ void __launch_bounds__(THREADS) attn_post_rows_kernel(ds41_attn_post_
   }
   int parity = 0;
   for (int rb = r0; rb < r1; rb += RB, parity ^= 1) {
-    Eight acc[RB];
-    int slot[RB], pos[RB];
+    constexpr int kOld = kPostTaps - 1;              // rows before the batch that it reaches
+    int own[kOld + RB], pos[RB];                   // slots of rows rb - kOld ..., -1 beyond the pass
 #pragma unroll
-    for (int j = 0; j < RB; ++j) {
-      slot[j] = rb + j < r1 ? p.row_slot[rb + j] : -1;
-      pos[j] = rb + j < r1 ? p.row_pos[rb + j] : 0;
+    for (int i = 0; i < kOld + RB; ++i) {
+      const int r = rb + i - kOld;
+      own[i] = r >= 0 && r < r1 && i >= kOld - back ? p.row_slot[r] : -1;
+    }
+#pragma unroll
+    for (int j = 0; j < RB; ++j) pos[j] = rb + j < r1 ? p.row_pos[rb + j] : 0;
+    RawUnit<PACKED> raw[kOld + RB];
+#pragma unroll
+    for (int i = 0; i < kOld + RB; ++i)
+      if (live && own[i] >= 0) raw[i].load(p.u, rb + i - kOld, t);
+    Eight acc[RB];
+#pragma unroll
+    for (int j = 0; j < RB; ++j)
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[j].v[e] = 0.f;
-    }
     if (live) {
-      // rows of this pass, from the oldest one that the batch reaches
 #pragma unroll
-      for (int s = 1 - kPostTaps; s < RB; ++s) {
-        const int r = rb + s;
-        if (r < 0 || s < -back || r >= r1) continue;
-        const int owner = p.row_slot[r];
-        if (owner < 0) continue;
-        const Eight x = proj_unit(p.u, r, t);
+      for (int i = 0; i < kOld + RB; ++i) {
+        if (own[i] < 0) continue;
+        const Eight x = raw[i].get();
 #pragma unroll
         for (int j = 0; j < RB; ++j) {
-          constexpr int kMost = kPostTaps - 1;
-          if (j >= s && j - s <= kMost && slot[j] == owner) {
+          const int d = j + kOld - i;              // positions back from row j, if both belong to one request
+          if (d >= 0 && d < kPostTaps && own[kOld + j] == own[i])
 #pragma unroll
-            for (int e = 0; e < 8; ++e) acc[j].v[e] += w[j - s < kPostTaps && j >= s ? j - s : 0].v[e] * x.v[e];
-          }
+            for (int e = 0; e < 8; ++e) acc[j].v[e] += w[d >= 0 && d < kPostTaps ? d : 0].v[e] * x.v[e];
         }
       }
       // what earlier passes left, for the first rows of a request's portion
@@ -228,9 +259,9 @@ __global__ void __launch_bounds__(THREADS) attn_post_rows_kernel(ds41_attn_post_
       for (int j = 0; j < RB; ++j)
 #pragma unroll
         for (int d = 1; d < kPostTaps; ++d) {
-          const int r = rb + j - d;
-          if (slot[j] < 0 || d > back || d > pos[j] || (r >= 0 && p.row_slot[r] == slot[j])) continue;
-          const Eight x = row_unit(p.state + (1ll * slot[j] * back + (pos[j] - d) % back) * C, t);
+          const int slot = own[kOld + j];
+          if (slot < 0 || d > back || d > pos[j] || own[kOld + j - d] == slot) continue;
+          const Eight x = row_unit(p.state + (1ll * slot * back + (pos[j] - d) % back) * C, t);
 #pragma unroll
           for (int e = 0; e < 8; ++e) acc[j].v[e] += w[d].v[e] * x.v[e];
         }
@@ -256,7 +287,8 @@ __global__ void __launch_bounds__(THREADS) attn_post_rows_kernel(ds41_attn_post_
     __syncthreads();                               // sums, and the sines of the first batch
 #pragma unroll
     for (int j = 0; j < RB; ++j) {
-      if (slot[j] < 0) continue;
+      const int slot = own[kOld + j];
+      if (slot < 0) continue;
       float f = 1.f;
       if (p.q_norm != nullptr) {                   // every lane takes part: a warp may hold keys and values
         const float q = warp_sum(lane < n_warps ? red[parity][lane][j] : 0.f);
@@ -265,7 +297,7 @@ __global__ void __launch_bounds__(THREADS) attn_post_rows_kernel(ds41_attn_post_
       if (!live) continue;
       __nv_bfloat16* row = blockIdx.y == 0 ? nullptr
                                            : cache_row(static_cast<__nv_bfloat16*>(p.pool), p.page_table, p.max_pages,
-                                                       p.page_tokens, nk + nv, slot[j], pos[j]);
+                                                       p.page_tokens, nk + nv, slot, pos[j]);
       post_store(p, t, acc[j], f, pr_turns + (rb - r0 + j) * half, static_cast<__nv_bfloat16*>(p.q) + (rb + j) * p.ld_q, row);
     }
   }
@@ -370,8 +402,15 @@ static int launch_post_fast(const ds41_attn_post_args& a, cudaStream_t st, bool&
   const int most = q_units > units - q_units ? q_units : units - q_units, threads = (most + 31) / 32 * 32;
   const dim3 grid((a.rows + kPostRows - 1) / kPostRows, 2);
   const int smem = kPostRows * (a.rot_dim / 2) * static_cast<int>(sizeof(float2));
-  if (threads <= 512 && smem <= 40 * 1024) return launch_pdl(attn_post_rows_kernel<4, 512>, grid, dim3(threads), smem, st, a);
-  if (threads <= 1024 && smem <= 40 * 1024) return launch_pdl(attn_post_rows_kernel<2, 1024>, grid, dim3(threads), smem, st, a);
+  if (threads <= 1024 && smem <= 40 * 1024) {
+    if (threads > 512)
+      return a.u.bf16 ? launch_pdl(attn_post_rows_kernel<2, 1024, true>, grid, dim3(threads), smem, st, a)
+                      : launch_pdl(attn_post_rows_kernel<2, 1024, false>, grid, dim3(threads), smem, st, a);
+    if (threads > 256 || !a.u.bf16)
+      return a.u.bf16 ? launch_pdl(attn_post_rows_kernel<4, 512, true>, grid, dim3(threads), smem, st, a)
+                      : launch_pdl(attn_post_rows_kernel<2, 512, false>, grid, dim3(threads), smem, st, a);
+    return launch_pdl(attn_post_rows_kernel<4, 256, true>, grid, dim3(threads), smem, st, a);
+  }
   done = false;
   return cudaSuccess;
 }
@@ -436,23 +475,20 @@ __global__ void __launch_bounds__(128) group_attend_plain_kernel(ds41_group_atte
   for (int i = tid; i < p.vdim_pad; i += 128) out[i] = from_f32<T>(os[i] * f);
 }
 
-// bf16 form: CTA (split, key/value head and 16 of its query heads, row).  A producer warp brings tiles of 64 keys and values
-// page by page with TMA (128-byte swizzle) through a ring of stages; each of four warps scores 16 of the 64 keys and
+// bf16 form: CTA (split, key/value head and 16 of its query heads, row).  A producer warp brings tiles of 16 NW keys and values
+// page by page with TMA (128-byte swizzle) through a ring of stages; each of NW warps scores 16 of the keys and
 // accumulates their values with a softmax state of its own - no block-wide wait until the partial results are merged: over
 // the warps in shared memory, over the CTAs of the cluster through distributed shared memory.
-// KD: 16-column pieces of the key width, NP: of the value width.
-constexpr int kTileKeys = 64;
-constexpr int kAttendWarps = 4;
-constexpr int kAttendThreads = 32 * (kAttendWarps + 1);
-constexpr int kTileChunk = kTileKeys * 128;           // bytes of 64 rows x 64 bf16 columns
+// KD: 16-column pieces of the key width, NP: of the value width.  A warp's walk is a chain of latencies, so a CTA has eight
+// of them; four, and two CTAs share an SM, where there are more CTAs than SMs (or the value width takes the registers).
+constexpr int kMaxStages = 4;
 
 struct AttendPlan {
-  int kc, vc, stages, box;                            // 64-column chunks, ring length, rows per TMA box
-  int stage_bytes() const { return (kc + vc) * kTileChunk; }
+  int warps, kc, vc, stages, box;                     // 64-column chunks, ring length, rows per TMA box
 };
 
 inline int attend_smem(const AttendPlan& t, int dp) {
-  return 1024 + t.stages * t.stage_bytes() + 16 * (dp + 8) * 2 + (kAttendWarps + 1) * 32 * 4 + 128;
+  return 1024 + t.stages * (t.kc + t.vc) * t.warps * 16 * 128 + 16 * (dp + 8) * 2 + (t.warps + 1) * 32 * 4 + 16 * kMaxStages;
 }
 
 // Tiles and pages of this launch; false: the plain form has to run.
@@ -460,33 +496,43 @@ inline bool plan_attend(const ds41_group_attend_args& a, AttendPlan& t) {
   if (a.f32 || a.vdim_pad > 256 || a.dim_pad > 256 || a.n_pages <= 0 || (a.ld_q & 7) || (a.ld_out & 3) ||
       ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.pool)) & 15) || (reinterpret_cast<uintptr_t>(a.out) & 7))
     return false;
-  t.box = a.page_tokens % kTileKeys == 0 ? kTileKeys : a.page_tokens;
-  if (t.box < 8 || kTileKeys % t.box != 0) return false;
   t.kc = (a.dim_pad + 63) / 64;
   t.vc = (a.vdim_pad + 63) / 64;
-  t.stages = 3;
-  return attend_smem(t, a.dim_pad) <= 226 * 1024;
+  const int m_tiles = (a.heads / a.kv_heads + 15) / 16;
+  const bool many = 1ll * a.n_splits * a.kv_heads * m_tiles * a.rows > sm_count();
+  for (t.warps = a.vdim_pad <= 128 && !many ? 8 : 4; t.warps >= 4; t.warps -= 4) {
+    const int keys = 16 * t.warps;
+    t.box = a.page_tokens % keys == 0 ? keys : a.page_tokens;
+    if (t.box < 8 || keys % t.box != 0) continue;
+    // the partial results of the warps and of the CTA take the place of the stages
+    const int merge = (t.warps + 1) * 16 * a.vdim_pad * 4, stage = (t.kc + t.vc) * keys * 128;
+    for (int room : {many ? 112 : 226, 226})
+      for (t.stages = kMaxStages; t.stages >= 2; --t.stages)
+        if (attend_smem(t, a.dim_pad) <= room * 1024 && t.stages * stage >= merge) return true;
+  }
+  return false;
 }
 
-template <int KD, int NP>
-__global__ void __launch_bounds__(kAttendThreads)
+template <int NW, int KD, int NP>
+__global__ void __launch_bounds__(32 * (NW + 1))
 group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_group_attend_args p, const AttendPlan plan) {
+  constexpr int kTileKeys = 16 * NW, kTileChunk = kTileKeys * 128;      // bytes of a tile's rows x 64 bf16 columns
   extern __shared__ uint8_t gm_raw[];
   uint8_t* stages = gm_raw + ((1024u - (smem_u32(gm_raw) & 1023u)) & 1023u);
   const int dp = p.dim_pad, vp = p.vdim_pad, KS = dp + 8, stage_bytes = (plan.kc + plan.vc) * kTileChunk;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, q2 = 2 * (lane & 3);
   __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(stages + plan.stages * stage_bytes);   // [16][KS]
   float* ml = reinterpret_cast<float*>(sq + 16 * KS);                                         // [warp][16]{max, sum}
-  float* cml = ml + kAttendWarps * 32;                                                        // [16]{max, sum} of the CTA
+  float* cml = ml + NW * 32;                                                        // [16]{max, sum} of the CTA
   uint64_t* full = reinterpret_cast<uint64_t*>(cml + 32);                                     // [stages]
-  uint64_t* empty = full + 4;
+  uint64_t* empty = full + kMaxStages;
   const int n = p.heads / p.kv_heads, m_tiles = (n + 15) / 16;
   const int split = blockIdx.x, g = blockIdx.y / m_tiles, h0 = g * n + (blockIdx.y % m_tiles) * 16, r = blockIdx.z;
   const int h_end = (g + 1) * n;                                               // heads [h0, min(h0 + 16, h_end))
   if (tid == 0) {
     for (int i = 0; i < plan.stages; ++i) {
       mbar_init(&full[i], 1);
-      mbar_init(&empty[i], kAttendWarps);
+      mbar_init(&empty[i], NW);
     }
     mbar_init_fence();
     tma_prefetch_desc(&pool);
@@ -504,8 +550,8 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
   const int first = chunk_start(pos, p.chunk), base = first - first % plan.box;
   const int tiles = (pos - base) / kTileKeys + 1, per = (tiles + p.n_splits - 1) / p.n_splits;
   const int t0 = min(tiles, split * per), t1 = min(tiles, t0 + per);
-  if (warp < kAttendWarps) {
-    for (int i = warp; i < 16; i += kAttendWarps) {
+  if (warp < NW) {
+    for (int i = warp; i < 16; i += NW) {
       const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + r * p.ld_q + (h0 + i) * dp;
       for (int d = lane * 8; d < dp; d += 256)
         *reinterpret_cast<uint4*>(sq + i * KS + d) = h0 + i < h_end ? *reinterpret_cast<const uint4*>(q + d) : make_uint4(0, 0, 0, 0);
@@ -514,7 +560,7 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
   __syncthreads();
   float acc[NP][2][4];
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  if (warp == kAttendWarps) {
+  if (warp == NW) {
     // ---- producer: lane i holds the pool row of box i of the walk (32 boxes at a time)
     const int boxes = kTileKeys / plan.box;
     const int* table = p.page_table + 1ll * slot * p.max_pages;
@@ -657,8 +703,8 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
   }
   __syncthreads();                       // the stages become the merge buffers
   float* po = reinterpret_cast<float*>(stages);                    // [warp][16][vp]
-  float* co = po + kAttendWarps * 16 * vp;                         // [16][vp] of the CTA
-  if (warp < kAttendWarps) {
+  float* co = po + NW * 16 * vp;                         // [16][vp] of the CTA
+  if (warp < NW) {
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       l[u] += __shfl_xor_sync(0xffffffffu, l[u], 1);
@@ -690,10 +736,10 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
     const int row = i / (vp / 4), c = 4 * (i % (vp / 4));
     float top = -INFINITY, sum = 0.f;
 #pragma unroll
-    for (int k = 0; k < kAttendWarps; ++k) top = fmaxf(top, ml[k * 32 + 2 * row]);
+    for (int k = 0; k < NW; ++k) top = fmaxf(top, ml[k * 32 + 2 * row]);
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int k = 0; k < kAttendWarps; ++k) {
+    for (int k = 0; k < NW; ++k) {
       const float wk = ml[k * 32 + 2 * row] == -INFINITY ? 0.f : ex2_approx(ml[k * 32 + 2 * row] - top);
       const float4 v = *reinterpret_cast<const float4*>(po + (k * 16 + row) * vp + c);
       sum += wk * ml[k * 32 + 2 * row + 1];
@@ -736,15 +782,15 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
   cluster.sync();                        // peers may still read this CTA's partial results
 }
 
-template <int KD, int NP>
+template <int NW, int KD, int NP>
 static int launch_group_attend(const ds41_group_attend_args& a, const AttendPlan& plan, cudaStream_t st) {
   const int smem = attend_smem(plan, a.dim_pad), row_len = a.kv_heads * (a.dim_pad + a.vdim_pad);
   static bool ready = false;
   cudaError_t e;
   if (!ready) {
-    e = cudaFuncSetAttribute(group_attend_mma_kernel<KD, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+    e = cudaFuncSetAttribute(group_attend_mma_kernel<NW, KD, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
     if (e != cudaSuccess) return e;
-    e = cudaFuncSetAttribute(group_attend_mma_kernel<KD, NP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    e = cudaFuncSetAttribute(group_attend_mma_kernel<NW, KD, NP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (e != cudaSuccess) return e;
     ready = true;
   }
@@ -753,16 +799,21 @@ static int launch_group_attend(const ds41_group_attend_args& a, const AttendPlan
                          plan.box, true);
   if (e != cudaSuccess) return e;
   const int m_tiles = (a.heads / a.kv_heads + 15) / 16;
-  const dim3 grid(a.n_splits, a.kv_heads * m_tiles, a.rows), block(kAttendThreads);
-  if (a.n_splits == 1) return launch_pdl(group_attend_mma_kernel<KD, NP>, grid, block, smem, st, pool, a, plan);
-  return launch_pdl_cluster(group_attend_mma_kernel<KD, NP>, grid, block, a.n_splits, smem, st, pool, a, plan);
+  const dim3 grid(a.n_splits, a.kv_heads * m_tiles, a.rows), block(32 * (NW + 1));
+  if (a.n_splits == 1) return launch_pdl(group_attend_mma_kernel<NW, KD, NP>, grid, block, smem, st, pool, a, plan);
+  return launch_pdl_cluster(group_attend_mma_kernel<NW, KD, NP>, grid, block, a.n_splits, smem, st, pool, a, plan);
 }
 
-template <int KD>
 static int dispatch_group_attend(const ds41_group_attend_args& a, const AttendPlan& plan, cudaStream_t st) {
-  if (a.vdim_pad <= 64) return launch_group_attend<KD, 4>(a, plan, st);
-  if (a.vdim_pad <= 128) return launch_group_attend<KD, 8>(a, plan, st);
-  return launch_group_attend<KD, 16>(a, plan, st);
+  if (plan.warps == 8) {
+    if (a.dim_pad > 128) return launch_group_attend<8, 16, 8>(a, plan, st);
+    if (a.dim_pad > 64) return a.vdim_pad <= 64 ? launch_group_attend<8, 8, 4>(a, plan, st) : launch_group_attend<8, 8, 8>(a, plan, st);
+    return a.vdim_pad <= 64 ? launch_group_attend<8, 4, 4>(a, plan, st) : launch_group_attend<8, 4, 8>(a, plan, st);
+  }
+  if (a.dim_pad > 128) return launch_group_attend<4, 16, 16>(a, plan, st);
+  if (a.vdim_pad > 128) return launch_group_attend<4, 8, 16>(a, plan, st);
+  if (a.dim_pad > 64) return launch_group_attend<4, 8, 8>(a, plan, st);
+  return a.vdim_pad <= 64 ? launch_group_attend<4, 4, 4>(a, plan, st) : launch_group_attend<4, 4, 8>(a, plan, st);
 }
 
 }  // namespace ds41
@@ -803,11 +854,8 @@ extern "C" int ds41_group_attend(const ds41_group_attend_args* a, void* stream) 
   if (!group_attend_ok(a) || a->n_splits < 1 || a->n_splits > kAttendSplits || a->rows > 65535) return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   AttendPlan plan;
-  if (plan_attend(*a, plan) && a->kv_heads * ((a->heads / a->kv_heads + 15) / 16) <= 65535) {
-    if (a->dim_pad <= 64) return dispatch_group_attend<4>(*a, plan, st);
-    if (a->dim_pad <= 128) return dispatch_group_attend<8>(*a, plan, st);
-    return dispatch_group_attend<16>(*a, plan, st);
-  }
+  if (plan_attend(*a, plan) && a->kv_heads * ((a->heads / a->kv_heads + 15) / 16) <= 65535)
+    return dispatch_group_attend(*a, plan, st);
   const size_t smem = (1ull * a->dim_pad + a->vdim_pad + 32) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const dim3 grid(a->heads, a->rows);

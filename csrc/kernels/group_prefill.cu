@@ -48,10 +48,10 @@ struct GroupForm {
   }
   // one tile of 128 keys, page by page; a page that is not leased reads as zeros (rows beyond the pool)
   __device__ void load_pages(uint8_t* dst, uint64_t* bar, int x, int chunks, int key) const {
-    const int* table = page_table + 1ll * row_slot[0] * max_pages;
+    const int slot = row_slot[0];
     for (int i = 0; i < kPreTile; i += page_tokens) {
       const int pg = (key + i) / page_tokens;
-      const int id = pg < max_pages ? __ldg(table + pg) : -1;
+      const int id = slot >= 0 && pg < max_pages ? __ldg(page_table + 1ll * slot * max_pages + pg) : -1;
       const int row = id >= 0 ? id * page_tokens : n_rows_pool;
       for (int c = 0; c < chunks; ++c) tma_load_3d(dst + c * kPreChunk + i * 128, &pool, bar, x + 64 * c, row, 0);
     }

@@ -218,13 +218,15 @@ __global__ void __launch_bounds__(kRouteThreads) route_softmax_kernel(ds41_route
   __shared__ unsigned int last;
   __shared__ int used[kRouteMax];
   __shared__ int slot_of_expert[kRouteMax];
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) last = atomicAdd(p.ticket, 1u) == gridDim.x - 1 ? 1u : 0u;
-  __syncthreads();
-  if (!last) return;
-  __threadfence();
   for (int e = tid; e < p.experts; e += kRouteThreads) used[e] = 0;
+  if (gridDim.x > 1) {
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) last = atomicAdd(p.ticket, 1u) == gridDim.x - 1 ? 1u : 0u;
+    __syncthreads();
+    if (!last) return;
+    __threadfence();
+  }
   for (int i = tid; i < p.max_active * p.row_w_ld; i += kRouteThreads) p.row_w[i] = 0.f;
   __syncthreads();
   const int n = p.rows * p.top;

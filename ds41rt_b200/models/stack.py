@@ -340,13 +340,13 @@ class GroupedAttention:
         return {"a": [(self.w_in.n, self.w_in.k)], "b": [(self.w_o.n, self.w_o.k)]}
 
     def splits(self, e: "StackEngine", rows: int) -> int:
-        """CTAs that share a row's keys: enough to fill the GPU about twice, static per batch size (a captured pass replays
-        while the context grows)."""
+        """CTAs that share a row's keys: enough to fill the GPU, static per batch size (a captured pass replays while the
+        context grows)."""
         sp = self.spec
         span = min(sp.chunk or e.cache.max_ctx, e.cache.max_ctx)
         blocks = rows * sp.kv_heads * -(-(sp.heads // sp.kv_heads) // 16)
-        n = max(1, min(2 * 148 // blocks, 16, -(-span // 128)))
-        return n if n <= 8 or n == 16 else 8
+        n = max(1, min(148 // blocks, 16, -(-span // 128)))
+        return n if n <= 8 else (16 if n == 16 and blocks <= 4 else 8)        # larger clusters than 8 do not fill the GPU
 
     def run(self, e: "StackEngine", l: int, R: int, src: int) -> Tuple[Proj, Optional[Proj]]:
         sp, k, c = self.spec, e.k, e.cache

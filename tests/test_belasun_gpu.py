@@ -336,6 +336,13 @@ class Attention:
         return got[..., :self.V]
 
 
+def test_attention_of_more_blocks_than_multiprocessors():
+    for shape in ((6, 2, 20, 24), (8, 1, 128, 128), (4, 2, 48, 80)):
+        c = Attention(*shape, 260, 200, 100, BF16, seed=7)
+        for splits in (1, 2):
+            torch.testing.assert_close(c.run("attend", splits), c.want(), rtol=0.03, atol=0.03)
+
+
 SHAPES = [(6, 2, 20, 24), (3, 3, 64, 64), (8, 1, 128, 128), (40, 2, 48, 80), (1, 1, 16, 200)]
 
 
