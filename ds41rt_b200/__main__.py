@@ -586,7 +586,7 @@ def main(argv=None) -> int:
     def model_args(p):
         from .models.registry import PRESETS
         p.add_argument("--model", default="tiny", choices=PRESETS)
-        p.add_argument("--layers", type=int, default=0, help="flash, genesun: number of layers to instantiate")
+        p.add_argument("--layers", type=int, default=0, help="flash, genesun-*, belasun-*: number of layers to instantiate")
         p.add_argument("--config", default="", help="config.json of any model family (overrides --model)")
 
     sub.add_parser("build")
@@ -640,7 +640,7 @@ def main(argv=None) -> int:
                     help="pinned host memory for snapshots that leave the device banks (0 = off; one-rank serving)")
     ps.add_argument("--reserve-gb", type=int, default=0, help="device memory to leave untouched by the KV pool")
     ps.add_argument("--peer-timeout", type=float, default=10.0, help="seconds without a heartbeat before a rank counts as gone")
-    ps.add_argument("--checkpoint", default="", help="directory with the model's safetensors files (ds41: official layout with an index; genesun: config.json "
+    ps.add_argument("--checkpoint", default="", help="directory with the model's safetensors files (ds41: official layout with an index; layer stacks: config.json "
                          "beside model.safetensors)")
     ps.add_argument("--tokenizer", default="", help="tokenizer.json; default: byte-level tokenizer")
     ps.add_argument("--expert-dtype", default="mxfp8", choices=["mxfp8", "mxfp4", "nvfp4", "bf16"])
