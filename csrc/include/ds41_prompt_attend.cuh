@@ -140,7 +140,8 @@ prompt_attend_kernel(const __grid_constant__ Form form, const PromptParams p) {
       return __all_sync(0xffffffffu, ok) != 0;
     };
     auto issue_s = [&](int t, int stage) {
-      const uint64_t qd = q_desc + static_cast<uint64_t>(t * q_bytes / 16), kd = k_desc + static_cast<uint64_t>(stage * k_bytes / 16);
+      const uint64_t qd = q_desc + static_cast<uint64_t>(t * q_bytes / 16);
+      const uint64_t kd = k_desc + static_cast<uint64_t>(stage * k_bytes / 16);
       for (int k = 0; k < kd16; ++k) {
         const uint64_t off = static_cast<uint64_t>((k >> 2) * (kPreChunk / 16) + (k & 3) * 2);
         umma_bf16_if(leader, tmem + t * 128, qd + off, kd + off, idesc_s, k > 0 ? 1u : 0u);
@@ -210,7 +211,8 @@ prompt_attend_kernel(const __grid_constant__ Form form, const PromptParams p) {
         if (edge) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (32 * c + i <= seen && (!Form::kLowerBound || 32 * c + i >= hidden)) top = fmaxf(top, __uint_as_float(v[i]) * p.scale_log2);
+            if (32 * c + i <= seen && (!Form::kLowerBound || 32 * c + i >= hidden))
+              top = fmaxf(top, __uint_as_float(v[i]) * p.scale_log2);
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) top = fmaxf(top, __uint_as_float(v[i]) * p.scale_log2);

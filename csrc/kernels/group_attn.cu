@@ -554,7 +554,8 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
     for (int i = warp; i < 16; i += NW) {
       const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q) + r * p.ld_q + (h0 + i) * dp;
       for (int d = lane * 8; d < dp; d += 256)
-        *reinterpret_cast<uint4*>(sq + i * KS + d) = h0 + i < h_end ? *reinterpret_cast<const uint4*>(q + d) : make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(sq + i * KS + d) =
+            h0 + i < h_end ? *reinterpret_cast<const uint4*>(q + d) : make_uint4(0, 0, 0, 0);
     }
   }
   __syncthreads();
@@ -688,7 +689,8 @@ group_attend_mma_kernel(const __grid_constant__ CUtensorMap pool, const ds41_gro
           uint32_t b[4][4];
 #pragma unroll
           for (int i = 0; i < 4; ++i)
-            if (16 * (i0 + i) < vp) ldmatrix_x4_trans(b[i][0], b[i][1], b[i][2], b[i][3], swizzled(vt, vrow, 2 * (i0 + i) + vpiece));
+            if (16 * (i0 + i) < vp)
+              ldmatrix_x4_trans(b[i][0], b[i][1], b[i][2], b[i][3], swizzled(vt, vrow, 2 * (i0 + i) + vpiece));
 #pragma unroll
           for (int i = 0; i < 4; ++i)
             if (16 * (i0 + i) < vp) {
@@ -807,7 +809,8 @@ static int launch_group_attend(const ds41_group_attend_args& a, const AttendPlan
 static int dispatch_group_attend(const ds41_group_attend_args& a, const AttendPlan& plan, cudaStream_t st) {
   if (plan.warps == 8) {
     if (a.dim_pad > 128) return launch_group_attend<8, 16, 8>(a, plan, st);
-    if (a.dim_pad > 64) return a.vdim_pad <= 64 ? launch_group_attend<8, 8, 4>(a, plan, st) : launch_group_attend<8, 8, 8>(a, plan, st);
+    if (a.dim_pad > 64)
+      return a.vdim_pad <= 64 ? launch_group_attend<8, 8, 4>(a, plan, st) : launch_group_attend<8, 8, 8>(a, plan, st);
     return a.vdim_pad <= 64 ? launch_group_attend<8, 4, 4>(a, plan, st) : launch_group_attend<8, 4, 8>(a, plan, st);
   }
   if (a.dim_pad > 128) return launch_group_attend<4, 16, 16>(a, plan, st);
@@ -828,7 +831,8 @@ extern "C" int ds41_attn_post(const ds41_attn_post_args* a, void* stream) {
     return cudaErrorInvalidValue;
   const int C = (a->heads + a->kv_heads) * a->dim_pad + a->kv_heads * a->vdim_pad;
   if ((a->taps > 1 && (a->conv == nullptr || a->state == nullptr)) || a->u.ld < a->u.col + C ||
-      a->ld_q < a->heads * a->dim_pad || (a->ld_q & 3) || (a->rot_dim & 1) || a->rot_dim < 0 || a->rot_dim > a->dim || a->rot_dim > 2 * kPostTurns || (a->rot_dim > 0 && a->freq == nullptr))
+      a->ld_q < a->heads * a->dim_pad || (a->ld_q & 3) || (a->rot_dim & 1) || a->rot_dim < 0 ||
+      a->rot_dim > a->dim || a->rot_dim > 2 * kPostTurns || (a->rot_dim > 0 && a->freq == nullptr))
     return cudaErrorInvalidValue;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   bool done = false;

@@ -103,7 +103,8 @@ extern "C" int ds41_group_prefill(const ds41_group_attend_args* a, void* stream)
   f.kv_heads = a->kv_heads; f.per_group = a->heads / a->kv_heads; f.chunk = a->chunk;
   f.max_pages = a->max_pages; f.page_tokens = a->page_tokens; f.n_rows_pool = a->n_pages * a->page_tokens;
   const int row_len = a->kv_heads * (p.dp + p.vp);
-  cudaError_t e = make_tensor_map_3d(&f.q, a->q, TmaDtype::kBF16, 1ull * p.heads * p.dp, p.rows, 1, a->ld_q * 2, 0, 64, kPreTile, true);
+  cudaError_t e = make_tensor_map_3d(&f.q, a->q, TmaDtype::kBF16, 1ull * p.heads * p.dp, p.rows, 1, a->ld_q * 2, 0, 64,
+                                     kPreTile, true);
   if (e != cudaSuccess) return e;
   e = make_tensor_map_3d(&f.pool, a->pool, TmaDtype::kBF16, row_len, f.n_rows_pool, 1, 2ull * row_len, 0, 64, a->page_tokens, true);
   if (e != cudaSuccess) return e;

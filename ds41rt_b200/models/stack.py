@@ -452,12 +452,14 @@ class RoutedExperts:
             return S.RoutedProj(ep.comb, self.ld, route=e.ids, top=top), gate
         I, n = self.ffp, e.max_active(sp)
         if e.f32:
-            e._run("gemm_fc1", S.gemm_f32, e.h, self.w13, e.moe_up, R, 2 * I, self.ld, e.ldh, self.ld, 2 * I, batch=n, sb=2 * I * self.ld,
-                   so=R * 2 * I, batch_map=e.active, n_active=e.n_active)
-            e._run("gated_act", k.ds41_gated_act, lib.ptr(e.moe_up), 2 * I, I, lib.ptr(e.row_w), e.moe_rows, lib.ptr(e.n_active), n, R,
-                   I, C.c_float(sp.limit), C.c_float(sp.alpha), C.c_float(sp.shift), lib.ptr(e.moe_act), I, lib.stream())
-            e._run("gemm_fc2", S.gemm_f32, e.moe_act, self.w2, e.moe_out, R, self.ld, I, I, I, self.ld, batch=n, sa=R * I,
-                   sb=self.ld * I, so=R * self.ld, batch_map=e.active, n_active=e.n_active)
+            some = dict(batch=n, batch_map=e.active, n_active=e.n_active)
+            e._run("gemm_fc1", S.gemm_f32, e.h, self.w13, e.moe_up, R, 2 * I, self.ld, e.ldh, self.ld, 2 * I,
+                   sb=2 * I * self.ld, so=R * 2 * I, **some)
+            e._run("gated_act", k.ds41_gated_act, lib.ptr(e.moe_up), 2 * I, I, lib.ptr(e.row_w), e.moe_rows,
+                   lib.ptr(e.n_active), n, R, I, C.c_float(sp.limit), C.c_float(sp.alpha), C.c_float(sp.shift),
+                   lib.ptr(e.moe_act), I, lib.stream())
+            e._run("gemm_fc2", S.gemm_f32, e.moe_act, self.w2, e.moe_out, R, self.ld, I, I, I, self.ld, sa=R * I,
+                   sb=self.ld * I, so=R * self.ld, **some)
         else:
             act = dict(act_limit=sp.limit, act_alpha=sp.alpha, act_shift=sp.shift)
             many = dict(batch=n, a_batches=E, batch_map=e.active, n_active=e.n_active, row_w=e.row_w, row_w_ld=e.moe_rows,

@@ -96,7 +96,8 @@ def work(cfg: StackConfig, R: int, n_keys: int, first: int, decode: bool, active
                     2.0 * pairs * H * (m.dim + m.vdim))
             else:
                 low = first - first % chunk if chunk else 0
-                add("group_prefill", (n_keys - low) * row * 2.0 + R * H * (m.dim + m.vdim) * 2.0, 2.0 * pairs * H * (m.dim + m.vdim))
+                add("group_prefill", (n_keys - low) * row * 2.0 + R * H * (m.dim + m.vdim) * 2.0,
+                    2.0 * pairs * H * (m.dim + m.vdim))
             gemm("gemm_o", W, H * m.vdim, 4)
         elif m.kind == "latent_attention":
             own = m.kv_from is None

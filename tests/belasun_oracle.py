@@ -235,7 +235,8 @@ def make_weights(doc, seed=0, steady=False):
                 w[p + "norm2"][:code] = 1.0
                 w[p + "mlp.router"], w[p + "mlp.router.b"] = torch.eye(E, W) * 4, torch.zeros(E)
             for e in range(E):
-                w.update({p + f"mlp.e{e}.gate": 2 * lin(ff, W), p + f"mlp.e{e}.up": lin(ff, W), p + f"mlp.e{e}.down": 2 * out(W, ff)})
+                w.update({p + f"mlp.e{e}.gate": 2 * lin(ff, W), p + f"mlp.e{e}.up": lin(ff, W),
+                          p + f"mlp.e{e}.down": 2 * out(W, ff)})
         w.update({p + "side.gate": lin(side, W), p + "side.proj": out(W, side), p + "side.norm": one(W)})
     return {k: v.to(torch.bfloat16).float() for k, v in w.items()}
 

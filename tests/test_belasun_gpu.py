@@ -387,11 +387,15 @@ class Post:
     """Projections of one request fed in portions through attn_post, followed by the attention launch that keeps the
     convolution's inputs, -> (queries, keys, values) of all positions."""
 
-    def __init__(self, T, H, G, D, V, taps, rot, dtype=F32, seed=0, norm=True):
+    def __init__(self, T, H, G, D, V, taps, rot, dtype=F32, seed=0, norm=True, packed=False):
+        """packed: the projection is one bf16 matrix (long passes), else two split-K planes."""
         g = gen(seed)
         self.T, self.H, self.G, self.D, self.V, self.taps, self.rot, self.dtype = T, H, G, D, V, taps, rot, dtype
         self.w = [torch.randn(h * d, max(taps, 1), generator=g) for h, d in ((H, D), (G, D), (G, V))]
         self.u = [torch.randn(T, h * d, generator=g) for h, d in ((H, D), (G, D), (G, V))]
+        self.packed = packed
+        if packed:
+            self.u = [x.to(BF16).float() for x in self.u]
         self.nq, self.nk = torch.rand(H * D, generator=g) + 0.5, torch.rand(G * D, generator=g) + 0.5
         self.norm = norm
 
@@ -413,7 +417,7 @@ class Post:
         heads = ((H, self.D, dp), (G, self.D, dp), (G, self.V, vp))
         u = torch.cat([pads(x, *h) for x, h in zip(self.u, heads)], 1)
         cols = u.shape[1]
-        planes = torch.stack([u * 0.25, u * 0.75]).contiguous().cuda()                        # two split-K planes
+        planes = (u.to(BF16)[None] if self.packed else torch.stack([u * 0.25, u * 0.75])).contiguous().cuda()
         conv = torch.cat([S.pad_heads(w, *h) for w, h in zip(self.w, heads)], 0).t().contiguous().cuda()
         nq, nk = (S.pad_heads(x, *h).cuda() for x, h in zip((self.nq, self.nk), heads))
         rot_dim, rope = belasun._rope(self.rot, "rot") if self.rot else (0, None)
@@ -429,7 +433,7 @@ class Post:
             slot = torch.ones(n, dtype=torch.int32).cuda()
             q, o = torch.zeros(n, H * dp, dtype=self.dtype).cuda(), torch.zeros(n, H * vp, dtype=self.dtype).cuda()
             a = S.AttnPostArgs()
-            a.u = S.Proj(x, cols, 2, n * cols).args()
+            a.u = (S.Proj(x, cols) if self.packed else S.Proj(x, cols, 2, n * cols)).args()
             a.conv, a.q_norm, a.k_norm, a.freq, a.state, a.q, a.pool = (lib.ptr(t) for t in (
                 conv if self.taps else None, nq if self.norm else None, nk if self.norm else None, freq, state, q, pages.pool))
             a.page_table, a.row_pos, a.row_slot, a.ld_q, a.eps = lib.ptr(pages.table), lib.ptr(pos), lib.ptr(slot), H * dp, eps
@@ -455,15 +459,18 @@ class Post:
         return q[..., :self.D], kk[..., :self.D], v[..., :self.V]
 
 
-@pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("sizes", [[100], [1], [2], [7, 1, 3, 2, 1, 1, 20]])
+@pytest.mark.parametrize("form", [(F32, False), (BF16, False), (BF16, True)])
+@pytest.mark.parametrize("sizes", [[100], [1], [2], [7, 1, 3, 2, 1, 1, 20], [40, 2, 38]])
 @pytest.mark.parametrize("shape", [dict(H=6, G=2, D=20, V=24, taps=4, rot=dict(base=40.0, dims=12, scaling=BANDS)),
                                    dict(H=1, G=1, D=16, V=16, taps=1, rot=dict(base=9.0, dims=16)),
                                    dict(H=20, G=4, D=128, V=64, taps=2, rot=dict(base=100.0, dims=128)),
+                                   dict(H=40, G=5, D=128, V=128, taps=3, rot=dict(base=100.0, dims=64)),
                                    dict(H=3, G=3, D=10, V=40, taps=7, rot=None, norm=False),
                                    dict(H=2, G=1, D=34, V=16, taps=0, rot=dict(base=100.0, dims=2))])
-def test_convolution_norm_rotation_and_cache_rows(shape, sizes, dtype):
-    c = Post(60, **shape, dtype=dtype, seed=shape["H"])
+def test_convolution_norm_rotation_and_cache_rows(shape, sizes, form):
+    """Every form of the launch: 32-bit or bf16 results, few rows or a block of them, portions shorter than the taps."""
+    dtype, packed = form
+    c = Post(80, **shape, dtype=dtype, seed=shape["H"], packed=packed)
     tol = 3e-5 if dtype == F32 else 1e-2
     for got, want in zip(c.run(sizes, 1e-3), c.want(1e-3)):
         torch.testing.assert_close(got, want, rtol=tol, atol=tol)
@@ -487,7 +494,8 @@ def test_router_choices_weights_and_plan(rows, experts, top):
     ids, wt, active, n_act, row_w, slot_of = i32(rows, top), f32(rows, top), i32(most), i32(1), f32(most, rows + 3), i32(rows, top)
     ticket = torch.zeros(1, dtype=torch.int32).cuda()
     a = S.RouteArgs()
-    a.z, a.bias, a.row_slot, a.ids, a.weights = S.Proj(Z, experts, 2, rows * experts).args(), *(lib.ptr(t) for t in (B, SL, ids, wt))
+    a.z = S.Proj(Z, experts, 2, rows * experts).args()
+    a.bias, a.row_slot, a.ids, a.weights = (lib.ptr(t) for t in (B, SL, ids, wt))
     a.active, a.n_active, a.row_w, a.slot_of, a.ticket = (lib.ptr(t) for t in (active, n_act, row_w, slot_of, ticket))
     a.rows, a.experts, a.top, a.max_active, a.row_w_ld = rows, experts, top, most, rows + 3
     for _ in range(2):                                         # the ticket is left ready for the next launch
@@ -546,8 +554,8 @@ def test_the_expert_activation_is_cut_where_it_should_be():
     x = torch.cat([g.reshape(1, -1), u.reshape(1, -1)], 1).cuda()
     n = g.numel()
     act, w, one = torch.zeros(1, n).cuda(), torch.full((1, 1), 0.5).cuda(), torch.ones(1, dtype=torch.int32).cuda()
-    _ok(k.ds41_gated_act(lib.ptr(x), 2 * n, n, lib.ptr(w), 1, lib.ptr(one), 1, 1, n, C.c_float(2.0), C.c_float(1.702), C.c_float(1.0),
-                         lib.ptr(act), n, lib.stream()))
+    _ok(k.ds41_gated_act(lib.ptr(x), 2 * n, n, lib.ptr(w), 1, lib.ptr(one), 1, 1, n, C.c_float(2.0), C.c_float(1.702),
+                         C.c_float(1.0), lib.ptr(act), n, lib.stream()))
     eye = {"gate": torch.ones(1, 1, dtype=torch.float64), "down": torch.ones(1, 1, dtype=torch.float64)}
     want = [float(expert(torch.ones(1, 1, dtype=torch.float64), dict(eye, gate=eye["gate"] * a, up=eye["gate"] * b), "", 2.0))
             for a, b in zip(g.reshape(-1).double(), u.reshape(-1).double())]
@@ -585,7 +593,8 @@ def test_result_norm_is_an_rms_norm_whatever_the_models_norm_is(rows, W):
     a.y, a.gate, a.post_w, a.x_in, a.x_out = S.Proj(Y, Lw).args(), S.NO_PROJ, lib.ptr(PW), lib.ptr(X), lib.ptr(out)
     a.ldx, a.ldh, a.rows, a.W, a.norm_kind, a.post_rms, a.eps, a.f32 = Lw, Lw, rows, W, 0, 1, 1e-5, 1
     _ok(k.ds41_resid_step(C.byref(a), lib.stream()))
-    torch.testing.assert_close(out[:, :W].cpu().double(), x.double() + rms_norm(y.double(), pw.double(), 1e-5), rtol=2e-5, atol=2e-5)
+    want = x.double() + rms_norm(y.double(), pw.double(), 1e-5)
+    torch.testing.assert_close(out[:, :W].cpu().double(), want, rtol=2e-5, atol=2e-5)
 
 
 def test_soft_cap_in_both_forms():
